@@ -469,6 +469,8 @@ typedef struct {
     const float* logdist;    /* [2][heads] or NULL: score <- score - r1[h] * ln(1 + r2[h] * (i - j)) with r1 = row 0, r2 = row 1 */
     int32_t cross_values;    /* != 0: every query head's weights are applied to the values of EVERY key/value head (the keys it reads stay
                               * those of its own): ws holds kv_heads * heads records per token, record (value head * heads + query head) */
+    int32_t chunk;           /* > 0 (then window is 0): query i sees key j <= i only when floor(i / chunk) = floor(j / chunk), positions
+                              * counted from the sequence's start */
 } sllm_seq_attn_opts;
 /* Causal softmax attention of every token over positions 0..pos of its own sequence: score = (q . k) * scale, query head h reads
  * key/value head h / (heads / kv_heads). Keys are visited in tiles of 32, cut into nsplit interleaved shares; the partial results
@@ -478,11 +480,25 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
                        float scale, const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws,
                        const sllm_seq_attn_opts* opts, sllm_stream_t stream);
 /* Merges the shares, normalises (sink [heads] or NULL: the denominator of head h also holds exp(sink[h]), a term without key or value),
- * turns every head's output back by -pos * vfreq[m] (vfreq NULL = not), multiplies head h by sigmoid(gate[t][h]) (gate NULL = not) and
- * stores out[t][h*dv ..]. */
+ * turns every head's output back by -pos * vfreq[m] (vfreq NULL = not), multiplies head h by sigmoid(gate[t][h]), or with gate_channels
+ * column c of head h by sigmoid(gate[t][h*dv + c]) (gate NULL = not), and stores out[t][h*dv ..] and / or out16, dense bf16 rows. */
 int sllm_seq_attention_finish(const sllm_seq_batch* b, const float* ws, int32_t nsplit, int32_t heads, int32_t dv, const double* vfreq,
-                              int32_t layout, const float* gate, int32_t ldg, const float* sink, float* out, int32_t ldo,
-                              sllm_stream_t stream);
+                              int32_t layout, const float* gate, int32_t ldg, int32_t gate_channels, const float* sink, float* out,
+                              int32_t ldo, void* out16, sllm_stream_t stream);
+/* Softmax attention whose SCORES are mixed over the heads before the softmax: own_g = (q_g . k of g's key head) * scale for every query
+ * head g, then score_h = sum_g talk[h][g] own_g (talk [heads][heads] fp32); values of head h's own value head. The keys of all heads of a
+ * token lie side by side in ONE pool row, k_pool [pages][1][page_len][kv_heads * dk]; v_pool [pages][kv_heads][page_len][dv]. Window,
+ * kept positions and chunks come from opts (the other options are not part of this form). q_mixed (or NULL): the mixed queries as dense
+ * bf16 [T][heads][kv_heads * dk], part u of head h = sum over the heads g of key head u of talk[h][g] q_g: with it, and bf16 pools, and
+ * widths the fragments take (sllm_seq_attention_talk_takes_mixed), steps run on the tensor cores and q is not read. The merge of
+ * sllm_seq_attention_finish (sink, gate per column, out / out16) is part of the call; ws [T][heads][nsplit][dv + 2] floats may be NULL
+ * for the tensor-core form with nsplit 1, which finishes in the same kernel. */
+int sllm_seq_attention_talk(const sllm_seq_batch* b, const float* q, int32_t ldq, const void* q_mixed, int32_t heads, int32_t kv_heads, int32_t dk,
+                            int32_t dv, float scale, const float* talk, const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit,
+                            float* ws, const sllm_seq_attn_opts* opts, const float* gate, int32_t ldg, const float* sink, float* out, int32_t ldo,
+                            void* out16, sllm_stream_t stream);
+/* 1 when head widths and counts fit the tensor-core form of sllm_seq_attention_talk */
+int sllm_seq_attention_talk_takes_mixed(int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, int32_t kv_dtype);
 /* Heads scaled to unit root mean square and the cache write, for mixers without rotation: bit 0 of `unit` = every query head of q (in
  * place), bit 1 = every key head, bit 2 = every value head is divided by sqrt(mean(head^2) + eps). share 1: the values (after the
  * division) are also kept in v_shared [T][kv_heads*dv]; share 2: v <- (1 - lambda) * v + lambda * v_shared (what an earlier layer kept
@@ -520,10 +536,13 @@ int sllm_seq_softcap(float* x, int64_t n, float cap, sllm_stream_t stream);
  * call read) moves them there. rms(v) = sqrt(mean(v^2) + eps). scales (or NULL): T floats of scratch; with it, steps of 64 tokens and
  * more run as two launches (sum and per-row scale, then the convolution element-wise) so that no row is normed more than once.
  * post_norm 0: the sum takes y as it is, x_out = x_in + y (a pre-norm layer). pre_w (or NULL) [d]: a weight per channel on the normed
- * row, stored as its distance from pre_w_offset: n[c] = pre_g * (pre_w_offset + pre_w[c]) * x[c] / rms(x). */
+ * row, stored as its distance from pre_w_offset: n[c] = pre_g * (pre_w_offset + pre_w[c]) * x[c] / rms(x). post_w (or NULL) [d]: a weight
+ * per channel on the normed y, x_out[c] = x_in[c] + post_g * post_w[c] * y[c] / rms(y). Without has_pre, h16 (if given) takes the stream after
+ * the sum as bf16 rows: the operand of a sublayer that reads the stream itself. */
 int sllm_seq_seam(const sllm_seq_batch* b, const float* x_in, float* x_out, const float* y, float post_g, int32_t has_pre, float pre_g,
                   float eps, const float* conv_w, int32_t taps, const float* ring, float* h, void* h16, float* stash, float* flush_ring,
-                  int32_t flush_taps, int32_t d, float* scales, int32_t post_norm, const float* pre_w, float pre_w_offset, sllm_stream_t stream);
+                  int32_t flush_taps, int32_t d, float* scales, int32_t post_norm, const float* pre_w, float pre_w_offset, const float* post_w,
+                  sllm_stream_t stream);
 /* out[t][c] = act(cb[c] + sum_j w[c][j] * x[t - taps + 1 + j][c]) (cb NULL = no bias; act 0 = none, 1 = silu), zeros before a sequence's
  * start; inputs before a portion come from ring [slots][taps-1][channels] (position p at row p % (taps-1)), which is NOT updated here
  * (sllm_seq_delta_rule, sllm_seq_ssd_scan, sllm_seq_selective_scan and sllm_seq_ring_store do that, after the convolution has run) */
@@ -566,6 +585,16 @@ int sllm_seq_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, in
                               int32_t kv_heads, const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps,
                               const double* freq, int32_t n_freq, int32_t layout, void* k_pool, void* v_pool, int32_t kv_dtype,
                               sllm_stream_t stream);
+/* The same preparation for mixers whose queries and keys are RMS-normed over the WHOLE projection (all heads of a token at once; weights
+ * q_norm_w [heads * dk] / k_norm_w [kv_heads * dk], NULL = not normed) before they are split into heads and turned. v: share 1 keeps the
+ * values in v_shared [T][kv_heads * dv], share 2 stores (1 - lambda) v + lambda v_shared. k_joint: the pool holds the heads of a token side by
+ * side ([pages][1][page_len][kv_heads * dk]) instead of head by head. q_mixed (or NULL; then talk [heads][heads] is not read): the queries
+ * mixed for sllm_seq_attention_talk go there as bf16 and q stays as it is; otherwise q is normed and turned in place. */
+int sllm_seq_wide_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk,
+                                   int32_t kv_heads, const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps,
+                                   const double* freq, int32_t n_freq, int32_t layout, float* v_shared, int32_t share, float lambda,
+                                   const float* talk, void* q_mixed, int32_t k_joint, void* k_pool, void* v_pool, int32_t kv_dtype,
+                                   sllm_stream_t stream);
 /* Heads mixed after the attention: in [T][kv_heads * heads * dv] as sllm_seq_attention_finish leaves it for cross_values (record = value
  * head * heads + query head); out[t][h] = sum_g mix[h][g] * in[t][(h / (heads / kv_heads)) * heads + g]: head h's mixed weights on the
  * values of its own key/value head. out fp32 [T][ldo] and / or out16 dense bf16 [T][heads * dv]. */
@@ -581,10 +610,11 @@ int sllm_seq_head_mix(const float* in, int32_t ldi, const float* mix, int32_t he
  * chosen (correction NULL = none; the lower index wins a tie); out / out16 [T][experts * ff] = act(up) * s for chosen experts with
  * weights (the first `experts` router outputs), zeros for the others; y [T][d] = (sum of s over chosen router outputs >= experts) * h:
  * those are experts whose output is their input. act 0 = exact gelu, 1 = tanh gelu, 2 = silu. route_w (or NULL) [T][n_route] = the
- * weights, zero where not chosen. */
+ * weights, zero where not chosen. shared_up (or NULL) [T][ldu]: a gated expert of width shared_ff that every token uses, its columns
+ * [gate | up]; its act(gate) * up follows the experts' columns, rows of out / out16 are then experts * ff + shared_ff wide. */
 int sllm_seq_moe_act(const float* logits, int32_t ldl, int32_t n_route, int32_t experts, int32_t top, const float* correction, const float* up,
                      int32_t ldu, int32_t ff, int32_t act, const float* h, int32_t ldh, int32_t d, float* out, void* out16, float* y,
-                     int32_t ldy, float* route_w, int32_t T, sllm_stream_t stream);
+                     int32_t ldy, float* route_w, const float* shared_up, int32_t shared_ff, int32_t T, sllm_stream_t stream);
 /* The same layer with the tokens gathered per expert, for steps of many tokens. sllm_seq_moe_route: routing as above; every (token,
  * chosen expert with weights) pair takes the next free row of that expert's buffer (counts [experts] int32, zeroed before the call;
  * buffers of cap >= T rows) and the token's input row h is copied there as bf16 (rows16 [experts][cap][d]) and / or fp32 (rows32);

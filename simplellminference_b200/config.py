@@ -65,7 +65,8 @@ PRESETS = {
 # ---------------------------------------------------------------------------------------------------------------------------
 @dataclass(frozen=True)
 class RotaryConfig:
-    """Rotary positions on the first ``dims`` dimensions of a head; ``scaling`` = YaRN-style (factor, original, fast, slow) or None."""
+    """Rotary positions on the first ``dims`` dimensions of a head; ``scaling`` = YaRN-style (factor, original, fast, slow) or by wavelength
+    bands (factor, original, low, high), whichever the mixer takes, or None."""
     dims: int
     base: float
     scaling: dict | None = None
@@ -292,11 +293,12 @@ class GatedFeedForwardConfig:
 @dataclass(frozen=True)
 class ExpertsConfig:
     """Mixture of experts: ``experts`` feed-forwards of width ``ff`` and ``identity`` experts without weights (their output is their
-    input) share one router; a token uses the ``top`` best."""
+    input) share one router; a token uses the ``top`` best. ``shared``: width of one more expert that every token uses (0 = none)."""
     experts: int
     identity: int
     top: int
     ff: int
+    shared: int = 0
 
 
 @dataclass(frozen=True)
@@ -483,8 +485,77 @@ class KodezenConfig:
                              int((c.get("canon") or {}).get("taps") or 1), float((c.get("embedding") or {}).get("scale", 1.0)), tuple(layers))
 
 
+@dataclass(frozen=True)
+class ScoreMixingAttentionConfig:
+    """Softmax attention whose queries and keys are normed over the whole projection and partly rotated (wavelength-band scaling; ``rot``
+    None = not), whose scores are mixed over the heads before the softmax, with a sink, a gate per output channel, keys visible inside
+    their own chunk of ``chunk`` positions only (None = all earlier keys), and values blended with those of the first such layer."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotaryConfig | None
+    chunk: int | None
+    v_mix: bool
+
+
+@dataclass(frozen=True)
+class LovulixLayerConfig:
+    type: str            # "attention"
+    mixer: ScoreMixingAttentionConfig
+    mlp: ExpertsConfig | None = None
+
+
+@dataclass(frozen=True)
+class LovulixConfig:
+    """The Lovulix design: sublayers read the residual stream itself and only their output is normed (RMS, a weight per channel); the mixer
+    is chunked attention with scores mixed over the heads before the softmax, the feed-forward a mixture of gated experts with sigmoid
+    scores on the experts' inputs and an expert every token uses. Every size and constant that may differ comes from config.json."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    logit_scale: float
+    layers: tuple
+
+    @staticmethod
+    def from_dict(c: dict) -> "LovulixConfig":
+        layers = []
+        for i, l in enumerate(c["layers"]):
+            m, mlp = l["mixer"], l.get("mlp")
+            if l["type"] != "attention":
+                raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
+            heads = int(m["heads"])
+            kv_heads = int(m.get("kv_heads") or heads)
+            if heads % kv_heads:
+                raise ValueError(f"layer {i}: {heads} query heads do not divide over {kv_heads} key/value heads")
+            dim, rot = int(m["dim"]), m.get("rot")
+            rot = RotaryConfig(int(rot["dims"]), float(rot["base"]), rot.get("scaling") or None) if rot and int(rot.get("dims") or 0) > 0 else None
+            if rot is not None and (rot.dims > dim or rot.dims % 2):
+                raise ValueError(f"layer {i}: {rot.dims} rotary dimensions do not fit heads of {dim}")
+            size = (m.get("mask") or {}).get("size")
+            mixer = ScoreMixingAttentionConfig(heads, kv_heads, dim, int(m.get("vdim") or dim), float(m["scale"]), rot, int(size) if size else None,
+                                               bool(m.get("v_mix")))
+            ff = None
+            if mlp is not None:
+                if mlp.get("kind", "moe") != "moe":
+                    raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not part of this design")
+                r = mlp["router"]
+                ff = ExpertsConfig(int(r["experts"]), 0, int(r["top"]), int(mlp["expert"]["ff"]), int((mlp.get("shared") or {}).get("ff") or 0))
+                if not 1 <= ff.top <= ff.experts:
+                    raise ValueError(f"layer {i}: {ff.top} of {ff.experts} experts")
+            layers.append(LovulixLayerConfig(l["type"], mixer, ff))
+        shared = [l.mixer for l in layers if l.mixer.v_mix]
+        if any((m.kv_heads, m.vdim) != (shared[0].kv_heads, shared[0].vdim) for m in shared):
+            raise ValueError("layers that blend their values with the first such layer's need the same key/value heads and value width")
+        scale = c.get("logit_scale")
+        return LovulixConfig(c["architecture"], int(c["vocab"]), int(c["width"]), float((c.get("norm") or {}).get("eps", 1e-6)),
+                             1.0 if scale is None else float(scale), tuple(layers))
+
+
 CONFIG_READERS = {"Munazen": MunazenConfig.from_dict, "Sopetar": SopetarConfig.from_dict, "Vasosun": VasosunConfig.from_dict,
-                  "Kodezen": KodezenConfig.from_dict}
+                  "Kodezen": KodezenConfig.from_dict, "Lovulix": LovulixConfig.from_dict}
 
 
 def read_model_config(model_dir: str):

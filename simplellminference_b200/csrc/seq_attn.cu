@@ -12,15 +12,13 @@
 // (16-byte shared loads, rows padded by 4 floats: conflict-free) and dv/32 output columns for the weighted sum; online softmax per query
 // with warp reductions. The key tiles are dealt to `nsplit` CTAs in turn (long contexts with few queries: decode), every CTA leaves
 // (max, sum, unnormalised output) and seq_attention_finish_kernel merges them.
-#include <climits>
-
-#include "seq_common.cuh"
+#include "seq_attn.cuh"
 
 namespace sllm {
 
 extern int g_tune_seq_attn_mma;   // runtime.cu: 1 (default) = tensor-core attention body where it applies, 0 = always the fp32 body
 
-constexpr int kBQ = 32, kBK = 32, kQW = 4;   // queries per CTA, keys per tile, queries per warp
+constexpr int kQW = 4;   // queries per warp of the fp32 body
 
 struct AttnArgs {
     sllm_seq_batch b;
@@ -36,20 +34,7 @@ struct AttnArgs {
     // Every query head's weights on every key/value head's values: `heads` then counts kv_heads * q_heads results, result u = (value
     // head u / q_heads, query head u % q_heads); the query head reads the KEYS of its own key/value head as always. Otherwise q_heads = heads.
     int q_heads, cross;
-};
-
-// The key tiles a CTA whose queries lie at positions first .. last has to visit: the tiles of the kept first positions, then the tiles
-// from the one that holds the oldest key inside the first query's window up to the last query's own tile.
-struct TileList {
-    int n_keep, lo, n;
-    __device__ __forceinline__ TileList(int first, int last, int window, int keep_first, int tile) {
-        const int nkt = last / tile + 1;
-        const int oldest = window > first ? 0 : first - window + 1;
-        lo = oldest / tile;
-        n_keep = min(lo, (min(keep_first, oldest) + tile - 1) / tile);
-        n = n_keep + nkt - lo;
-    }
-    __device__ __forceinline__ int tile_of(int idx) const { return idx < n_keep ? idx : lo + idx - n_keep; }
+    int chunk;                // > 0: a query sees its own chunk of `chunk` positions only (then window / keep_first are not used)
 };
 
 __device__ __forceinline__ float seq_score(float dot, float scale, float softcap, float slope, float r1, float r2, int qpos, int key) {
@@ -59,10 +44,6 @@ __device__ __forceinline__ float seq_score(float dot, float scale, float softcap
     if (r1 != 0.0f) sc -= r1 * log1pf(r2 * (float)(qpos - key));
     return sc;
 }
-__device__ __forceinline__ bool seq_sees(int qpos, int key, int window, int keep_first) {
-    return key <= qpos && (qpos - key < window || key < keep_first);
-}
-
 template <typename KV, int kMaxDvChunks>   // dv <= 32 * kMaxDvChunks
 __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs p) {
     extern __shared__ __align__(16) float sm[];
@@ -111,8 +92,11 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs p) {
         r1[i] = has ? p.logdist[row_qhead(warp * kQW + i)] : 0.0f;
         r2[i] = has ? p.logdist[p.q_heads + row_qhead(warp * kQW + i)] : 0.0f;
     }
+    int wnd[kQW];             // how far back each row sees
+#pragma unroll
+    for (int i = 0; i < kQW; ++i) wnd[i] = seq_row_window(row_pos(warp * kQW + i), p.window, p.chunk);
     const int last_pos = row_pos(nq - 1);
-    const TileList tiles(row_pos(0), last_pos, p.window, p.keep_first, kBK);
+    const TileList tiles(row_pos(0), last_pos, seq_row_window(row_pos(0), p.window, p.chunk), p.keep_first, kBK);
     for (int idx = split; idx < tiles.n; idx += p.nsplit) {
         const int j0 = tiles.tile_of(idx) * kBK;
         const int page = b.block_table[(size_t)slot * b.max_pages + j0 / b.page_len], in_page = j0 % b.page_len;
@@ -167,7 +151,7 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs p) {
 #pragma unroll
         for (int i = 0; i < kQW; ++i) {
             const int qi = warp * kQW + i;
-            const bool see = qi < nq && seq_sees(row_pos(qi), j0 + lane, p.window, p.keep_first);
+            const bool see = qi < nq && seq_sees(row_pos(qi), j0 + lane, wnd[i], p.keep_first);
             const float sc = see ? seq_score(s[i], p.scale, p.softcap, slope[i], r1[i], r2[i], row_pos(qi), j0 + lane) : -INFINITY;
             const float mn = fmaxf(m[i], warp_max(sc));
             const float corr = (mn == -INFINITY) ? 1.0f : expf(m[i] - mn);   // m = -inf: nothing accumulated yet, expf(-inf) = 0 is right too
@@ -218,29 +202,6 @@ __global__ void __launch_bounds__(256) seq_attention_kernel(AttnArgs p) {
 // register-for-register onto an A fragment of P. K and V tiles are staged row-major as cached (rows padded by 16 bytes: conflict-free
 // fragment loads; V's B fragments come out of ldmatrix.trans) by cp.async into two stages, the next tile in flight while this one is
 // multiplied; four warps = two query heads of one kv head share a staged tile when the group size is even. Writes the same (max, sum, unnormalised output) records as the fp32 body.
-__device__ __forceinline__ void mma_bf16_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { return (uint32_t)f32_to_bf16_bits(lo) | ((uint32_t)f32_to_bf16_bits(hi) << 16); }
-// p = hi + lo with both terms bf16: hi = round(p), lo = round(p - hi)
-__device__ __forceinline__ void split_bf16(float p0, float p1, uint32_t* hi, uint32_t* lo) {
-    const uint16_t h0 = f32_to_bf16_bits(p0), h1 = f32_to_bf16_bits(p1);
-    *hi = (uint32_t)h0 | ((uint32_t)h1 << 16);
-    *lo = pack_bf16(p0 - __uint_as_float((uint32_t)h0 << 16), p1 - __uint_as_float((uint32_t)h1 << 16));
-}
-
-
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-// 16 bytes global -> shared without passing through registers; bytes = 0 writes zeros and reads nothing
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, int bytes) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
 // kExact: dk = 16 * kMmaDkSteps and dv = 8 * kMmaDvTiles exactly — the loops over fragments then have no run-time bounds, and the compiler
 // is free to interleave independent products (the common head widths are instantiated so).
 template <int kMmaDkSteps, int kMmaDvTiles, bool kExact>   // dk <= 16 * kMmaDkSteps (multiple of 16), dv <= 8 * kMmaDvTiles (multiple of 8)
@@ -264,7 +225,8 @@ __global__ void __launch_bounds__(128) seq_attention_mma_kernel(AttnArgs p) {
     const int r0 = wq * 16 + g, r1 = r0 + 8;           // this thread's two query rows inside the tile
     const bool ok0 = r0 < nq, ok1 = r1 < nq;
     const int last_pos = pos0 + nq - 1;
-    const TileList tiles(pos0, last_pos, p.window, p.keep_first, kBK);
+    const TileList tiles(pos0, last_pos, seq_row_window(pos0, p.window, p.chunk), p.keep_first, kBK);
+    const int wnd0 = seq_row_window(pos0 + r0, p.window, p.chunk), wnd1 = seq_row_window(pos0 + r1, p.window, p.chunk);
     const float slope = p.slopes ? p.slopes[hq] : 0.0f;
     const float ld1 = p.logdist ? p.logdist[hq] : 0.0f, ld2 = p.logdist ? p.logdist[p.q_heads + hq] : 0.0f;
 
@@ -342,7 +304,7 @@ __global__ void __launch_bounds__(128) seq_attention_mma_kernel(AttnArgs p) {
             for (int e = 0; e < 4; ++e) {
                 const int key = j0 + nt * 8 + 2 * c + (e & 1);
                 const int qpos = pos0 + ((e < 2) ? r0 : r1);
-                const bool see = ((e < 2) ? ok0 : ok1) && seq_sees(qpos, key, p.window, p.keep_first);
+                const bool see = ((e < 2) ? ok0 : ok1) && seq_sees(qpos, key, (e < 2) ? wnd0 : wnd1, p.keep_first);
                 s[nt][e] = see ? seq_score(s[nt][e], p.scale, p.softcap, slope, ld1, ld2, qpos, key) : -INFINITY;
             }
             mx0 = fmaxf(mx0, fmaxf(s[nt][0], s[nt][1]));
@@ -427,7 +389,8 @@ __global__ void __launch_bounds__(128) seq_attention_mma_kernel(AttnArgs p) {
 // Warp 0 turns the shares' (max, sum) into one weight per share (exp(m_s - max) / total, zero for a share that saw no key); every thread
 // then adds its column over the shares with coalesced loads; pairs meet through shared memory for the rotation.
 __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __restrict__ ws, int nsplit, int heads, int dv, const double* __restrict__ vfreq,
-                                            int layout, const float* __restrict__ gate, int ldg, const float* __restrict__ sink, float* __restrict__ out, int ldo) {
+                                            int layout, const float* __restrict__ gate, int ldg, int gate_channels, const float* __restrict__ sink, float* __restrict__ out,
+                                            int ldo, uint16_t* __restrict__ out16) {
     extern __shared__ float fsm[];
     float* s_w = fsm;            // [nsplit]
     float* s_o = fsm + nsplit;   // [dv]
@@ -459,10 +422,16 @@ __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __res
         s_o[col] = v;
     }
     __syncthreads();
-    const float gv = gate ? seq_sigmoid(gate[(size_t)t * ldg + h]) : 1.0f;
-    float* orow = out + (size_t)t * ldo + (size_t)h * dv;
+    // one gate per head, or (gate_channels) one per column of the row of heads
+    const float gv = gate && !gate_channels ? seq_sigmoid(gate[(size_t)t * ldg + h]) : 1.0f;
+    const float* grow = gate && gate_channels ? gate + (size_t)t * ldg + (size_t)h * dv : nullptr;
+    auto put = [&](int c, float v) {
+        v *= grow ? seq_sigmoid(grow[c]) : gv;
+        if (out) out[(size_t)t * ldo + (size_t)h * dv + c] = v;
+        if (out16) out16[((size_t)t * heads + h) * dv + c] = f32_to_bf16_bits(v);
+    };
     if (!vfreq) {
-        if (col < dv) orow[col] = s_o[col] * gv;
+        if (col < dv) put(col, s_o[col]);
         return;
     }
     const int half = dv / 2, mi = threadIdx.x;
@@ -471,8 +440,8 @@ __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __res
         const float u = s_o[ia], v = s_o[ib];
         float sn, cs;
         seq_angle(b.tok_pos[t], vfreq[mi], &sn, &cs);
-        orow[ia] = (u * cs + v * sn) * gv;    // rotation by the negative angle
-        orow[ib] = (v * cs - u * sn) * gv;
+        put(ia, u * cs + v * sn);             // rotation by the negative angle
+        put(ib, v * cs - u * sn);
     }
 }
 
@@ -544,6 +513,19 @@ static int check_batch(const sllm_seq_batch* b, const char* who) {
     return SLLM_OK;
 }
 
+int sllm::launch_attention_finish(const sllm_seq_batch* b, const float* ws, int nsplit, int heads, int dv, const double* vfreq, int layout, const float* gate,
+                                  int ldg, int gate_channels, const float* sink, float* out, int ldo, uint16_t* out16, cudaStream_t st) {
+    if (int rc = check_batch(b, "seq_attention_finish")) return rc;
+    SLLM_REQUIRE(ws && (out || out16) && nsplit >= 1 && heads > 0 && dv > 0 && (!vfreq || dv % 2 == 0), SLLM_EINVAL, "seq_attention_finish: bad argument");
+    SLLM_REQUIRE(dv <= 1024 && nsplit <= 8192, SLLM_ENOTSUP, "seq_attention_finish: value width %d / %d shares beyond what one CTA merges", dv, nsplit);
+    const int threads = std::max(32, (dv + 31) / 32 * 32);
+    seq_attention_finish_kernel<<<b->T * heads, threads, (size_t)(nsplit + dv) * sizeof(float), st>>>(*b, ws, nsplit, heads, dv, vfreq, layout, gate, ldg, gate_channels,
+                                                                                                     sink, out, ldo, out16);
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    return SLLM_OK;
+}
+
 extern "C" {
 
 int sllm_seq_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk, int32_t kv_heads,
@@ -578,14 +560,15 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
     SLLM_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0, SLLM_EINVAL, "seq_attention: %d query heads over %d kv heads", heads, kv_heads);
     SLLM_REQUIRE(dv > 0 && dv <= 512, SLLM_ENOTSUP, "seq_attention: value width %d beyond 512", dv);
     SLLM_REQUIRE(!v_in_k || dv <= dk, SLLM_EINVAL, "seq_attention: %d value columns inside key rows of %d", dv, dk);
-    SLLM_REQUIRE(!opts || (opts->window >= 0 && opts->keep_first >= 0 && opts->softcap >= 0.0f), SLLM_EINVAL, "seq_attention: bad options");
+    SLLM_REQUIRE(!opts || (opts->window >= 0 && opts->keep_first >= 0 && opts->softcap >= 0.0f && opts->chunk >= 0), SLLM_EINVAL, "seq_attention: bad options");
+    SLLM_REQUIRE(!opts || !opts->chunk || !opts->window, SLLM_EINVAL, "seq_attention: a window or chunks, not both");
     SLLM_REQUIRE(b->page_len % kBK == 0, SLLM_ENOTSUP, "seq_attention: pages of a multiple of %d positions", kBK);
     SLLM_REQUIRE(nsplit >= 1 && nsplit <= 65535, SLLM_EINVAL, "seq_attention: nsplit");
     SLLM_REQUIRE(kv_dtype == SLLM_F32 || kv_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_attention: fp32 or bf16 pools");
     const int dkp = ((dk + 3) & ~3) + 4;
     const size_t smem = ((size_t)(kBQ + kBK) * dkp + (v_in_k ? 0 : (size_t)kBK * dv)) * sizeof(float);
     SLLM_REQUIRE(smem <= (size_t)smem_optin_bytes(), SLLM_ENOTSUP, "seq_attention: heads of %d + %d floats need %zu bytes of shared memory", dk, dv, smem);
-    AttnArgs p{*b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, nsplit, ws, 0, INT_MAX, 0, 0.0f, nullptr, 0, nullptr, heads, 0};
+    AttnArgs p{*b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, nsplit, ws, 0, INT_MAX, 0, 0.0f, nullptr, 0, nullptr, heads, 0, 0};
     if (opts && opts->cross_values) {
         SLLM_REQUIRE(!v_in_k, SLLM_EINVAL, "seq_attention: values of every head need a value pool");
         p.cross = 1;
@@ -598,6 +581,7 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
         p.slopes = opts->slopes;
         p.v_in_k = v_in_k;
         p.logdist = opts->logdist;
+        p.chunk = opts->chunk;
     }
     dim3 grid(b->n_qtiles, p.heads, nsplit);
     // steps that hold a portion of a prompt, bf16 pools, head widths the fragments take: the tensor-core body
@@ -638,16 +622,9 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
 }
 
 int sllm_seq_attention_finish(const sllm_seq_batch* b, const float* ws, int32_t nsplit, int32_t heads, int32_t dv, const double* vfreq, int32_t layout,
-                              const float* gate, int32_t ldg, const float* sink, float* out, int32_t ldo, sllm_stream_t stream) {
-    if (int rc = check_batch(b, "seq_attention_finish")) return rc;
-    SLLM_REQUIRE(ws && out && nsplit >= 1 && heads > 0 && dv > 0 && (!vfreq || dv % 2 == 0), SLLM_EINVAL, "seq_attention_finish: bad argument");
-    SLLM_REQUIRE(dv <= 1024 && nsplit <= 8192, SLLM_ENOTSUP, "seq_attention_finish: value width %d / %d shares beyond what one CTA merges", dv, nsplit);
-    const int threads = std::max(32, (dv + 31) / 32 * 32);
-    seq_attention_finish_kernel<<<b->T * heads, threads, (size_t)(nsplit + dv) * sizeof(float), as_stream(stream)>>>(*b, ws, nsplit, heads, dv, vfreq, layout, gate,
-                                                                                                                  ldg, sink, out, ldo);
-    ++g_launches;
-    SLLM_LAUNCH_CHECK();
-    return SLLM_OK;
+                              const float* gate, int32_t ldg, int32_t gate_channels, const float* sink, float* out, int32_t ldo, void* out16,
+                              sllm_stream_t stream) {
+    return launch_attention_finish(b, ws, nsplit, heads, dv, vfreq, layout, gate, ldg, gate_channels, sink, out, ldo, (uint16_t*)out16, as_stream(stream));
 }
 
 }  // extern "C"

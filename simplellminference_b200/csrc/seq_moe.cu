@@ -24,7 +24,8 @@ __device__ __forceinline__ float moe_act(float z, int kind) {
 // one CTA per token; shared: scores [n_route], weights [n_route]
 __global__ void seq_moe_act_kernel(const float* __restrict__ logits, int ldl, int n_route, int experts, int top, const float* __restrict__ correction,
                                    const float* __restrict__ up, int ldu, int ff, int act, const float* __restrict__ h, int ldh, int d,
-                                   float* __restrict__ out, uint16_t* __restrict__ out16, float* __restrict__ y, int ldy, float* __restrict__ route_w) {
+                                   float* __restrict__ out, uint16_t* __restrict__ out16, float* __restrict__ y, int ldy, float* __restrict__ route_w,
+                                   const float* __restrict__ shared_up, int shared_ff) {
     extern __shared__ float msm[];
     float* s_score = msm;
     float* s_choice = msm + n_route;
@@ -82,7 +83,7 @@ __global__ void seq_moe_act_kernel(const float* __restrict__ logits, int ldl, in
     if (route_w)
         for (int e = threadIdx.x; e < n_route; e += blockDim.x) route_w[(size_t)t * n_route + e] = s_w[e];
     const float* ur = up + (size_t)t * ldu;
-    const size_t orow = (size_t)t * experts * ff;
+    const size_t orow = (size_t)t * (experts * ff + shared_ff);
     const bool gated = act & kMoeGated, on_input = act & kMoeScaleInput;
     for (int i = threadIdx.x; i < experts * ff; i += blockDim.x) {
         const int e = i / ff;
@@ -96,6 +97,12 @@ __global__ void seq_moe_act_kernel(const float* __restrict__ logits, int ldl, in
         if (out) out[orow + i] = v;
         if (out16) out16[orow + i] = f32_to_bf16_bits(v);
     }
+    const float* sr = shared_up + (size_t)t * ldu;       // the expert every token uses, with weight one
+    for (int i = threadIdx.x; i < shared_ff; i += blockDim.x) {
+        const float v = moe_act(sr[i], act) * sr[shared_ff + i];
+        if (out) out[orow + experts * ff + i] = v;
+        if (out16) out16[orow + experts * ff + i] = f32_to_bf16_bits(v);
+    }
     const float ident = s_identity;
     for (int j = threadIdx.x; j < d; j += blockDim.x) y[(size_t)t * ldy + j] = ident * h[(size_t)t * ldh + j];
 }
@@ -106,16 +113,17 @@ using namespace sllm;
 
 extern "C" int sllm_seq_moe_act(const float* logits, int32_t ldl, int32_t n_route, int32_t experts, int32_t top, const float* correction, const float* up,
                                 int32_t ldu, int32_t ff, int32_t act, const float* h, int32_t ldh, int32_t d, float* out, void* out16, float* y, int32_t ldy,
-                                float* route_w, int32_t T, sllm_stream_t stream) {
+                                float* route_w, const float* shared_up, int32_t shared_ff, int32_t T, sllm_stream_t stream) {
+    SLLM_REQUIRE(shared_ff >= 0 && (shared_ff == 0 || shared_up), SLLM_EINVAL, "seq_moe_act: a shared expert needs its columns");
     SLLM_REQUIRE(logits && up && h && y && (out || out16) && T > 0 && ff > 0 && d > 0, SLLM_EINVAL, "seq_moe_act: bad argument");
     SLLM_REQUIRE(experts >= 0 && n_route >= experts && n_route > 0 && top >= 1 && top <= n_route, SLLM_EINVAL, "seq_moe_act: %d of %d router outputs, %d experts with weights",
                  top, n_route, experts);
     SLLM_REQUIRE(act >= 0 && (act & 3) <= 2 && act < 32, SLLM_EINVAL, "seq_moe_act: activation 0 (gelu), 1 (tanh gelu) or 2 (silu), plus SLLM_MOE_* bits");
     SLLM_REQUIRE(n_route <= 4096, SLLM_ENOTSUP, "seq_moe_act: %d router outputs beyond 4096", n_route);
-    const int work = std::max(experts * ff, d);
+    const int work = std::max(experts * ff + shared_ff, d);
     const int threads = T >= 64 ? 256 : std::min(1024, std::max(128, (work + 31) / 32 * 32));
     seq_moe_act_kernel<<<T, threads, 3 * (size_t)n_route * sizeof(float), as_stream(stream)>>>(logits, ldl, n_route, experts, top, correction, up, ldu, ff, act, h, ldh,
-                                                                                                d, out, (uint16_t*)out16, y, ldy, route_w);
+                                                                                                d, out, (uint16_t*)out16, y, ldy, route_w, shared_up, shared_ff);
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     return SLLM_OK;

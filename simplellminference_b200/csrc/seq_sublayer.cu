@@ -2,7 +2,9 @@
 // through a short causal convolution: x <- x + g_post * y / rms(y) (the residual sum, fp32), then h = n + conv(n) with
 // n = g_pre * x / rms(x) and conv a per-channel causal convolution over time, as ONE kernel. A norm here has one number as its weight.
 // The same seam serves pre-norm layers: the sum may take y as it is (no norm on the sublayer's output), and the norm in front of the
-// next sublayer may carry a weight per channel stored as its distance from a constant, n = g_pre * (offset + w[c]) * x / rms(x).
+// next sublayer may carry a weight per channel stored as its distance from a constant, n = g_pre * (offset + w[c]) * x / rms(x); and layers
+// whose only norm sits on the sublayer's OUTPUT, with a weight per channel: x <- x + g_post * w[c] * y / rms(y), the next sublayer reading x
+// itself (the seam then leaves x as bf16 operand rows).
 //
 // The convolution reaches taps-1 tokens back. Inside a portion those are rows of this step: a CTA (one per token) recomputes the
 // residual sum and the norm of its predecessors from the sublayer's input and output (x is therefore read from one buffer and written to
@@ -27,9 +29,12 @@ struct SeamArgs {
     int d;
     int post_norm;                            // 0 = y is added as it is
     const float* pre_w; float pre_off;        // [d] or NULL: channel c of the normed row is also multiplied by pre_off + pre_w[c]
+    const float* post_w;                      // [d] or NULL: channel c of the normed sublayer output is also multiplied by post_w[c]
 };
 
 __device__ __forceinline__ float seam_gain(const SeamArgs& p, int j) { return p.pre_w ? p.pre_off + p.pre_w[j] : 1.0f; }
+
+__device__ __forceinline__ float seam_post(const SeamArgs& p, int j) { return p.post_w ? p.post_w[j] : 1.0f; }
 
 // is token t among the last `keep` tokens of its portion?
 __device__ __forceinline__ bool seam_is_last(const sllm_seq_batch& b, int t, int slot, int keep) {
@@ -72,9 +77,10 @@ __global__ void seq_seam_kernel(SeamArgs p) {
         for (int j = threadIdx.x; j < d; j += blockDim.x) {
             float v = p.x_in[r + j];
             if (p.y) {
-                v = fmaf(p.y[r + j], inv_y, v);
+                v = fmaf(p.y[r + j] * seam_post(p, j), inv_y, v);
                 if (back == 0) p.x_out[r + j] = v;
             }
+            if (!p.has_pre && p.h16) p.h16[r + j] = f32_to_bf16_bits(v);
             s_row[j] = v;
             ss = fmaf(v, v, ss);
         }
@@ -105,6 +111,70 @@ __global__ void seq_seam_kernel(SeamArgs p) {
     }
 }
 
+// ---- the same seam without a convolution or a ring, rows of a multiple of four floats: the row stays in registers ----------------------------
+// CTA = token, R groups of four channels per thread; x and y are read once, in flight together, and everything is stored once.
+template <int R>
+__global__ void __launch_bounds__(1024) seq_seam_row_kernel(SeamArgs p) {
+    __shared__ float red[33];
+    const int d4 = p.d / 4;
+    const size_t r = (size_t)blockIdx.x * p.d;
+    float x[R][4], y[R][4];
+    float sy = 0.0f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+        const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float4 xv = j < d4 ? *reinterpret_cast<const float4*>(p.x_in + r + 4 * j) : zero;
+        const float4 yv = j < d4 && p.y ? *reinterpret_cast<const float4*>(p.y + r + 4 * j) : zero;
+        x[i][0] = xv.x; x[i][1] = xv.y; x[i][2] = xv.z; x[i][3] = xv.w;
+        y[i][0] = yv.x; y[i][1] = yv.y; y[i][2] = yv.z; y[i][3] = yv.w;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sy = fmaf(y[i][e], y[i][e], sy);
+    }
+    auto pack = [&](const float (&v)[4]) {
+        return make_uint2((uint32_t)f32_to_bf16_bits(v[0]) | ((uint32_t)f32_to_bf16_bits(v[1]) << 16), (uint32_t)f32_to_bf16_bits(v[2]) | ((uint32_t)f32_to_bf16_bits(v[3]) << 16));
+    };
+    float ss = 0.0f;
+    if (p.y) {
+        const float inv_y = p.post_norm ? p.post_g / sqrtf(block_sum(sy, red) / (float)p.d + p.eps) : 1.0f;
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int j = threadIdx.x + i * blockDim.x;
+            if (j >= d4) continue;
+            const float4 w = p.post_w ? *reinterpret_cast<const float4*>(p.post_w + 4 * j) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+            x[i][0] = fmaf(y[i][0] * w.x, inv_y, x[i][0]);
+            x[i][1] = fmaf(y[i][1] * w.y, inv_y, x[i][1]);
+            x[i][2] = fmaf(y[i][2] * w.z, inv_y, x[i][2]);
+            x[i][3] = fmaf(y[i][3] * w.w, inv_y, x[i][3]);
+            *reinterpret_cast<float4*>(p.x_out + r + 4 * j) = make_float4(x[i][0], x[i][1], x[i][2], x[i][3]);
+        }
+    }
+    if (!p.has_pre) {
+        if (p.h16)
+#pragma unroll
+            for (int i = 0; i < R; ++i) {
+                const int j = threadIdx.x + i * blockDim.x;
+                if (j < d4) *reinterpret_cast<uint2*>(p.h16 + r + 4 * j) = pack(x[i]);
+            }
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss = fmaf(x[i][e], x[i][e], ss);     // channels beyond the row are zeros
+    const float inv = p.pre_g / sqrtf(block_sum(ss, red) / (float)p.d + p.eps);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+        if (j >= d4) continue;
+        const float4 w = p.pre_w ? *reinterpret_cast<const float4*>(p.pre_w + 4 * j) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float off = p.pre_w ? p.pre_off : 1.0f;
+        const float v[4] = {x[i][0] * inv * (off + w.x), x[i][1] * inv * (off + w.y), x[i][2] * inv * (off + w.z), x[i][3] * inv * (off + w.w)};
+        *reinterpret_cast<float4*>(p.h + r + 4 * j) = make_float4(v[0], v[1], v[2], v[3]);
+        if (p.h16) *reinterpret_cast<uint2*>(p.h16 + r + 4 * j) = pack(v);
+    }
+}
+
 // ---- the same seam as two launches, for steps of many tokens: no row is normed more than once ------------------------------------------
 // (1) one CTA per token: the residual sum and the scale of the next norm, scale[t] = g_pre / rms(x_new[t]);
 // (2) element-wise over (token, channel): h = n + conv(n) with n = scale * x_new read from the step's rows (complete after launch 1) or
@@ -124,7 +194,7 @@ __global__ void seq_seam_sum_kernel(SeamArgs p, float* __restrict__ scale) {
         }
         const float inv_y = p.post_norm ? p.post_g / sqrtf(block_sum(sy, red) / (float)d + p.eps) : 1.0f;
         for (int j = threadIdx.x; j < d; j += blockDim.x) {
-            const float v = fmaf(seam_sm[j], inv_y, p.x_in[r + j]);
+            const float v = fmaf(seam_sm[j] * seam_post(p, j), inv_y, p.x_in[r + j]);
             p.x_out[r + j] = v;
             ss = fmaf(v, v, ss);
         }
@@ -222,7 +292,8 @@ using namespace sllm;
 
 extern "C" int sllm_seq_seam(const sllm_seq_batch* b, const float* x_in, float* x_out, const float* y, float post_g, int32_t has_pre, float pre_g,
                              float eps, const float* conv_w, int32_t taps, const float* ring, float* h, void* h16, float* stash, float* flush_ring,
-                             int32_t flush_taps, int32_t d, float* scales, int32_t post_norm, const float* pre_w, float pre_w_offset, sllm_stream_t stream) {
+                             int32_t flush_taps, int32_t d, float* scales, int32_t post_norm, const float* pre_w, float pre_w_offset, const float* post_w,
+                             sllm_stream_t stream) {
     SLLM_REQUIRE(b && b->T > 0 && b->tok_slot && b->tok_pos, SLLM_EINVAL, "seq_seam: incomplete batch description");
     SLLM_REQUIRE(x_in && d > 0 && (!y || (x_out && x_out != x_in)), SLLM_EINVAL, "seq_seam: the residual sum needs a second buffer for x");
     SLLM_REQUIRE(!has_pre || h, SLLM_EINVAL, "seq_seam: no output for the normed rows");
@@ -232,11 +303,22 @@ extern "C" int sllm_seq_seam(const sllm_seq_batch* b, const float* x_in, float* 
     const size_t smem = 2 * (size_t)d * sizeof(float);
     SLLM_REQUIRE(smem <= (size_t)smem_optin_bytes() - 1024, SLLM_ENOTSUP, "seq_seam: rows of %d floats do not fit shared memory", d);
     if (smem > 48 * 1024) SLLM_CUDA(cudaFuncSetAttribute(seq_seam_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    SeamArgs p{*b, x_in, x_out, y, post_g, has_pre, pre_g, eps, conv_w, taps, ring, h, (uint16_t*)h16, stash, flush_ring, flush_taps, d, post_norm, pre_w, pre_w_offset};
+    SeamArgs p{*b, x_in, x_out, y, post_g, has_pre, pre_g, eps, conv_w, taps, ring, h, (uint16_t*)h16, stash, flush_ring, flush_taps, d, post_norm, pre_w, pre_w_offset, post_w};
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    if (!conv_w && !flush_ring && d % 4 == 0 && d <= 4 * 4 * 1024 && aligned(x_in) && aligned(x_out) && aligned(y) && aligned(h) && aligned(h16) && aligned(pre_w) &&
+        aligned(post_w)) {
+        // many tokens: CTAs of 256 threads with up to four groups of channels each; few: a thread per group of channels
+        const int d4 = d / 4, cta = std::min(1024, (((b->T >= 64 ? std::max(std::min(d4, 256), (d4 + 3) / 4) : d4) + 31) / 32) * 32), per = (d4 + cta - 1) / cta;
+        if (per == 1) seq_seam_row_kernel<1><<<b->T, cta, 0, as_stream(stream)>>>(p);
+        else if (per == 2) seq_seam_row_kernel<2><<<b->T, cta, 0, as_stream(stream)>>>(p);
+        else seq_seam_row_kernel<4><<<b->T, cta, 0, as_stream(stream)>>>(p);
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     const int threads = b->T >= 64 ? (d >= 2048 ? 256 : 128) : std::min(1024, std::max(128, (d + 31) / 32 * 32));
     if (scales && has_pre && conv_w && b->T >= 64 && b->T <= 65535) {       // many tokens: two launches, every row normed once
         seq_seam_sum_kernel<<<b->T, threads, smem / 2, as_stream(stream)>>>(p, scales);
-        auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
         const int vec = d % 4 == 0 && aligned(x_in) && aligned(x_out) && aligned(ring) && aligned(h) && aligned(stash) && aligned(flush_ring) &&
                         (h16 == nullptr || ((uintptr_t)h16 % 8) == 0);
         seq_seam_conv_kernel<<<dim3(b->T, std::max(1, std::min(4, d / 4096))), 256, 0, as_stream(stream)>>>(p, scales, vec);

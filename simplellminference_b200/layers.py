@@ -4,10 +4,12 @@ values and a head gate over a paged cache; softmax attention with unit-rms heads
 the first positions; latent attention (one cached row per token, absorbed form) with a sink and a head gate; a Griffin-style recurrent block (short causal convolution + real-gated linear recurrent unit);
 gated linear attention with a decay per key channel; a PolyNorm feed-forward; a clamped gated feed-forward; softmax attention with a charge on the
 logarithm of the distance and a query temperature; the gated delta rule behind short convolutions; a gated (silu) feed-forward and a mixture of
-experts with identity experts (softmax or sigmoid scores, plain or gated experts, the score on the expert's output or on its input);
+experts with identity experts (softmax or sigmoid scores, plain or gated experts, the score on the expert's output or on its input, an
+expert every token uses);
 state-space duality (Mamba-2) and the selective scan (Mamba) behind short convolutions; softmax attention whose queries and keys pass a
 convolution and a per-head norm, whose values are the keys before the norm, and whose weights are mixed over the heads after the softmax;
-a feed-forward with biases and the exact gelu. A mechanism says which per-sequence state it needs
+a feed-forward with biases and the exact gelu; chunked softmax attention with whole-projection norms on queries and keys, scores mixed over
+the heads before the softmax, a sink, blended values and a gate per channel. A mechanism says which per-sequence state it needs
 (``state_spec``); the engine's state manager owns that memory and hands it to ``forward`` — no mechanism keeps a cache of its own.
 
 Additive to the reference, whose only model is the Llama forward of source/model/model.cpp:40-140."""
@@ -41,6 +43,25 @@ def yarn_frequencies(dims: int, base: float, scaling: dict | None):
         ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
         out.append(fi / factor * ramp + fi * (1.0 - ramp))
     return out, 0.1 * math.log(factor) + 1.0
+
+
+def band_frequencies(dims: int, base: float, scaling: dict | None):
+    """Angular step per position of each of the dims/2 rotary pairs, scaled by wavelength bands. ``scaling`` = {factor, original, low,
+    high}: wavelengths below original/high keep their frequency, those above original/low are slowed down by ``factor``, and between
+    the two the frequency is a blend whose weight is linear in original / wavelength."""
+    out = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims)
+        if scaling:
+            factor, turns = float(scaling["factor"]), float(scaling["original"]) * f / (2.0 * math.pi)      # original / wavelength
+            low, high = float(scaling["low"]), float(scaling["high"])
+            if turns < low:
+                f /= factor
+            elif turns <= high and high > low:
+                keep = (turns - low) / (high - low)
+                f = (1.0 - keep) * f / factor + keep * f
+        out.append(f)
+    return out
 
 
 class FusedLinear:
@@ -526,6 +547,83 @@ class TalkingHeadsAttention:
         return rows16 is not None
 
 
+class ScoreMixingAttention:
+    """Softmax attention over a paged cache with grouped query heads in which: q and k are RMS-normed over the WHOLE projection (weights
+    ``q.norm`` / ``k.norm`` of its size) and then rotated on the first ``rot.dims`` dimensions of each head (pairs i, i + dims/2; frequencies
+    scaled by wavelength bands); the heads' scores are mixed BEFORE the softmax, score_h <- sum_g talk[h][g] score_g; a query sees the
+    earlier keys of its own chunk of positions only; the softmax's denominator also holds exp(``sink``_h); the values may be blended with
+    those an earlier layer kept (``share`` = "keep" / "blend", lambda = ``vmix``; the cache holds the blended ones); and the heads'
+    results are multiplied channel by channel with sigmoid(``g`` h). State per sequence: the pool of key rows (all key heads of a token side
+    by side: every mixed score needs all of them) and the value pool.
+
+    Portions of prompts in bf16 mode hand the attention kernel mixed QUERIES (the sum over the heads of a key head taken on the query, so
+    that a head's mixed score is one product with the whole key row); single tokens, the fp32 mode and widths the fragments do not take
+    score every head once and mix the scores."""
+
+    key_tile = 32        # keys per tile of the kernel that mixes scores; the tensor-core form takes twice as many
+
+    def __init__(self, cfg, w, pre, ops, device, eps, layout=1, share=None):
+        self.cfg, self.ops, self.eps, self.layout, self.share = cfg, ops, eps, layout, share
+        H, G = cfg.heads, cfg.kv_heads
+        self.gated = pre + "g" in w
+        self.inputs = [(w[pre + n], w.get(pre + n + ".b")) for n in ("q", "k", "v")] + ([(w[pre + "g"], None)] if self.gated else [])
+        vector = lambda n, size: self._vector(w, pre + n, size)   # noqa: E731
+        self.q_norm, self.k_norm = vector("q.norm", H * cfg.dim), vector("k.norm", G * cfg.dim)
+        self.sink = vector("sink", H)
+        self.talk = w[pre + "talk"].float().contiguous() if pre + "talk" in w else torch.eye(H, device=device)
+        if tuple(self.talk.shape) != (H, H):
+            raise ValueError(f"{pre}talk is {tuple(self.talk.shape)} for {H} heads")
+        self.lam = float(w[pre + "vmix"].float().item()) if share == "blend" else 0.0
+        self.n_freq = cfg.rot.dims // 2 if cfg.rot is not None else 0
+        self.freq = torch.tensor(band_frequencies(cfg.rot.dims, cfg.rot.base, cfg.rot.scaling), dtype=torch.float64, device=device) if self.n_freq else None
+        self.opts = ops.attention_options(chunk=cfg.chunk)
+        self.mixes_queries = ops.attention_talk_takes_mixed(H, G, cfg.dim, cfg.vdim)
+        self.out = FusedLinear([(w[pre + "o"], w.get(pre + "o.b"))], ops, device)
+        self.width = H * cfg.vdim
+
+    @staticmethod
+    def _vector(w, name, size):
+        if name not in w:
+            return None
+        v = w[name].float().contiguous()
+        if tuple(v.shape) != (size,):
+            raise ValueError(f"{name} is {tuple(v.shape)}, the configuration says {size}")
+        return v
+
+    def state_spec(self):
+        c = self.cfg
+        return {"pages": [("k", 1, c.kv_heads * c.dim), ("v", c.kv_heads, c.vdim)], "slots": []}
+
+    def _shares(self, step, mixed: bool) -> int:
+        """How many CTAs share a work item's key tiles. Depends on the batch's shape only, never on the context lengths (steps of single
+        tokens are captured as graphs)."""
+        c = self.cfg
+        visible = min(c.chunk or step.max_len, step.max_len)
+        tile = 2 * self.key_tile if mixed else self.key_tile
+        tiles = -(-visible // tile) + 1                # a chunk may begin inside a tile
+        if step.T == step.nseg:
+            return max(1, min(tiles, step.sms // step.nseg))
+        ctas = step.b.n_qtiles * (c.heads // math.gcd(c.heads // c.kv_heads, 4)) if mixed else -(-step.T // 4)
+        return max(1, min(tiles, 2 * step.sms // ctas))
+
+    def forward(self, step, cols, ld, state, out):
+        c, ops, T = self.cfg, self.ops, step.T
+        H, G, dk, dv = c.heads, c.kv_heads, c.dim, c.vdim
+        q, k, v = cols[:3]
+        gate = cols[3] if self.gated else None
+        kept = step.scratch("v_kept", T * G * dv) if self.share else None
+        mixed = step.scratch("talk_q", (T * H * G * dk + 1) // 2) if self.mixes_queries and T > step.nseg else None
+        ops.wide_normed_rotary_kv(step.b, q, ld, H, dk, k, ld, G, v, ld, dv, self.q_norm, self.k_norm, self.eps, self.freq, self.n_freq, self.layout, state["k"],
+                                  state["v"], step.st, v_shared=kept, share={None: 0, "keep": 1, "blend": 2}[self.share], lam=self.lam, talk=self.talk,
+                                  q_mixed=mixed, k_joint=True)
+        nsplit = self._shares(step, mixed is not None)
+        ws = step.scratch("attn_ws", T * H * nsplit * (dv + 2)) if mixed is None or nsplit > 1 else None
+        rows16 = self.out.operand_rows(step)
+        ops.attention_talk(step.b, q, ld, mixed, H, G, dk, dv, c.scale, self.talk, state["k"], state["v"], nsplit, ws, step.st, opts=self.opts, gate_ptr=gate,
+                           ldg=ld, sink=self.sink, out=None if rows16 is not None else out, ldo=self.width, out16=rows16)
+        return rows16 is not None
+
+
 class MixerGroup:
     """One or more mechanisms reading the same input: their input projections run as one fused product, each mechanism's result goes
     through its own output projection, and the results are added with the given weights."""
@@ -666,7 +764,11 @@ class ExpertsFeedForward:
     per expert an up product, the activation, a down product over the rows in use (their count never leaves the device), and a kernel
     that adds each token's rows times their scores. Steps of one or two tokens (decoding) whose experts are large take the indexed
     form: the router, a routing kernel, and ONE up and ONE down launch in which every (token, choice) pair streams only its own expert's
-    matrix, chosen on the device. All forms give the same numbers up to where the score is multiplied in."""
+    matrix, chosen on the device. All forms give the same numbers up to where the score is multiplied in.
+
+    ``shared`` > 0 (tensors ``shared.gate`` / ``shared.up`` / ``shared.down``; gated experts): one more expert of that width which every token
+    uses with weight one. Its first product rides with the experts' (wide form) or the router's (the others), its second with the wide down
+    product or as a product of its own that adds to the result."""
 
     activation = 0          # the exact (erf) gelu
     GATED, SCALE_INPUT, SIGMOID = 4, 8, 16      # SLLM_MOE_* bits beside the activation
@@ -694,19 +796,38 @@ class ExpertsFeedForward:
         self.correction = w[pre + "correction"].float().contiguous() if pre + "correction" in w else None
         # experts first, router last: the experts' columns then start at a 16-byte boundary for every ff
         first = [torch.cat([w[f"{pre}e{e}.gate"], w[f"{pre}e{e}.up"]], dim=0) if gated else w[f"{pre}e{e}.up"] for e in range(E)]
-        self.up = FusedLinear([(m, None) for m in first] + [(w[pre + "router"], None)], ops, device, pad_rows=8)
-        self.down = FusedLinear([(torch.cat([w[f"{pre}e{e}.down"] for e in range(E)], dim=1).contiguous(), None)], ops, device)
-        self.wide = E * cfg.ff                     # columns of the activation = rows of the concatenated down matrices
-        self.wide_up = E * self.ff_up              # columns of all experts' first products; the router's follow
+        self.shared_ff = cfg.shared
+        if self.shared_ff and not gated:
+            raise ValueError("an expert that every token uses is a gated one here")
+        common = [(w[f"{pre}shared.{n}"], None) for n in ("gate", "up")] if self.shared_ff else []
+        self.up = FusedLinear([(m, None) for m in first] + common + [(w[pre + "router"], None)], ops, device, pad_rows=8)
+        downs = [w[f"{pre}e{e}.down"] for e in range(E)] + ([w[pre + "shared.down"]] if self.shared_ff else [])
+        self.down = FusedLinear([(torch.cat(downs, dim=1).contiguous(), None)], ops, device)
+        self.wide = E * cfg.ff + self.shared_ff    # columns of the activation = rows of the concatenated down matrices
+        self.wide_up = E * self.ff_up              # columns of all experts' first products; the shared expert's, then the router's follow
+        if self.up.sizes[E] != (self.shared_ff or self.n_route):
+            raise ValueError(f"{pre}shared.gate has {self.up.sizes[E]} rows, the configuration says {self.shared_ff}")
         # the gathered form: the router as a product of its own, the down matrices one behind the other [E][d][ff]
         self.gathers = cfg.top < self.n_route and E > 0
         if self.gathers:
-            self.router = FusedLinear([(w[pre + "router"], None)], ops, device, pad_rows=64)    # wide enough for the tensor-core tiles
+            # padded to be wide enough for the tensor-core tiles
+            self.router = FusedLinear(common + [(w[pre + "router"], None)], ops, device, pad_rows=64)
+            self.shared_down = FusedLinear([(w[pre + "shared.down"], None)], ops, device) if self.shared_ff else None
             self.down_each = torch.stack([w[f"{pre}e{e}.down"] for e in range(E)]).contiguous()
 
     @property
     def proj(self):
         return self.up
+
+    def _add_shared(self, step, first_ptr, ld, y):
+        """y += the shared expert's result; its [gate | up] columns lie at ``first_ptr``."""
+        if not self.shared_ff:
+            return
+        n = self.shared_ff
+        rows16 = self.shared_down.operand_rows(step)
+        act = step.scratch("moe_shared", step.T * n)
+        self.ops.gated_act(first_ptr, ld, first_ptr + n * F32B, ld, None if rows16 is not None else act, n, step.T, n, step.st, out16=rows16)
+        self.shared_down(step, act.data_ptr(), n, y.data_ptr(), self.shared_down.N, accumulate=True, a16_ready=rows16 is not None)
 
     def _forward_gathered(self, step, h, y, h16_ready=False):
         c, ops, T, d, st = self.cfg, self.ops, step.T, self.up.K, step.st
@@ -726,7 +847,8 @@ class ExpertsFeedForward:
         act = step.scratch("moe_act", -(-E * cap * ff // per)).data_ptr()
         down_out = step.scratch("moe_down", E * cap * d).data_ptr()
         ops.zero(counts, 4 * E, st)
-        ops.moe_route(logits.data_ptr(), ldl, self.n_route, E, top, self.correction, h, d, d, counts, cap, sel_e, sel_pos, sel_w, ident,
+        scores = logits.data_ptr() + 2 * self.shared_ff * F32B         # the shared expert's columns come first
+        ops.moe_route(scores, ldl, self.n_route, E, top, self.correction, h, d, d, counts, cap, sel_e, sel_pos, sel_w, ident,
                       rows if tc else None, None if tc else rows, T, st, mode=self.mode)
         wb = self.up.w.element_size()
         for e in range(E):
@@ -739,6 +861,7 @@ class ExpertsFeedForward:
             ops.linear(a, ff, self.down_each, ff, None, down_out + 4 * e * cap * d, d, cap, d, ff, st, scratch=a if tc else None, a16_ready=tc,
                        rows_dev=counts + 4 * e, w_ptr=self.down_each.data_ptr() + e * d * ff * wb)
         ops.moe_combine(down_out, sel_e, sel_pos, sel_w, top, ident, h, d, cap, d, y, d, T, st)
+        self._add_shared(step, logits.data_ptr(), ldl, y)
 
     def _gathered_pays(self, T: int) -> bool:
         c = self.cfg
@@ -761,7 +884,8 @@ class ExpertsFeedForward:
         sel_e, sel_pos, sel_w, ident = book + 4 * E, book + 4 * (E + pairs), book + 4 * (E + 2 * pairs), book + 4 * (E + 3 * pairs)
         # the products read the token's row as it is; a score on the expert's input is applied to their results (they are linear), so the
         # routing kernel is asked for the plain scores
-        ops.moe_route(logits.data_ptr(), ldl, self.n_route, E, top, self.correction, h, d, d, None, T, sel_e, sel_pos, sel_w, ident, None, None, T, st,
+        scores = logits.data_ptr() + 2 * self.shared_ff * F32B         # the shared expert's columns come first
+        ops.moe_route(scores, ldl, self.n_route, E, top, self.correction, h, d, d, None, T, sel_e, sel_pos, sel_w, ident, None, None, T, st,
                       mode=self.mode & ~self.SCALE_INPUT)
         up_out = step.scratch("moe_up", pairs * fu).data_ptr()
         down_out = step.scratch("moe_down", pairs * d).data_ptr()
@@ -776,6 +900,7 @@ class ExpertsFeedForward:
         ops.linear_indexed(act, ff, ff, 1, self.down_each, ff, d * ff, sel_e, down_out, d, d, pairs, d, ff, st)
         # row (t, k) of down_out is pair t * top + k: the combine kernel's (expert, row) address with buffers of 0 rows
         ops.moe_combine(down_out, sel_e, sel_pos, weights, top, ident, h, d, 0, d, y, d, T, st)
+        self._add_shared(step, logits.data_ptr(), ldl, y)
 
     def forward(self, step, h, y, h16_ready=False):
         if self._gathered_pays(step.T):
@@ -787,6 +912,8 @@ class ExpertsFeedForward:
         self.up(step, h.data_ptr(), d, z.data_ptr(), N, a16_ready=h16_ready)
         rows16 = self.down.operand_rows(step)
         act = step.scratch("ff_act", T * self.wide)   # fp32 rows; not written when the product reads the bf16 rows
-        self.ops.moe_act(z.data_ptr() + self.wide_up * F32B, N, self.n_route, c.experts, c.top, self.correction, z.data_ptr(), N, c.ff, self.mode,
-                         h, d, d, None if rows16 is not None else act, rows16, y, d, T, step.st)
+        common = z.data_ptr() + self.wide_up * F32B
+        self.ops.moe_act(common + 2 * self.shared_ff * F32B, N, self.n_route, c.experts, c.top, self.correction, z.data_ptr(), N, c.ff, self.mode,
+                         h, d, d, None if rows16 is not None else act, rows16, y, d, T, step.st, shared_ptr=common if self.shared_ff else None,
+                         shared_ff=self.shared_ff)
         self.down(step, act.data_ptr(), self.wide, y.data_ptr(), d, accumulate=True, a16_ready=rows16 is not None)

@@ -38,6 +38,8 @@ class Step:
         self.b = _lib.SeqBatch()
         self.st = None
         self.nsplit = 1
+        self.max_len = engine.max_len     # the most positions a request can hold
+        self.sms = torch.cuda.get_device_properties(engine.device).multi_processor_count if engine.device.type == "cuda" else 1
         self.prev_ids = None      # device array [T]: the token before each token in its sequence, -1 at a sequence's start
 
     def scratch(self, name: str, n_floats: int) -> torch.Tensor:

@@ -89,18 +89,36 @@ class Ops:
         self._ck(self.lib.sllm_seq_attention(C.byref(b), q_ptr, ldq, heads, kv_heads, dk, dv, scale, _p(k_pool), _p(v_pool), self.kv_dtype, nsplit,
                                              _p(ws), C.byref(opts) if opts is not None else None, st))
 
-    def attention_finish(self, b, ws, nsplit, heads, dv, vfreq, layout, gate_ptr, ldg, out, ldo, st, sink=None):
-        self._ck(self.lib.sllm_seq_attention_finish(C.byref(b), _p(ws), nsplit, heads, dv, _p(vfreq), layout, gate_ptr, ldg, _p(sink), _p(out), ldo, st))
+    def attention_finish(self, b, ws, nsplit, heads, dv, vfreq, layout, gate_ptr, ldg, out, ldo, st, sink=None, gate_channels=False, out16=None):
+        """``gate_channels``: the gate has a column per output column instead of one per head."""
+        self._ck(self.lib.sllm_seq_attention_finish(C.byref(b), _p(ws), nsplit, heads, dv, _p(vfreq), layout, gate_ptr, ldg, int(bool(gate_channels)), _p(sink),
+                                                    _p(out), ldo, _p(out16), st))
+
+    def attention_talk(self, b, q_ptr, ldq, q_mixed, heads, kv_heads, dk, dv, scale, talk, k_pool, v_pool, nsplit, ws, st, opts=None, gate_ptr=None, ldg=0,
+                       sink=None, out=None, ldo=0, out16=None):
+        """Attention with the scores mixed over the heads before the softmax, merge and gate (per column) included; ``q_mixed``: the mixed
+        queries ``wide_normed_rotary_kv`` left (tensor-core form), else ``q_ptr`` is read."""
+        self._ck(self.lib.sllm_seq_attention_talk(C.byref(b), q_ptr, ldq, _p(q_mixed), heads, kv_heads, dk, dv, scale, _p(talk), _p(k_pool), _p(v_pool), self.kv_dtype,
+                                                  nsplit, _p(ws), C.byref(opts) if opts is not None else None, gate_ptr, ldg, _p(sink), _p(out), ldo, _p(out16), st))
+
+    def attention_talk_takes_mixed(self, heads, kv_heads, dk, dv):
+        return bool(self.lib.sllm_seq_attention_talk_takes_mixed(heads, kv_heads, dk, dv, self.kv_dtype))
 
     @staticmethod
-    def attention_options(window=0, keep_first=0, softcap=0.0, slopes=None, values_in_keys=False, logdist=None, cross_values=False):
+    def attention_options(window=0, keep_first=0, softcap=0.0, slopes=None, values_in_keys=False, logdist=None, cross_values=False, chunk=0):
         """The options structure of ``attention``; the caller keeps the ``slopes`` and ``logdist`` tensors alive."""
         return _lib.SeqAttnOpts(int(window or 0), int(keep_first or 0), float(softcap or 0.0), _p(slopes), int(bool(values_in_keys)), _p(logdist),
-                                int(bool(cross_values)))
+                                int(bool(cross_values)), int(chunk or 0))
 
     def normed_rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, q_norm_w, k_norm_w, eps, freq, n_freq, layout, k_pool, v_pool, st):
         self._ck(self.lib.sllm_seq_normed_rotary_kv(C.byref(b), q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, _p(q_norm_w), _p(k_norm_w), eps,
                                                     _p(freq), n_freq, layout, _p(k_pool), _p(v_pool), self.kv_dtype, st))
+
+    def wide_normed_rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, q_norm_w, k_norm_w, eps, freq, n_freq, layout, k_pool, v_pool,
+                              st, v_shared=None, share=0, lam=0.0, talk=None, q_mixed=None, k_joint=False):
+        self._ck(self.lib.sllm_seq_wide_normed_rotary_kv(C.byref(b), q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, _p(q_norm_w), _p(k_norm_w), eps,
+                                                         _p(freq), n_freq, layout, _p(v_shared), share, lam, _p(talk), _p(q_mixed), int(bool(k_joint)), _p(k_pool),
+                                                         _p(v_pool), self.kv_dtype, st))
 
     def head_mix(self, x, ldx, mix, heads, kv_heads, dv, out, ldo, T, st, out16=None):
         self._ck(self.lib.sllm_seq_head_mix(_p(x), ldx, _p(mix), heads, kv_heads, dv, _p(out), ldo, _p(out16), T, st))
@@ -120,11 +138,12 @@ class Ops:
         self._ck(self.lib.sllm_seq_embed_pair(_p(ids), _p(prev_ids), _p(table), _p(pairs), self.w_dtype, vocab, d, buckets, mul_prev, mul_cur, _p(out), T, st))
 
     def seam(self, b, x_in, d, st, x_out=None, y=None, post_g=1.0, pre_g=None, eps=0.0, conv_w=None, taps=1, ring=None, h=None, h16=None, stash=None,
-             flush_ring=None, flush_taps=0, scales=None, post_norm=True, pre_w=None, pre_w_offset=0.0):
+             flush_ring=None, flush_taps=0, scales=None, post_norm=True, pre_w=None, pre_w_offset=0.0, post_w=None):
         """x_out = x_in + post_g * y / rms(y) (if ``y``; ``post_norm`` False: x_in + y), then h = n + conv(n), n = pre_g * x / rms(x) (if
-        ``pre_g`` is given), times (pre_w_offset + pre_w) per channel if ``pre_w`` is."""
+        ``pre_g`` is given), times (pre_w_offset + pre_w) per channel if ``pre_w`` is; ``post_w``: a weight per channel on the normed y;
+        without ``pre_g``, ``h16`` takes the stream after the sum."""
         self._ck(self.lib.sllm_seq_seam(C.byref(b), _p(x_in), _p(x_out), _p(y), post_g, int(pre_g is not None), pre_g or 0.0, eps, _p(conv_w), taps, _p(ring),
-                                        _p(h), _p(h16), _p(stash), _p(flush_ring), flush_taps, d, _p(scales), int(bool(post_norm)), _p(pre_w), pre_w_offset, st))
+                                        _p(h), _p(h16), _p(stash), _p(flush_ring), flush_taps, d, _p(scales), int(bool(post_norm)), _p(pre_w), pre_w_offset, _p(post_w), st))
 
     def rmsnorm_rows(self, x_ptr, ldx, w, eps, y_ptr, ldy, T, n, st):
         self._ck(self.lib.sllm_seq_rmsnorm_rows(x_ptr, ldx, _p(w), eps, y_ptr, ldy, T, n, st))
@@ -135,9 +154,10 @@ class Ops:
     def softcap(self, x, n, cap, st):
         self._ck(self.lib.sllm_seq_softcap(_p(x), n, cap, st))
 
-    def moe_act(self, logits_ptr, ldl, n_route, experts, top, correction, up_ptr, ldu, ff, act, h, ldh, d, out, out16, y, ldy, T, st, route_w=None):
+    def moe_act(self, logits_ptr, ldl, n_route, experts, top, correction, up_ptr, ldu, ff, act, h, ldh, d, out, out16, y, ldy, T, st, route_w=None, shared_ptr=None,
+                shared_ff=0):
         self._ck(self.lib.sllm_seq_moe_act(logits_ptr, ldl, n_route, experts, top, _p(correction), up_ptr, ldu, ff, act, _p(h), ldh, d, _p(out), _p(out16),
-                                           _p(y), ldy, _p(route_w), T, st))
+                                           _p(y), ldy, _p(route_w), shared_ptr, shared_ff, T, st))
 
     # ---- mixture of experts with the tokens gathered per expert ----
     def zero(self, ptr, n_bytes, st):
