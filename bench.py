@@ -77,6 +77,11 @@ def parse():
                     help="instead of the headline workload: prefill and decode throughput of the Kodezen design (pre-norm layers behind an input convolution; "
                          "Mamba-2, Mamba and talking-heads window attention; biased gelu and gated experts) beside the closest model (Vasosun) at equal width "
                          "and depth, at the sizes of simplellminference_b200/bench_kodezen.py (w1024,w2048,w4096) or 'all'. One GPU; prints one JSON line {\"kodezen\": [...]}")
+    ap.add_argument("--lovulix", default=None, metavar="SIZES",
+                    help="instead of the headline workload: prefill and decode throughput of the Lovulix design (post-norm layers; chunked attention with scores mixed "
+                         "over the heads before the softmax; gated experts beside a shared one) beside the closest model (Kodezen) at equal width and depth, and "
+                         "the two designs' attention alone, at the sizes of simplellminference_b200/bench_lovulix.py (w1024,w2048,w4096) or 'all'. One GPU; prints "
+                         "one JSON line {\"lovulix\": [...]}")
     ap.add_argument("--no-batch", action="store_true", help="(kept for old command lines: the secondary measurements are opt-in now, see --extras)")
     return ap.parse_args()
 
@@ -652,9 +657,12 @@ def main():
     real_stdout = os.dup(1)
     os.dup2(2, 1)
     sys.stdout = os.fdopen(real_stdout, "w", buffering=1)
-    if args.hybrid or args.sopetar or args.vasosun or args.kodezen:
+    if args.hybrid or args.sopetar or args.vasosun or args.kodezen or args.lovulix:
         import torch
-        if args.kodezen:
+        if args.lovulix:
+            from simplellminference_b200 import bench_lovulix as bench_hybrid
+            key, wanted = "lovulix", args.lovulix
+        elif args.kodezen:
             from simplellminference_b200 import bench_kodezen as bench_hybrid
             key, wanted = "kodezen", args.kodezen
         elif args.hybrid:

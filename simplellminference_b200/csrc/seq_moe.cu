@@ -53,7 +53,7 @@ __global__ void seq_moe_act_kernel(const float* __restrict__ logits, int ldl, in
         for (int e = lane; e < n_route; e += 32) {
             const float s = s_score[e] * inv;
             s_score[e] = s;
-            s_choice[e] = s + (correction ? correction[e] : 0.0f);
+            s_choice[e] = correction ? s + correction[e] : z[e];   // without a correction the order of the scores is the logits' own, which do not saturate
             s_w[e] = 0.0f;
         }
         __syncwarp();
@@ -168,7 +168,7 @@ __global__ void seq_moe_route_kernel(int act, const float* __restrict__ logits, 
         for (int e = lane; e < n_route; e += 32) {
             const float s = s_score[e] * inv;
             s_score[e] = s;
-            s_choice[e] = s + (correction ? correction[e] : 0.0f);
+            s_choice[e] = correction ? s + correction[e] : z[e];   // without a correction the order of the scores is the logits' own, which do not saturate
         }
         __syncwarp();
         float ident = 0.0f;
