@@ -393,7 +393,8 @@ __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __res
                                             int ldo, uint16_t* __restrict__ out16) {
     extern __shared__ float fsm[];
     float* s_w = fsm;            // [nsplit]
-    float* s_o = fsm + nsplit;   // [dv]
+    float* s_o = fsm + nsplit;   // [groups][dv]
+    const int cols = (dv + 31) & ~31, groups = blockDim.x / cols;   // groups of `cols` threads take the shares in turn
     const int t = blockIdx.x / heads, h = blockIdx.x % heads, lane = threadIdx.x & 31;
     const float* rec = ws + ((size_t)t * heads + h) * nsplit * (dv + 2);
     if (threadIdx.x < 32) {
@@ -414,14 +415,19 @@ __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __res
         for (int s = lane; s < nsplit; s += 32) s_w[s] *= inv_den;
     }
     __syncthreads();
-    const int col = threadIdx.x;
+    const int col = threadIdx.x % cols, grp = threadIdx.x / cols;
     if (col < dv) {
         float v = 0.0f;
 #pragma unroll 4
-        for (int s = 0; s < nsplit; ++s) v = fmaf(s_w[s], rec[(size_t)s * (dv + 2) + 2 + col], v);
-        s_o[col] = v;
+        for (int s = grp; s < nsplit; s += groups) v = fmaf(s_w[s], rec[(size_t)s * (dv + 2) + 2 + col], v);
+        s_o[grp * dv + col] = v;
     }
     __syncthreads();
+    if (groups > 1) {
+        if (grp == 0 && col < dv)
+            for (int i = 1; i < groups; ++i) s_o[col] += s_o[i * dv + col];
+        __syncthreads();
+    }
     // one gate per head, or (gate_channels) one per column of the row of heads
     const float gv = gate && !gate_channels ? seq_sigmoid(gate[(size_t)t * ldg + h]) : 1.0f;
     const float* grow = gate && gate_channels ? gate + (size_t)t * ldg + (size_t)h * dv : nullptr;
@@ -431,7 +437,7 @@ __global__ void seq_attention_finish_kernel(sllm_seq_batch b, const float* __res
         if (out16) out16[((size_t)t * heads + h) * dv + c] = f32_to_bf16_bits(v);
     };
     if (!vfreq) {
-        if (col < dv) put(col, s_o[col]);
+        if (grp == 0 && col < dv) put(col, s_o[col]);
         return;
     }
     const int half = dv / 2, mi = threadIdx.x;
@@ -518,8 +524,9 @@ int sllm::launch_attention_finish(const sllm_seq_batch* b, const float* ws, int 
     if (int rc = check_batch(b, "seq_attention_finish")) return rc;
     SLLM_REQUIRE(ws && (out || out16) && nsplit >= 1 && heads > 0 && dv > 0 && (!vfreq || dv % 2 == 0), SLLM_EINVAL, "seq_attention_finish: bad argument");
     SLLM_REQUIRE(dv <= 1024 && nsplit <= 8192, SLLM_ENOTSUP, "seq_attention_finish: value width %d / %d shares beyond what one CTA merges", dv, nsplit);
-    const int threads = std::max(32, (dv + 31) / 32 * 32);
-    seq_attention_finish_kernel<<<b->T * heads, threads, (size_t)(nsplit + dv) * sizeof(float), st>>>(*b, ws, nsplit, heads, dv, vfreq, layout, gate, ldg, gate_channels,
+    // many shares (single tokens): up to eight groups of threads add them side by side, each at least four
+    const int cols = (dv + 31) / 32 * 32, groups = std::max(1, std::min({8, 1024 / cols, nsplit / 4})), threads = cols * groups;
+    seq_attention_finish_kernel<<<b->T * heads, threads, (size_t)(nsplit + groups * dv) * sizeof(float), st>>>(*b, ws, nsplit, heads, dv, vfreq, layout, gate, ldg, gate_channels,
                                                                                                      sink, out, ldo, out16);
     ++g_launches;
     SLLM_LAUNCH_CHECK();

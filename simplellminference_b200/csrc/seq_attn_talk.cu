@@ -47,17 +47,28 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t add
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
-template <int kDvTiles, int kKeys>   // dv <= 8 * kDvTiles (multiple of 8); kKeys keys per tile
-__global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p) {
+// 2^x; tiny results become zero
+__device__ __forceinline__ float fast_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+constexpr int kTalkKeys = 64;   // keys per tile
+
+template <int kDvTiles, int kHeads>   // dv <= 8 * kDvTiles (multiple of 8); kHeads heads (= warps) per CTA
+__global__ void __launch_bounds__(32 * kHeads) seq_attention_talk_mma_kernel(TalkArgs p) {
+    constexpr int kKeys = kTalkKeys, kThreads = 32 * kHeads, qrows = kHeads * kBQ;
     extern __shared__ __align__(128) uint16_t smh[];
     const sllm_seq_batch& b = p.b;
     const int qt = blockIdx.x, split = blockIdx.z;
     const int seg = b.qt_seg[qt], off = b.qt_off[qt];
     const int nq = min(kBQ, b.seg_len[seg] - off), t0 = b.seg_start[seg] + off, pos0 = b.seg_pos0[seg] + off, slot = b.seg_slot[seg];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
-    const int hpc = blockDim.x >> 5, h0 = blockIdx.y * hpc, h = h0 + warp, gv = h0 / (p.heads / p.kv_heads);
+    const int h0 = blockIdx.y * kHeads, h = h0 + warp, gv = h0 / (p.heads / p.kv_heads);
     const int dv = p.dv, dvt = dv / 8, ldv = dv + 8, wide = p.kv_heads * p.dk, pieces = (wide + kTalkCols - 1) / kTalkCols;
-    const int qrows = hpc * kBQ, stage_elems = (qrows + kKeys) * kTalkCols, v_elems = kKeys * ldv, v_bufs = pieces == 1 ? 3 : 2;
+    constexpr int stage_elems = (qrows + kKeys) * kTalkCols;
+    const int v_elems = kKeys * ldv, v_bufs = pieces == 1 ? 3 : 2;
     uint16_t* smv = smh + kTalkStages * stage_elems;
     const uint16_t* kp = reinterpret_cast<const uint16_t*>(p.k_pool);
     const uint16_t* vp = reinterpret_cast<const uint16_t*>(p.v_pool);
@@ -65,38 +76,42 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
     const TileList tiles(pos0, last_pos, seq_row_window(pos0, p.window, p.chunk), p.keep_first, kKeys);
     const int my_tiles = tiles.n > split ? (tiles.n - split + p.nsplit - 1) / p.nsplit : 0, total = my_tiles * pieces;
 
-    // piece `ip` of this CTA's tile number `it` -> stage `st`, asynchronously; rows that do not exist and columns beyond the row are zeros
+    // piece `ip` of this CTA's tile number `it` -> stage `st`, asynchronously; rows that do not exist and columns beyond the row are zeros.
+    // A thread copies the same 16-byte unit of a piece's rows in every pass over them, kRowStep rows apart.
+    constexpr int kRowStep = kThreads / 8;
+    const int my_row = threadIdx.x >> 3, my_unit = threadIdx.x & 7;
     auto issue = [&](int it, int ip, int st) {
-        const int j0 = tiles.tile_of(split + it * p.nsplit) * kKeys, col0 = ip * kTalkCols;
+        const int j0 = tiles.tile_of(split + it * p.nsplit) * kKeys, col = ip * kTalkCols + my_unit * 8;
+        const bool col_ok = col < wide;
         uint16_t* sQ = smh + st * stage_elems;
         uint16_t* sK = sQ + qrows * kTalkCols;
-        for (int i = threadIdx.x; i < qrows * 8; i += blockDim.x) {
-            const int row = i >> 3, unit = i & 7, r = row & (kBQ - 1), col = col0 + unit * 8;
-            const bool take = r < nq && col < wide;
-            const uint16_t* src = p.qm + ((size_t)(t0 + r) * p.heads + h0 + (row >> 5)) * wide + col;
-            cp_async16(sQ + row * kTalkCols + ((unit ^ (row & 7)) << 3), take ? src : p.qm, take ? 16 : 0);
-        }
-        size_t krow[kKeys / 32], vrow[kKeys / 32];      // pages hold a multiple of 32 positions: one look-up per 32 keys
+        const uint16_t* qsrc = p.qm + ((size_t)t0 * p.heads + h0) * wide + col;
 #pragma unroll
-        for (int q = 0; q < kKeys / 32; ++q) {
+        for (int k = 0; k < qrows / kRowStep; ++k) {
+            const int row = my_row + k * kRowStep, r = row & (kBQ - 1), hh = row / kBQ;
+            const bool take = col_ok && r < nq;
+            cp_async16(sQ + row * kTalkCols + ((my_unit ^ (row & 7)) << 3), take ? qsrc + (r * p.heads + hh) * wide : p.qm, take ? 16 : 0);
+        }
+        size_t krow[2], vrow[2];      // pages hold a multiple of 32 positions: one look-up per 32 keys
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
             const int j = j0 + 32 * q;
             const int page = j <= last_pos ? b.block_table[(size_t)slot * b.max_pages + j / b.page_len] : 0, in_page = j % b.page_len;
             krow[q] = ((size_t)page * b.page_len + in_page) * wide;
             vrow[q] = seq_pool_row(page, p.kv_heads, gv, b.page_len, in_page, dv);
         }
-        for (int i = threadIdx.x; i < kKeys * 8; i += blockDim.x) {
-            const int row = i >> 3, unit = i & 7, col = col0 + unit * 8;
-            const bool take = j0 + row <= last_pos && col < wide;
-            const uint16_t* src = kp + (row < 32 ? krow[0] : krow[kKeys / 32 - 1]) + (size_t)(row & 31) * wide + col;
-            cp_async16(sK + row * kTalkCols + ((unit ^ (row & 7)) << 3), take ? src : kp, take ? 16 : 0);
+#pragma unroll
+        for (int k = 0; k < kKeys / kRowStep; ++k) {
+            const int row = my_row + k * kRowStep;
+            const bool take = col_ok && j0 + row <= last_pos;
+            cp_async16(sK + row * kTalkCols + ((my_unit ^ (row & 7)) << 3), take ? kp + (k * kRowStep >= 32 ? krow[1] : krow[0]) + (row & 31) * wide + col : kp, take ? 16 : 0);
         }
         if (ip == 0) {
             uint16_t* sV = smv + (it % v_bufs) * v_elems;
-            for (int i = threadIdx.x; i < kKeys * dvt; i += blockDim.x) {
+            for (int i = threadIdx.x; i < kKeys * dvt; i += kThreads) {
                 const int row = i / dvt, cc = (i % dvt) * 8;
                 const bool take = j0 + row <= last_pos;
-                const uint16_t* src = vp + (row < 32 ? vrow[0] : vrow[kKeys / 32 - 1]) + (size_t)(row & 31) * dv + cc;
-                cp_async16(sV + row * ldv + cc, take ? src : vp, take ? 16 : 0);
+                cp_async16(sV + row * ldv + cc, take ? vp + (row < 32 ? vrow[0] : vrow[1]) + (row & 31) * dv + cc : vp, take ? 16 : 0);
             }
         }
     };
@@ -116,7 +131,6 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
 #pragma unroll
     for (int i = 0; i < kTalkStages - 1; ++i) issue_next();
 
-    const bool two = nq > 16;   // a second block of 16 queries?
     int rpos[4], rwnd[4];       // the thread's rows: (block, half) -> 2 * block + half
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -136,7 +150,7 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
 #pragma unroll
         for (int nt = 0; nt < kKeys / 8; ++nt) s[mt][nt][0] = s[mt][nt][1] = s[mt][nt][2] = s[mt][nt][3] = 0.0f;
     }
-    constexpr float kLog2e = 1.4426950408889634f;
+    const float scale2 = p.scale * 1.4426950408889634f;    // the running softmax works in powers of two
     int st = 0;
     for (int it = 0; it < my_tiles; ++it) {
         for (int ip = 0; ip < pieces; ++ip) {
@@ -145,14 +159,12 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
             issue_next();
             const uint32_t aQ = smem_u32(smh + st * stage_elems + warp * kBQ * kTalkCols), aK = smem_u32(smh + st * stage_elems + qrows * kTalkCols);
             st = st + 1 == kTalkStages ? 0 : st + 1;
-            const int ksteps = min(kTalkCols, wide - ip * kTalkCols + 15) / 16;
 #pragma unroll
-            for (int ks = 0; ks < kTalkCols / 16; ++ks) {
-                if (ks >= ksteps) break;
+            for (int ks = 0; ks < kTalkCols / 16; ++ks) {       // columns beyond the row are zeros in both operands
                 uint32_t a0[4], a1[4];
                 const uint32_t arow = (uint32_t)(lane & 15) * (kTalkCols * 2) + (uint32_t)(((2 * ks + (lane >> 4)) ^ (lane & 7)) << 4);
                 ldmatrix_x4(a0, aQ + arow);
-                if (two) ldmatrix_x4(a1, aQ + 16 * kTalkCols * 2 + arow);
+                ldmatrix_x4(a1, aQ + 16 * kTalkCols * 2 + arow);
 #pragma unroll
                 for (int np = 0; np < kKeys / 16; ++np) {
                     uint32_t bb[4];
@@ -160,10 +172,8 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
                     ldmatrix_x4(bb, aK + (uint32_t)row * (kTalkCols * 2) + (uint32_t)(((2 * ks + ((lane >> 3) & 1)) ^ (lane & 7)) << 4));
                     mma_bf16_16816(s[0][2 * np], a0, bb[0], bb[1]);
                     mma_bf16_16816(s[0][2 * np + 1], a0, bb[2], bb[3]);
-                    if (two) {
-                        mma_bf16_16816(s[1][2 * np], a1, bb[0], bb[1]);
-                        mma_bf16_16816(s[1][2 * np + 1], a1, bb[2], bb[3]);
-                    }
+                    mma_bf16_16816(s[1][2 * np], a1, bb[0], bb[1]);
+                    mma_bf16_16816(s[1][2 * np + 1], a1, bb[2], bb[3]);
                 }
             }
         }
@@ -174,14 +184,13 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
         const bool inside = nq == kBQ && j0 + kKeys - 1 <= pos0 && last_pos - j0 < seq_row_window(last_pos, p.window, p.chunk);
 #pragma unroll
         for (int mt = 0; mt < 2; ++mt) {
-            if (mt == 1 && !two) break;
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int nt = 0; nt < kKeys / 8; ++nt) {
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int i = 2 * mt + (e >> 1), key = j0 + nt * 8 + 2 * c + (e & 1);
-                    const float sc = s[mt][nt][e] * p.scale;
+                    const float sc = s[mt][nt][e] * scale2;
                     s[mt][nt][e] = inside || seq_sees(rpos[i], key, rwnd[i], p.keep_first) ? sc : -INFINITY;
                     mx[e >> 1] = fmaxf(mx[e >> 1], s[mt][nt][e]);
                 }
@@ -192,14 +201,15 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
                 mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 1));
                 mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 2));
                 const float mn = fmaxf(m[i], mx[hf]);
-                const float corr = mn == -INFINITY ? 1.0f : exp2f((m[i] - mn) * kLog2e);
+                const float ref = mn == -INFINITY ? 0.0f : mn;        // no key seen yet: every weight below is 2^-inf = 0
+                const float corr = fast_exp2(m[i] - ref);
                 m[i] = mn;
                 float sum = 0.0f;
 #pragma unroll
                 for (int nt = 0; nt < kKeys / 8; ++nt) {
 #pragma unroll
                     for (int e = 2 * hf; e < 2 * hf + 2; ++e) {
-                        s[mt][nt][e] = s[mt][nt][e] == -INFINITY ? 0.0f : exp2f((s[mt][nt][e] - mn) * kLog2e);
+                        s[mt][nt][e] = fast_exp2(s[mt][nt][e] - ref);
                         sum += s[mt][nt][e];
                     }
                 }
@@ -230,16 +240,12 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
                     ldmatrix_x4_trans(bb, vrow + nt * 16);
                     mma_bf16_16816(o[0][nt], ah[0], bb[0], bb[1]);
                     mma_bf16_16816(o[0][nt + 1], ah[0], bb[2], bb[3]);
-                    if (two) {
-                        mma_bf16_16816(o[1][nt], ah[1], bb[0], bb[1]);
-                        mma_bf16_16816(o[1][nt + 1], ah[1], bb[2], bb[3]);
-                    }
+                    mma_bf16_16816(o[1][nt], ah[1], bb[0], bb[1]);
+                    mma_bf16_16816(o[1][nt + 1], ah[1], bb[2], bb[3]);
                     mma_bf16_16816(o[0][nt], al[0], bb[0], bb[1]);
                     mma_bf16_16816(o[0][nt + 1], al[0], bb[2], bb[3]);
-                    if (two) {
-                        mma_bf16_16816(o[1][nt], al[1], bb[0], bb[1]);
-                        mma_bf16_16816(o[1][nt + 1], al[1], bb[2], bb[3]);
-                    }
+                    mma_bf16_16816(o[1][nt], al[1], bb[0], bb[1]);
+                    mma_bf16_16816(o[1][nt + 1], al[1], bb[2], bb[3]);
                 }
             }
         }
@@ -256,6 +262,7 @@ __global__ void __launch_bounds__(128) seq_attention_talk_mma_kernel(TalkArgs p)
         l[i] += __shfl_xor_sync(0xffffffffu, l[i], 2);
         const int r = (i >> 1) * 16 + (i & 1) * 8 + g, t = t0 + r;
         if (r >= nq) continue;
+        m[i] *= 0.6931471805599453f;           // back to natural units (a share that saw no key stays at -inf)
         if (p.nsplit > 1) {
             float* rec = p.ws + (((size_t)t * p.heads + h) * p.nsplit + split) * (dv + 2);
             if (c == 0) {
@@ -535,16 +542,19 @@ int sllm_seq_attention_talk(const sllm_seq_batch* b, const float* q, int32_t ldq
         SLLM_REQUIRE(sllm_seq_attention_talk_takes_mixed(heads, kv_heads, dk, dv, kv_dtype), SLLM_ENOTSUP, "seq_attention_talk: mixed queries for heads of %d + %d", dk, dv);
         SLLM_REQUIRE(nsplit == 1 || ws, SLLM_EINVAL, "seq_attention_talk: %d shares need a workspace", nsplit);
         const int group = heads / kv_heads, hpc = group % 4 == 0 ? 4 : (group % 2 == 0 ? 2 : 1), pieces = (kv_heads * dk + kTalkCols - 1) / kTalkCols;
-        const dim3 grid(b->n_qtiles, heads / hpc, nsplit), block(32 * hpc);
-        constexpr int kKeys = 64;
-        const size_t smem = (kTalkStages * (size_t)(hpc * kBQ + kKeys) * kTalkCols + (size_t)(pieces == 1 ? 3 : 2) * kKeys * (dv + 8)) * sizeof(uint16_t);
+        const dim3 grid(b->n_qtiles, heads / hpc, nsplit);
+        const size_t smem = (kTalkStages * (size_t)(hpc * kBQ + kTalkKeys) * kTalkCols + (size_t)(pieces == 1 ? 3 : 2) * kTalkKeys * (dv + 8)) * sizeof(uint16_t);
+#define SLLM_TALK_LAUNCH(DV, HEADS)                                                                                                                    \
+    do {                                                                                                                                               \
+        SLLM_CUDA(cudaFuncSetAttribute(seq_attention_talk_mma_kernel<DV, HEADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));             \
+        seq_attention_talk_mma_kernel<DV, HEADS><<<grid, 32 * HEADS, smem, st>>>(p);                                                                   \
+    } while (0)
         if (dv <= 64) {
-            SLLM_CUDA(cudaFuncSetAttribute(seq_attention_talk_mma_kernel<8, kKeys>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            seq_attention_talk_mma_kernel<8, kKeys><<<grid, block, smem, st>>>(p);
+            if (hpc == 4) SLLM_TALK_LAUNCH(8, 4); else if (hpc == 2) SLLM_TALK_LAUNCH(8, 2); else SLLM_TALK_LAUNCH(8, 1);
         } else {
-            SLLM_CUDA(cudaFuncSetAttribute(seq_attention_talk_mma_kernel<16, kKeys>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-            seq_attention_talk_mma_kernel<16, kKeys><<<grid, block, smem, st>>>(p);
+            if (hpc == 4) SLLM_TALK_LAUNCH(16, 4); else if (hpc == 2) SLLM_TALK_LAUNCH(16, 2); else SLLM_TALK_LAUNCH(16, 1);
         }
+#undef SLLM_TALK_LAUNCH
         ++g_launches;
         SLLM_LAUNCH_CHECK();
         if (nsplit == 1) return SLLM_OK;

@@ -351,6 +351,20 @@ __global__ void seq_gated_act_kernel(const float* __restrict__ gate, int ldg, co
     }
 }
 
+// the same four columns at a time: grid (T, parts of a row), 16-byte loads
+__global__ void seq_gated_act_vec_kernel(const float* __restrict__ gate, int ldg, const float* __restrict__ up, int ldu, float* __restrict__ out, int ldo,
+                                         uint16_t* __restrict__ out16, int n) {
+    const size_t t = blockIdx.x;
+    for (int j = (blockIdx.y * blockDim.x + threadIdx.x) * 4; j < n; j += gridDim.y * blockDim.x * 4) {
+        const float4 g = *reinterpret_cast<const float4*>(gate + t * ldg + j), u = *reinterpret_cast<const float4*>(up + t * ldu + j);
+        const float4 v = make_float4(g.x * seq_sigmoid(g.x) * u.x, g.y * seq_sigmoid(g.y) * u.y, g.z * seq_sigmoid(g.z) * u.z, g.w * seq_sigmoid(g.w) * u.w);
+        if (out) *reinterpret_cast<float4*>(out + t * ldo + j) = v;
+        if (out16)
+            *reinterpret_cast<uint2*>(out16 + t * n + j) = make_uint2((uint32_t)f32_to_bf16_bits(v.x) | ((uint32_t)f32_to_bf16_bits(v.y) << 16),
+                                                                     (uint32_t)f32_to_bf16_bits(v.z) | ((uint32_t)f32_to_bf16_bits(v.w) << 16));
+    }
+}
+
 // x <- cap * tanh(x / cap)
 __global__ void seq_softcap_kernel(float* __restrict__ x, size_t n, float cap) {
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] = cap * tanhf(x[i] / cap);
@@ -507,6 +521,14 @@ int sllm_seq_gated_act(const float* gate, int32_t ldg, const float* up, int32_t 
                        sllm_stream_t stream) {
     SLLM_REQUIRE(gate && up && (out || out16) && T > 0 && n > 0 && ldg >= n && ldu >= n && (!out || ldo >= n), SLLM_EINVAL, "seq_gated_act: bad argument");
     SLLM_REQUIRE(act == 0, SLLM_ENOTSUP, "seq_gated_act: activation 0 (silu)");
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    if (n % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && (!out || ldo % 4 == 0) && aligned(gate) && aligned(up) && aligned(out) && aligned(out16)) {
+        const int parts = std::min(64, (n / 4 + 255) / 256);
+        seq_gated_act_vec_kernel<<<dim3(T, parts), n >= 1024 ? 256 : 64, 0, as_stream(stream)>>>(gate, ldg, up, ldu, out, ldo, (uint16_t*)out16, n);
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     const size_t total = (size_t)T * n;
     seq_gated_act_kernel<<<(int)std::min<size_t>((total + 255) / 256, (size_t)sm_count() * 8), 256, 0, as_stream(stream)>>>(gate, ldg, up, ldu, act, out, ldo,
                                                                                                                      (uint16_t*)out16, T, n);

@@ -237,6 +237,17 @@ __global__ void seq_moe_expert_act_kernel(const float* __restrict__ up, const in
     if (r >= counts[e]) return;
     const size_t row = ((size_t)e * cap + r) * ff;
     const bool gated = act & kMoeGated;                  // rows of `up` then hold [gate ff | up ff]
+    if (gated && ff % 4 == 0) {                          // four columns at a time
+        for (int j = 4 * threadIdx.x; j < ff; j += 4 * blockDim.x) {
+            const float4 g = *reinterpret_cast<const float4*>(up + 2 * row + j), u = *reinterpret_cast<const float4*>(up + 2 * row + ff + j);
+            const float4 v = make_float4(moe_act(g.x, act) * u.x, moe_act(g.y, act) * u.y, moe_act(g.z, act) * u.z, moe_act(g.w, act) * u.w);
+            if (out16)
+                *reinterpret_cast<uint2*>(out16 + row + j) = make_uint2((uint32_t)f32_to_bf16_bits(v.x) | ((uint32_t)f32_to_bf16_bits(v.y) << 16),
+                                                                       (uint32_t)f32_to_bf16_bits(v.z) | ((uint32_t)f32_to_bf16_bits(v.w) << 16));
+            if (out32) *reinterpret_cast<float4*>(out32 + row + j) = v;
+        }
+        return;
+    }
     for (int j = threadIdx.x; j < ff; j += blockDim.x) {
         const float v = gated ? moe_act(up[2 * row + j], act) * up[2 * row + ff + j] : moe_act(up[row + j], act);
         if (out16) out16[row + j] = f32_to_bf16_bits(v);
@@ -244,8 +255,8 @@ __global__ void seq_moe_expert_act_kernel(const float* __restrict__ up, const in
     }
 }
 
-// one CTA per (token, choice) pair, rows in the pairs' own order: out = act(s * up) or act(s * gate) * (s * up), with s the pair's score when
-// the score multiplies what the expert reads (the products are linear: the score is applied to their results) and 1 otherwise;
+// grid (pairs, parts of a row), rows in the (token, choice) pairs' own order: out = act(s * up) or act(s * gate) * (s * up), with s the pair's
+// score when the score multiplies what the expert reads (the products are linear: the score is applied to their results) and 1 otherwise;
 // w_out takes what the combine kernel has to multiply the pair's down row by: 1 in the first case, the score in the second
 __global__ void seq_moe_pair_act_kernel(const float* __restrict__ up, const float* __restrict__ sel_w, int ff, int act, float* __restrict__ out,
                                         float* __restrict__ w_out) {
@@ -253,9 +264,9 @@ __global__ void seq_moe_pair_act_kernel(const float* __restrict__ up, const floa
     const bool gated = act & kMoeGated, on_input = act & kMoeScaleInput;
     const float score = sel_w[p], s = on_input ? score : 1.0f;
     const float* row = up + (size_t)p * ff * (gated ? 2 : 1);
-    for (int j = threadIdx.x; j < ff; j += blockDim.x)
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < ff; j += gridDim.y * blockDim.x)
         out[(size_t)p * ff + j] = gated ? moe_act(s * row[j], act) * (s * row[ff + j]) : moe_act(s * row[j], act);
-    if (threadIdx.x == 0) w_out[p] = on_input ? 1.0f : score;
+    if (threadIdx.x == 0 && blockIdx.y == 0) w_out[p] = on_input ? 1.0f : score;
 }
 
 __global__ void seq_moe_combine_kernel(const float* __restrict__ down, const int32_t* __restrict__ sel_e, const int32_t* __restrict__ sel_pos,
@@ -326,7 +337,7 @@ int sllm_seq_moe_expert_act(const float* up, const int32_t* counts, int32_t expe
 
 int sllm_seq_moe_pair_act(const float* up, const float* sel_w, int32_t pairs, int32_t ff, int32_t act, float* out, float* w_out, sllm_stream_t stream) {
     SLLM_REQUIRE(up && sel_w && out && w_out && pairs > 0 && ff > 0 && act >= 0 && (act & 3) <= 2 && act < 32, SLLM_EINVAL, "seq_moe_pair_act: bad argument");
-    seq_moe_pair_act_kernel<<<pairs, 256, 0, as_stream(stream)>>>(up, sel_w, ff, act, out, w_out);
+    seq_moe_pair_act_kernel<<<dim3(pairs, std::min(64, (ff + 255) / 256)), 256, 0, as_stream(stream)>>>(up, sel_w, ff, act, out, w_out);
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     return SLLM_OK;

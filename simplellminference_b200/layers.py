@@ -604,7 +604,8 @@ class ScoreMixingAttention:
         if step.T == step.nseg:
             return max(1, min(tiles, step.sms // step.nseg))
         ctas = step.b.n_qtiles * (c.heads // math.gcd(c.heads // c.kv_heads, 4)) if mixed else -(-step.T // 4)
-        return max(1, min(tiles, 2 * step.sms // ctas))
+        # (a work item's keys number anything from one to a whole chunk: several CTAs' worth per SM even that out)
+        return max(1, min(tiles, (4 if mixed else 2) * step.sms // ctas))
 
     def forward(self, step, cols, ld, state, out):
         c, ops, T = self.cfg, self.ops, step.T
