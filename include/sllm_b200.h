@@ -585,14 +585,16 @@ int sllm_seq_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, in
                               int32_t kv_heads, const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps,
                               const double* freq, int32_t n_freq, int32_t layout, void* k_pool, void* v_pool, int32_t kv_dtype,
                               sllm_stream_t stream);
-/* The same preparation for mixers whose queries and keys are RMS-normed over the WHOLE projection (all heads of a token at once; weights
+/* out [T][n_freq] (cos, sin) of pos * freq[i] for every token, the angle formed in double: once per step for all layers that turn alike */
+int sllm_seq_angles(const sllm_seq_batch* b, const double* freq, int32_t n_freq, float* out, sllm_stream_t stream);
+/* The same preparation (angles = the table of sllm_seq_angles) for mixers whose queries and keys are RMS-normed over the WHOLE projection (all heads of a token at once; weights
  * q_norm_w [heads * dk] / k_norm_w [kv_heads * dk], NULL = not normed) before they are split into heads and turned. v: share 1 keeps the
  * values in v_shared [T][kv_heads * dv], share 2 stores (1 - lambda) v + lambda v_shared. k_joint: the pool holds the heads of a token side by
  * side ([pages][1][page_len][kv_heads * dk]) instead of head by head. q_mixed (or NULL; then talk [heads][heads] is not read): the queries
  * mixed for sllm_seq_attention_talk go there as bf16 and q stays as it is; otherwise q is normed and turned in place. */
 int sllm_seq_wide_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk,
                                    int32_t kv_heads, const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps,
-                                   const double* freq, int32_t n_freq, int32_t layout, float* v_shared, int32_t share, float lambda,
+                                   const float* angles, int32_t n_freq, int32_t layout, float* v_shared, int32_t share, float lambda,
                                    const float* talk, void* q_mixed, int32_t k_joint, void* k_pool, void* v_pool, int32_t kv_dtype,
                                    sllm_stream_t stream);
 /* Heads mixed after the attention: in [T][kv_heads * heads * dv] as sllm_seq_attention_finish leaves it for cross_values (record = value

@@ -151,6 +151,7 @@ SIGNATURES.update({
     "sllm_seq_attention_finish": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _I, _P, _P]),
     "sllm_seq_attention_talk": (C.c_int, [_B, _P, _I, _P, _I, _I, _I, _I, _F, _P, _P, _P, _I, _I, _P, C.POINTER(SeqAttnOpts), _P, _I, _P, _P, _I, _P, _P]),
     "sllm_seq_attention_talk_takes_mixed": (C.c_int, [_I, _I, _I, _I, _I]),
+    "sllm_seq_angles": (C.c_int, [_B, _P, _I, _P, _P]),
     "sllm_seq_wide_normed_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _P, _F, _P, _I, _I, _P, _I, _F, _P, _P, _I, _P, _P, _I, _P]),
     "sllm_seq_unit_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _F, _I, _P, _I, _F, _P, _P, _I, _F, _I, _P]),
     "sllm_seq_latent_kv": (C.c_int, [_B, _P, _I, _I, _I, _I, _P, _I, _I, _P, _F, _P, _I, _P, _I, _P, _I, _F, _P]),

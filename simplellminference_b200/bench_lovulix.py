@@ -124,6 +124,7 @@ def _attention_alone(T: int, width: int, mixes_first: bool, context: int = 0):
             c = cols[:step.T] if step.T > 1 else cols[-1:]
 
             def call():
+                step.turned.clear()
                 step.st = torch.cuda.current_stream(dev).cuda_stream
                 mech.forward(step, [c.data_ptr() + 4 * o for o in offs[:len(mech.inputs)]], n, states[0], step.scratch("mix_part", step.T * mech.width))
             self.call = call

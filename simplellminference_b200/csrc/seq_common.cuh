@@ -29,6 +29,12 @@ __device__ __forceinline__ void seq_ld16(const uint16_t* p, bool take, float (&o
 }
 __device__ __forceinline__ void seq_st(float* p, size_t i, float v) { p[i] = v; }
 __device__ __forceinline__ void seq_st(uint16_t* p, size_t i, float v) { p[i] = f32_to_bf16_bits(v); }
+// two floats rounded to bf16 (nearest even) in one register, `lo` in the low half
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+    uint32_t r;
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(hi), "f"(lo));
+    return r;
+}
 // nearest-even rounding to bf16 and back: one cvt instruction + one shift (the same values as f32_to_bf16_bits for finite inputs)
 __device__ __forceinline__ float seq_round_bf16(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 

@@ -8,7 +8,8 @@
 // (4) sllm_seq_head_mix — after the attention: the heads' results mixed by a heads x heads matrix;
 // (5) sllm_seq_wide_normed_rotary_kv — queries and keys RMS-normed over the whole projection (all heads of a token at once), then rotated;
 // values optionally blended as in (1); the keys of a token's heads may be stored side by side, and the queries may leave as the mixed
-// bf16 operand rows of attention whose scores are mixed over the heads before the softmax.
+// bf16 operand rows of attention whose scores are mixed over the heads before the softmax;
+// (6) sllm_seq_angles — cos and sin of every token's position times every frequency, once per step for all layers that turn alike.
 // All arithmetic is fp32 (angles in double); the pools hold fp32 or bf16.
 #include "seq_common.cuh"
 
@@ -160,53 +161,104 @@ __global__ void seq_normed_rotary_kv_kernel(sllm_seq_batch b, float* __restrict_
     for (int j = 2 * n_freq + lane; j < dk; j += 32) put(j, s_row[j] * inv * (w ? w[j] : 1.0f));
 }
 
+// four consecutive elements of a pool
+__device__ __forceinline__ void seq_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void seq_st4(uint16_t* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+
+// thread = (token, frequency)
+__global__ void seq_angles_kernel(sllm_seq_batch b, const double* __restrict__ freq, int n_freq, float2* __restrict__ out) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= b.T * n_freq) return;
+    float sn, cs;
+    seq_angle(b.tok_pos[i / n_freq], freq[i % n_freq], &sn, &cs);
+    out[i] = make_float2(cs, sn);
+}
+
 // grid (T, 2): CTA y = 0 takes a token's queries, CTA y = 1 its keys and values. The whole row sits in shared memory (its root mean square
-// is over all heads); a token's angles are the same for every head, so each is formed once.
+// is over all heads); the token's angles come from the step's table.
 constexpr int kMixGroup = 8;   // query heads of a key head whose values a thread holds at once while it mixes
 
 template <typename KV>
 __global__ void __launch_bounds__(256) seq_wide_normed_rotary_kv_kernel(sllm_seq_batch b, float* __restrict__ q, int ldq, int heads, int dk, const float* __restrict__ k,
                                                                         int ldk, int kv_heads, const float* __restrict__ v, int ldv, int dv, const float* __restrict__ q_w,
-                                                                        const float* __restrict__ k_w, float eps, const double* __restrict__ freq, int n_freq, int layout,
+                                                                        const float* __restrict__ k_w, float eps, const float2* __restrict__ angles, int n_freq, int layout,
                                                                         float* __restrict__ v_shared, int share, float lambda, const float* __restrict__ talk,
-                                                                        uint16_t* __restrict__ q_mixed, int k_joint, KV* __restrict__ k_pool, KV* __restrict__ v_pool) {
-    extern __shared__ __align__(16) float wr_sm[];       // the row, cos [n_freq], sin [n_freq], and for the mix talk transposed [heads][heads]
+                                                                        uint16_t* __restrict__ q_mixed, int k_joint, KV* __restrict__ k_pool, KV* __restrict__ v_pool,
+                                                                        int vec) {
+    extern __shared__ __align__(16) float wr_sm[];       // the row, and for the mix talk [heads][heads]
     __shared__ float red[33];
     const int t = blockIdx.x, pos = b.tok_pos[t], slot = b.tok_slot[t];
     const bool is_q = blockIdx.y == 0;
     const int n_heads = is_q ? heads : kv_heads, n = n_heads * dk, group = heads / kv_heads;
     float* s_row = wr_sm;
-    float* s_cos = wr_sm + ((max(heads, kv_heads) * dk + 3) & ~3);
-    float* s_sin = s_cos + n_freq;
-    float* s_talk = s_cos + ((2 * n_freq + 3) & ~3);
+    float* s_talk = wr_sm + ((heads * dk + 3) & ~3);
+    const float2* turn = angles + (size_t)t * n_freq;
     float* row = is_q ? q + (size_t)t * ldq : nullptr;
     const float* src = is_q ? row : k + (size_t)t * ldk;
     const float* w = is_q ? q_w : k_w;
-    for (int i = threadIdx.x; i < n_freq; i += blockDim.x) seq_angle(pos, freq[i], s_sin + i, s_cos + i);
     if (is_q && q_mixed)
         for (int i = threadIdx.x; i < heads * heads; i += blockDim.x) s_talk[i] = talk[i];
     float ss = 0.0f;
-    for (int j = threadIdx.x; j < n; j += blockDim.x) {
-        const float x = src[j];
-        s_row[j] = x;
-        ss = fmaf(x, x, ss);
+    if (vec) {                                           // four columns at a time, every thread its own columns in both passes
+#pragma unroll 4
+        for (int j = 4 * threadIdx.x; j < n; j += 4 * blockDim.x) {
+            const float4 x = *reinterpret_cast<const float4*>(src + j);
+            *reinterpret_cast<float4*>(s_row + j) = x;
+            ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss))));
+        }
+    } else {
+        for (int j = threadIdx.x; j < n; j += blockDim.x) {
+            const float x = src[j];
+            s_row[j] = x;
+            ss = fmaf(x, x, ss);
+        }
     }
     ss = block_sum(ss, red);
     if (w) {
         const float inv = 1.0f / sqrtf(ss / (float)n + eps);
-        for (int j = threadIdx.x; j < n; j += blockDim.x) s_row[j] = (s_row[j] * inv) * w[j];      // every thread its own elements
+        if (vec) {
+#pragma unroll 4
+            for (int j = 4 * threadIdx.x; j < n; j += 4 * blockDim.x) {
+                const float4 x = *reinterpret_cast<const float4*>(s_row + j), g = *reinterpret_cast<const float4*>(w + j);
+                *reinterpret_cast<float4*>(s_row + j) = make_float4((x.x * inv) * g.x, (x.y * inv) * g.y, (x.z * inv) * g.z, (x.w * inv) * g.w);
+            }
+        } else {
+            for (int j = threadIdx.x; j < n; j += blockDim.x) s_row[j] = (s_row[j] * inv) * w[j];
+        }
         __syncthreads();
     }
     for (int i = threadIdx.x; i < n_heads * n_freq; i += blockDim.x) {
         const int h = i / n_freq, mi = i % n_freq;
         const int ia = h * dk + (layout == 0 ? 2 * mi : mi), ib = h * dk + (layout == 0 ? 2 * mi + 1 : mi + n_freq);
-        const float u = s_row[ia], x = s_row[ib], cs = s_cos[mi], sn = s_sin[mi];
-        s_row[ia] = u * cs - x * sn;
-        s_row[ib] = x * cs + u * sn;
+        const float2 a = turn[mi];
+        const float u = s_row[ia], x = s_row[ib];
+        s_row[ia] = u * a.x - x * a.y;
+        s_row[ib] = x * a.x + u * a.y;
     }
     __syncthreads();
     if (!is_q) {
         const int page = b.block_table[(size_t)slot * b.max_pages + pos / b.page_len], in_page = pos % b.page_len;
+        if (vec) {
+            for (int j = 4 * threadIdx.x; j < n; j += 4 * blockDim.x) {
+                const size_t dst = k_joint ? ((size_t)page * b.page_len + in_page) * n + j : seq_pool_row(page, kv_heads, j / dk, b.page_len, in_page, dk) + j % dk;
+                seq_st4(k_pool + dst, *reinterpret_cast<const float4*>(s_row + j));
+            }
+            for (int j = 4 * threadIdx.x; j < kv_heads * dv; j += 4 * blockDim.x) {
+                float4 val = *reinterpret_cast<const float4*>(v + (size_t)t * ldv + j);
+                float4* sh = share ? reinterpret_cast<float4*>(v_shared + (size_t)t * kv_heads * dv + j) : nullptr;
+                if (share == 1) {
+                    *sh = val;
+                } else if (share == 2) {
+                    const float4 first = *sh;
+                    const float mine = 1.0f - lambda;
+                    val = make_float4(mine * val.x + lambda * first.x, mine * val.y + lambda * first.y, mine * val.z + lambda * first.z, mine * val.w + lambda * first.w);
+                }
+                seq_st4(v_pool + seq_pool_row(page, kv_heads, j / dv, b.page_len, in_page, dv) + j % dv, val);
+            }
+            return;
+        }
         if (k_joint) {
             const size_t dst = ((size_t)page * b.page_len + in_page) * n;
             for (int j = threadIdx.x; j < n; j += blockDim.x) seq_st(k_pool, dst + j, s_row[j]);
@@ -238,18 +290,28 @@ __global__ void __launch_bounds__(256) seq_wide_normed_rotary_kv_kernel(sllm_seq
                 if (g < group) x[g] = *reinterpret_cast<const float4*>(s_row + (size_t)(u * group + g) * dk + c);
             for (int h = i / quads; h < heads; h += lanes) {
                 float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                const float* tr = s_talk + h * heads + u * group;
+                __align__(16) float tws[kMixGroup];
+                if (group % 4 == 0) {                    // (then heads is a multiple of four, and so is the row's start)
+#pragma unroll
+                    for (int g = 0; g < kMixGroup; g += 4)
+                        if (g < group) *reinterpret_cast<float4*>(tws + g) = *reinterpret_cast<const float4*>(tr + g);
+                } else {
+#pragma unroll
+                    for (int g = 0; g < kMixGroup; ++g)
+                        if (g < group) tws[g] = tr[g];
+                }
 #pragma unroll
                 for (int g = 0; g < kMixGroup; ++g) {
                     if (g < group) {
-                        const float tw = s_talk[h * heads + u * group + g];
+                        const float tw = tws[g];
                         acc.x = fmaf(tw, x[g].x, acc.x);
                         acc.y = fmaf(tw, x[g].y, acc.y);
                         acc.z = fmaf(tw, x[g].z, acc.z);
                         acc.w = fmaf(tw, x[g].w, acc.w);
                     }
                 }
-                *reinterpret_cast<uint2*>(out + (size_t)h * wide + 4 * qd) = make_uint2((uint32_t)f32_to_bf16_bits(acc.x) | ((uint32_t)f32_to_bf16_bits(acc.y) << 16),
-                                                                                       (uint32_t)f32_to_bf16_bits(acc.z) | ((uint32_t)f32_to_bf16_bits(acc.w) << 16));
+                seq_st4(out + (size_t)h * wide + 4 * qd, acc);
             }
         }
         return;
@@ -347,27 +409,38 @@ int sllm_seq_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, in
     return SLLM_OK;
 }
 
+int sllm_seq_angles(const sllm_seq_batch* b, const double* freq, int32_t n_freq, float* out, sllm_stream_t stream) {
+    SLLM_REQUIRE(b && b->T > 0 && b->tok_pos && freq && out && n_freq > 0 && (uintptr_t)out % 8 == 0, SLLM_EINVAL, "seq_angles: bad argument");
+    seq_angles_kernel<<<(b->T * n_freq + 127) / 128, 128, 0, as_stream(stream)>>>(*b, freq, n_freq, (float2*)out);
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    return SLLM_OK;
+}
+
 int sllm_seq_wide_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk, int32_t kv_heads,
-                                   const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps, const double* freq,
+                                   const float* v, int32_t ldv, int32_t dv, const float* q_norm_w, const float* k_norm_w, float eps, const float* angles,
                                    int32_t n_freq, int32_t layout, float* v_shared, int32_t share, float lambda, const float* talk, void* q_mixed,
                                    int32_t k_joint, void* k_pool, void* v_pool, int32_t kv_dtype, sllm_stream_t stream) {
     SLLM_REQUIRE(b && b->T > 0 && b->tok_slot && b->tok_pos && b->block_table, SLLM_EINVAL, "seq_wide_normed_rotary_kv: incomplete batch description");
     SLLM_REQUIRE(q && k && v && k_pool && v_pool && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0, SLLM_EINVAL,
                  "seq_wide_normed_rotary_kv: bad argument");
-    SLLM_REQUIRE(n_freq >= 0 && 2 * n_freq <= dk && (n_freq == 0 || freq), SLLM_EINVAL, "seq_wide_normed_rotary_kv: %d rotary pairs do not fit %d dimensions", n_freq, dk);
+    SLLM_REQUIRE(n_freq >= 0 && 2 * n_freq <= dk && (n_freq == 0 || angles), SLLM_EINVAL, "seq_wide_normed_rotary_kv: %d rotary pairs do not fit %d dimensions", n_freq, dk);
     SLLM_REQUIRE(layout == 0 || layout == 1, SLLM_EINVAL, "seq_wide_normed_rotary_kv: layout 0 (interleaved) or 1 (halves)");
     SLLM_REQUIRE(share >= 0 && share <= 2 && (share == 0 || v_shared), SLLM_EINVAL, "seq_wide_normed_rotary_kv: share 0 (none), 1 (write) or 2 (blend) with a buffer");
     SLLM_REQUIRE(!q_mixed || (talk && (uintptr_t)q_mixed % 16 == 0), SLLM_EINVAL, "seq_wide_normed_rotary_kv: mixed queries need the mixing matrix and an aligned buffer");
     SLLM_REQUIRE(kv_dtype == SLLM_F32 || kv_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_wide_normed_rotary_kv: fp32 or bf16 pools");
-    const size_t smem = ((((size_t)heads * dk + 3) & ~(size_t)3) + ((2 * (size_t)n_freq + 3) & ~(size_t)3) + (q_mixed ? (size_t)heads * heads : 0)) * sizeof(float);
+    const size_t smem = ((((size_t)heads * dk + 3) & ~(size_t)3) + (q_mixed ? (size_t)heads * heads : 0)) * sizeof(float);
     SLLM_REQUIRE(smem <= (size_t)smem_optin_bytes() - 1024, SLLM_ENOTSUP, "seq_wide_normed_rotary_kv: %d heads of %d do not fit shared memory", heads, dk);
+    auto aligned = [](const void* x) { return x == nullptr || ((uintptr_t)x % 16) == 0; };
+    const int vec = dk % 4 == 0 && dv % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && aligned(q) && aligned(k) && aligned(v) && aligned(q_norm_w) &&
+                    aligned(k_norm_w) && aligned(v_shared) && aligned(k_pool) && aligned(v_pool);
 #define SLLM_WIDE_LAUNCH(KV)                                                                                                                               \
     do {                                                                                                                                                   \
         if (smem > 48 * 1024)                                                                                                                              \
             SLLM_CUDA(cudaFuncSetAttribute(seq_wide_normed_rotary_kv_kernel<KV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));                 \
         seq_wide_normed_rotary_kv_kernel<KV><<<dim3(b->T, 2), 256, smem, as_stream(stream)>>>(*b, q, ldq, heads, dk, k, ldk, kv_heads, v, ldv, dv, q_norm_w, \
-                                                                                             k_norm_w, eps, freq, n_freq, layout, v_shared, share, lambda, talk, \
-                                                                                             (uint16_t*)q_mixed, k_joint, (KV*)k_pool, (KV*)v_pool);        \
+                                                                                             k_norm_w, eps, (const float2*)angles, n_freq, layout, v_shared, share, lambda, talk, \
+                                                                                             (uint16_t*)q_mixed, k_joint, (KV*)k_pool, (KV*)v_pool, vec);   \
     } while (0)
     if (kv_dtype == SLLM_F32) SLLM_WIDE_LAUNCH(float);
     else SLLM_WIDE_LAUNCH(uint16_t);

@@ -575,7 +575,8 @@ class ScoreMixingAttention:
             raise ValueError(f"{pre}talk is {tuple(self.talk.shape)} for {H} heads")
         self.lam = float(w[pre + "vmix"].float().item()) if share == "blend" else 0.0
         self.n_freq = cfg.rot.dims // 2 if cfg.rot is not None else 0
-        self.freq = torch.tensor(band_frequencies(cfg.rot.dims, cfg.rot.base, cfg.rot.scaling), dtype=torch.float64, device=device) if self.n_freq else None
+        self.freq_key = tuple(band_frequencies(cfg.rot.dims, cfg.rot.base, cfg.rot.scaling)) if self.n_freq else ()
+        self.freq = torch.tensor(self.freq_key, dtype=torch.float64, device=device) if self.n_freq else None
         self.opts = ops.attention_options(chunk=cfg.chunk)
         self.mixes_queries = ops.attention_talk_takes_mixed(H, G, cfg.dim, cfg.vdim)
         self.out = FusedLinear([(w[pre + "o"], w.get(pre + "o.b"))], ops, device)
@@ -614,7 +615,8 @@ class ScoreMixingAttention:
         gate = cols[3] if self.gated else None
         kept = step.scratch("v_kept", T * G * dv) if self.share else None
         mixed = step.scratch("talk_q", (T * H * G * dk + 1) // 2) if self.mixes_queries and T > step.nseg else None
-        ops.wide_normed_rotary_kv(step.b, q, ld, H, dk, k, ld, G, v, ld, dv, self.q_norm, self.k_norm, self.eps, self.freq, self.n_freq, self.layout, state["k"],
+        angles = step.angles(self.freq_key, self.freq) if self.n_freq else None
+        ops.wide_normed_rotary_kv(step.b, q, ld, H, dk, k, ld, G, v, ld, dv, self.q_norm, self.k_norm, self.eps, angles, self.n_freq, self.layout, state["k"],
                                   state["v"], step.st, v_shared=kept, share={None: 0, "keep": 1, "blend": 2}[self.share], lam=self.lam, talk=self.talk,
                                   q_mixed=mixed, k_joint=True)
         nsplit = self._shares(step, mixed is not None)

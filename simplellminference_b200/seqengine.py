@@ -40,10 +40,21 @@ class Step:
         self.nsplit = 1
         self.max_len = engine.max_len     # the most positions a request can hold
         self.sms = torch.cuda.get_device_properties(engine.device).multi_processor_count if engine.device.type == "cuda" else 1
+        self.turned = set()       # frequency sets whose angles this step has already
         self.prev_ids = None      # device array [T]: the token before each token in its sequence, -1 at a sequence's start
 
     def scratch(self, name: str, n_floats: int) -> torch.Tensor:
         return self.engine._scratch(name, n_floats)
+
+    def angles(self, key: tuple, freq: torch.Tensor) -> torch.Tensor:
+        """(cos, sin) of every token's position times every frequency of ``freq``, [T][n][2]: made by the step's first layer with these
+        frequencies (``key``: their values), the same memory for the others."""
+        n = len(key)
+        table = self.engine._scratch(("angles", key), 2 * self.T * n)
+        if key not in self.turned:
+            self.engine.ops.angles(self.b, freq, n, table, self.st)
+            self.turned.add(key)
+        return table
 
     def gemm_scratch(self, K: int, N: int):
         """bf16 copy of the activations + the plain product, for products that go to the tensor cores (None: too few rows to pay)."""
@@ -123,7 +134,7 @@ class SequenceEngine:
         return self.pages.free
 
     # ---- memory ----
-    def _scratch(self, name: str, n_floats: int) -> torch.Tensor:
+    def _scratch(self, name, n_floats: int) -> torch.Tensor:
         t = self._bufs.get(name)
         if t is None or t.numel() < n_floats:
             t = torch.empty(max(n_floats, 1), dtype=torch.float32, device=self.device)
@@ -202,6 +213,7 @@ class SequenceEngine:
         p = self._upload(arrays)
         step = self.step_obj
         step.T, step.nseg = T, nseg
+        step.turned.clear()
         b = step.b
         b.T, b.nseg = T, nseg
         b.tok_slot, b.tok_pos, b.seg_start, b.seg_len, b.seg_slot, b.seg_pos0 = p[1], p[2], p[3], p[4], p[5], p[6]

@@ -114,10 +114,13 @@ class Ops:
         self._ck(self.lib.sllm_seq_normed_rotary_kv(C.byref(b), q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, _p(q_norm_w), _p(k_norm_w), eps,
                                                     _p(freq), n_freq, layout, _p(k_pool), _p(v_pool), self.kv_dtype, st))
 
-    def wide_normed_rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, q_norm_w, k_norm_w, eps, freq, n_freq, layout, k_pool, v_pool,
+    def angles(self, b, freq, n_freq, out, st):
+        self._ck(self.lib.sllm_seq_angles(C.byref(b), _p(freq), n_freq, _p(out), st))
+
+    def wide_normed_rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, q_norm_w, k_norm_w, eps, angles, n_freq, layout, k_pool, v_pool,
                               st, v_shared=None, share=0, lam=0.0, talk=None, q_mixed=None, k_joint=False):
         self._ck(self.lib.sllm_seq_wide_normed_rotary_kv(C.byref(b), q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, _p(q_norm_w), _p(k_norm_w), eps,
-                                                         _p(freq), n_freq, layout, _p(v_shared), share, lam, _p(talk), _p(q_mixed), int(bool(k_joint)), _p(k_pool),
+                                                         _p(angles), n_freq, layout, _p(v_shared), share, lam, _p(talk), _p(q_mixed), int(bool(k_joint)), _p(k_pool),
                                                          _p(v_pool), self.kv_dtype, st))
 
     def head_mix(self, x, ldx, mix, heads, kv_heads, dv, out, ldo, T, st, out16=None):
