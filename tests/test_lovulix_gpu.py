@@ -126,7 +126,7 @@ def test_each_mixer_alone_bf16(portions):
     tiles), single tokens the form that mixes scores."""
     rng = np.random.default_rng(7)
     d, T = 64, 80
-    for layer_cfg in (L.layer(heads=4, kv_heads=2, dim=32, vdim=32, chunk=30), L.layer(heads=8, kv_heads=2, dim=48, vdim=64, chunk=70), L.layer(heads=3, kv_heads=1, dim=16, vdim=24, chunk=None),
+    for layer_cfg in (L.layer(heads=4, kv_heads=2, dim=32, vdim=32, chunk=30), L.layer(heads=8, kv_heads=2, dim=56, vdim=48, chunk=70), L.layer(heads=3, kv_heads=1, dim=16, vdim=24, chunk=None),
                       L.layer(heads=6, kv_heads=2, dim=64, vdim=40, chunk=33), L.layer(heads=16, kv_heads=4, dim=128, vdim=128, chunk=64, rot_dims=128),
                       L.layer(heads=4, kv_heads=4, dim=80, vdim=72, chunk=20), L.layer(heads=3, kv_heads=1, dim=13, vdim=12, chunk=None), L.layer(heads=4, kv_heads=1, dim=32, vdim=136, chunk=17),
                       L.layer(heads=18, kv_heads=2, dim=20, vdim=16, chunk=33)):
@@ -142,7 +142,7 @@ def test_the_two_bf16_forms_agree_on_one_step():
     rounding of the mixed queries."""
     rng = np.random.default_rng(17)
     d, T = 64, 150
-    layer_cfg = L.layer(heads=8, kv_heads=2, dim=48, vdim=64, chunk=70)
+    layer_cfg = L.layer(heads=8, kv_heads=2, dim=56, vdim=48, chunk=70)
     w = L.random_weights(L.make_config([layer_cfg], width=d), seed=14)
     h = L.bf16_round(rng.standard_normal((T, d))).astype(np.float32)
     stub = _mixer_stub([layer_cfg], w, d, dtype="bfloat16")
