@@ -444,6 +444,12 @@ int sllm_seq_linear(const float* A, int32_t lda, const void* W, int32_t w_dtype,
 int sllm_seq_linear_indexed(const float* A, int32_t lda, int64_t a_bs, int32_t a_div, const void* W, int32_t w_dtype, int32_t ldw, int64_t w_bs,
                             const int32_t* w_index, float* C, int32_t ldc, int64_t c_bs, int32_t batch, int32_t N, int32_t K, int32_t round_a,
                             sllm_stream_t stream);
+/* `groups` products one behind the other in ONE launch: C [groups][cap][N] = A [groups][cap][K] . W [groups][N][K]^T for the first counts[g]
+ * rows (device memory) of every group; rows beyond a group's count hold anything. a_bf16 1: A is bf16 (tensor cores: K and N >= 64, K a
+ * multiple of 8, N of 4, aligned), 0: fp32 (FMA tiles, the all-fp32 mode or odd shapes; bf16 weights round A as sllm_seq_linear does).
+ * rows_hint: rows a group is expected to hold. */
+int sllm_seq_linear_grouped(const void* A, int32_t a_bf16, const void* W, int32_t w_dtype, float* C, const int32_t* counts, int32_t groups,
+                            int32_t cap, int32_t rows_hint, int32_t N, int32_t K, sllm_stream_t stream);
 /* 1 when sllm_seq_linear with a bf16 scratch sends this shape to the tensor cores (the weights must also be 16-byte aligned) */
 int sllm_seq_linear_on_tensor_cores(int32_t T, int32_t N, int32_t K, int32_t w_dtype, int32_t ldw, int32_t batch, int32_t round_a);
 /* PolyNorm: out = c0*N(z) + c1*N(z^2) + c2*N(z^3) + c3, powers element-wise, N(v) = v / sqrt(mean(v^2) + eps) over a row; coef: 4 floats */
@@ -543,6 +549,11 @@ int sllm_seq_seam(const sllm_seq_batch* b, const float* x_in, float* x_out, cons
                   float eps, const float* conv_w, int32_t taps, const float* ring, float* h, void* h16, float* stash, float* flush_ring,
                   int32_t flush_taps, int32_t d, float* scales, int32_t post_norm, const float* pre_w, float pre_w_offset, const float* post_w,
                   sllm_stream_t stream);
+/* The seam of a layer whose sublayers run side by side: x_out = x_in + sum_i gain_i * y_i, channel by channel (y_i [T][d], gain_i [d], both host
+ * arrays of n device pointers; normed[i]: y_i is first divided by its rms over d), then, if norm_w [d], h = norm_w * x_out / rms(x_out) as fp32
+ * (h) and / or dense bf16 rows (h16). x_out may be x_in. n <= 4; n = 0 only norms. */
+int sllm_seq_branch_seam(const float* x_in, float* x_out, int32_t n, const float* const* y, const float* const* gain, const int32_t* normed,
+                         float eps, const float* norm_w, float* h, void* h16, int32_t T, int32_t d, sllm_stream_t stream);
 /* out[t][c] = act(cb[c] + sum_j w[c][j] * x[t - taps + 1 + j][c]) (cb NULL = no bias; act 0 = none, 1 = silu), zeros before a sequence's
  * start; inputs before a portion come from ring [slots][taps-1][channels] (position p at row p % (taps-1)), which is NOT updated here
  * (sllm_seq_delta_rule, sllm_seq_ssd_scan, sllm_seq_selective_scan and sllm_seq_ring_store do that, after the convolution has run) */
@@ -558,6 +569,19 @@ int sllm_seq_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, co
                         const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias,
                         int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o,
                         int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, sllm_stream_t stream);
+/* The same rule with a decay per head and key channel: step_logit [T][heads * dk], dt_bias [heads * dk], S[c][:] <- g[c] S[c][:] with
+ * g[c] = exp(-exp(A_log[h]) * softplus(step_logit[h * dk + c] + dt_bias[h * dk + c])); everything else as above. */
+int sllm_seq_channel_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
+                                const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log,
+                                const float* dt_bias, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale,
+                                float* state, float* o, int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps,
+                                float* ring, sllm_stream_t stream);
+/* Linear attention with a constant decay per head over each sequence, state [slots][heads][dk][dv] fp32: S <- decay[h] S + k v^T, o = S^T q.
+ * rate[h] = -ln(decay[h]). silu 1: q, k and v pass silu first; angles (or NULL): (cos, sin) [T][n_freq] of sllm_seq_angles that turn q and k,
+ * pairs by layout as in sllm_seq_rotary_kv; k is then multiplied by kscale. scratch as in sllm_seq_ssd_scan. */
+int sllm_seq_decay_scan(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
+                        const float* decay, const float* rate, const float* angles, int32_t n_freq, int32_t layout, int32_t silu, float kscale,
+                        int32_t heads, int32_t dk, int32_t dv, float* state, float* o, int32_t ldo, float* scratch, sllm_stream_t stream);
 /* State-space duality (Mamba-2) per head h over each sequence, state [slots][heads][n_state][dv] fp32: dt = softplus(step_logit + dt_bias[h]),
  * S <- exp(-exp(A_log[h]) dt) S + dt B x^T, y = S^T C + skip[h] x (skip NULL = no such term); x [T][heads * dv], B and C
  * [T][groups * n_state], head h reads group h / (heads / groups). The kernel of sllm_seq_delta_rule without its correction term; ring as there.
@@ -597,6 +621,15 @@ int sllm_seq_wide_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ld
                                    const float* angles, int32_t n_freq, int32_t layout, float* v_shared, int32_t share, float lambda,
                                    const float* talk, void* q_mixed, int32_t k_joint, void* k_pool, void* v_pool, int32_t kv_dtype,
                                    sllm_stream_t stream);
+/* Between the projections and the attention of a mixer with short convolutions: q, k and v [T][heads * width] each pass a causal convolution per
+ * channel (conv_w [taps][channels], oldest tap first, channels = those of q, k, v in this order; NULL = none; inputs before a portion come from
+ * ring [slots][taps-1][channels]), the first 2*n_freq dimensions of every q and k head are turned by angles [T][n_freq] (sllm_seq_angles), and
+ * with unit 1 every q and k head is divided by sqrt(mean(x^2) + eps). q to q_out (which may be q when there is no convolution), k and v to
+ * their pools. In steps whose portions are all single tokens the ring takes the token's inputs; otherwise sllm_seq_ring_store has to follow. */
+int sllm_seq_conv_rotary_kv(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk,
+                            int32_t kv_heads, const float* v, int32_t ldv, int32_t dv, const float* conv_w, int32_t taps, float* ring,
+                            const float* angles, int32_t n_freq, int32_t layout, int32_t unit, float eps, float* q_out, int32_t ldqo,
+                            void* k_pool, void* v_pool, int32_t kv_dtype, sllm_stream_t stream);
 /* Heads mixed after the attention: in [T][kv_heads * heads * dv] as sllm_seq_attention_finish leaves it for cross_values (record = value
  * head * heads + query head); out[t][h] = sum_g mix[h][g] * in[t][(h / (heads / kv_heads)) * heads + g]: head h's mixed weights on the
  * values of its own key/value head. out fp32 [T][ldo] and / or out16 dense bf16 [T][heads * dv]. */
@@ -604,34 +637,47 @@ int sllm_seq_head_mix(const float* in, int32_t ldi, const float* mix, int32_t he
                       void* out16, int32_t T, sllm_stream_t stream);
 /* Bits of the `act` argument of the mixture-of-experts calls beside the activation (bits 0-1): scores = sigmoid of each router output by
  * itself instead of the softmax over all; gated experts, whose `up` columns are [gate ff | up ff] and which compute act(gate) * up; the
- * score multiplies what the expert reads instead of what it returns. */
+ * score multiplies what the expert reads instead of what it returns; the weights are the chosen scores divided by their sum (+ 1e-20).
+ * Activation 3 (gated experts only): g * sigmoid(1.702 g) * (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit). */
 #define SLLM_MOE_GATED 4
 #define SLLM_MOE_SCALE_INPUT 8
 #define SLLM_MOE_SIGMOID 16
+#define SLLM_MOE_NORMALISE 32
+/* Options (NULL = none): groups > 1: the router outputs form that many equal groups of neighbours, and only those of the `keep` groups with the
+ * largest sum of two choice scores can be chosen; scale: a factor on the weights; limit / shared_limit: of activation 3. */
+typedef struct {
+    int32_t groups, keep;
+    float scale, limit, shared_limit;
+} sllm_seq_moe_opts;
 /* Routing and activation of a mixture of experts, per token: s = softmax(logits[0..n_route)); the `top` largest s + correction are
  * chosen (correction NULL = none; the lower index wins a tie); out / out16 [T][experts * ff] = act(up) * s for chosen experts with
  * weights (the first `experts` router outputs), zeros for the others; y [T][d] = (sum of s over chosen router outputs >= experts) * h:
  * those are experts whose output is their input. act 0 = exact gelu, 1 = tanh gelu, 2 = silu. route_w (or NULL) [T][n_route] = the
- * weights, zero where not chosen. shared_up (or NULL) [T][ldu]: a gated expert of width shared_ff that every token uses, its columns
+ * weights, zero where not chosen. shared_up (or NULL) [T][ld_shared]: a gated expert of width shared_ff that every token uses, its columns
  * [gate | up]; its act(gate) * up follows the experts' columns, rows of out / out16 are then experts * ff + shared_ff wide. */
 int sllm_seq_moe_act(const float* logits, int32_t ldl, int32_t n_route, int32_t experts, int32_t top, const float* correction, const float* up,
                      int32_t ldu, int32_t ff, int32_t act, const float* h, int32_t ldh, int32_t d, float* out, void* out16, float* y,
-                     int32_t ldy, float* route_w, const float* shared_up, int32_t shared_ff, int32_t T, sllm_stream_t stream);
+                     int32_t ldy, float* route_w, const float* shared_up, int32_t ld_shared, int32_t shared_ff, int32_t T,
+                     const sllm_seq_moe_opts* opts, sllm_stream_t stream);
 /* The same layer with the tokens gathered per expert, for steps of many tokens. sllm_seq_moe_route: routing as above; every (token,
  * chosen expert with weights) pair takes the next free row of that expert's buffer (counts [experts] int32, zeroed before the call;
  * buffers of cap >= T rows) and the token's input row h is copied there as bf16 (rows16 [experts][cap][d]) and / or fp32 (rows32);
  * sel_e / sel_pos / sel_w [T][top] = expert (-1: none), row and score of each choice, ident [T] = the sum of the chosen identity scores.
+ * h16 (or NULL): the rows h as dense bf16, copied instead of h (which may then be NULL; d a multiple of 8).
  * Which row a pair gets depends on timing; the numbers in it do not. sllm_seq_moe_expert_act: act over the rows in use of
- * up [experts][cap][ff]. sllm_seq_moe_combine: y[t] = ident[t] * h[t] + sum_k sel_w * down[sel_e][sel_pos] (down [experts][cap][d]). */
+ * up [experts][cap][ff]. sllm_seq_moe_combine: y[t] = ident[t] * h[t] + sum_k sel_w * down[sel_e][sel_pos] (down [experts][cap][d];
+ * h NULL = no identity experts). */
 int sllm_seq_moe_route(const float* logits, int32_t ldl, int32_t n_route, int32_t experts, int32_t top, const float* correction, const float* h,
                        int32_t ldh, int32_t d, int32_t* counts, int32_t cap, int32_t* sel_e, int32_t* sel_pos, float* sel_w, float* ident,
-                       void* rows16, float* rows32, int32_t T, int32_t act, sllm_stream_t stream);
+                       void* rows16, float* rows32, int32_t T, int32_t act, const void* h16, const sllm_seq_moe_opts* opts,
+                       sllm_stream_t stream);
 int sllm_seq_moe_expert_act(const float* up, const int32_t* counts, int32_t experts, int32_t cap, int32_t ff, int32_t act, void* out16,
-                            float* out32, sllm_stream_t stream);
+                            float* out32, float limit, sllm_stream_t stream);
 /* For experts chosen on the device (rows in the order of the (token, choice) pairs, sel_w the pairs' scores as sllm_seq_moe_route leaves them
  * WITHOUT SLLM_MOE_SCALE_INPUT): out [pairs][ff] = act(s * up) or, gated, act(s * gate) * (s * up) over up [pairs][ff or 2 ff], s = the score
  * when `act` has SLLM_MOE_SCALE_INPUT and 1 otherwise; w_out [pairs] = the weight sllm_seq_moe_combine has to use (1, or the score). */
-int sllm_seq_moe_pair_act(const float* up, const float* sel_w, int32_t pairs, int32_t ff, int32_t act, float* out, float* w_out, sllm_stream_t stream);
+int sllm_seq_moe_pair_act(const float* up, const float* sel_w, int32_t pairs, int32_t ff, int32_t act, float* out, float* w_out, float limit,
+                          sllm_stream_t stream);
 int sllm_seq_moe_combine(const float* down, const int32_t* sel_e, const int32_t* sel_pos, const float* sel_w, int32_t top, const float* ident,
                          const float* h, int32_t ldh, int32_t cap, int32_t d, float* y, int32_t ldy, int32_t T, sllm_stream_t stream);
 /* x <- act(x) over n floats (act as in sllm_seq_moe_act). With counts, rows16 and rows32 all NULL sllm_seq_moe_route only routes: nothing is
@@ -670,8 +716,9 @@ int sllm_seq_rglru_scan(const sllm_seq_batch* b, const float* u, int32_t ldu, co
 int sllm_seq_gla_scan(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                       const float* z, int32_t ldz, int32_t heads, int32_t dk, int32_t dv, float qscale, float tau, float* state, float* o,
                       int32_t ldo, void* scratch, sllm_stream_t stream);
-/* out[t][h*dv + j] = o[t][h*dv + j] / sqrt(mean_j(o^2) + eps) * w[j] * silu(g[t][h*dv + j]). mode bit 0: the gate comes first,
- * u = o * silu(g), out = u / sqrt(mean_j(u^2) + eps) * w; bit 1: w has heads * dv entries (one per channel of the row) instead of dv.
+/* out[t][h*dv + j] = o[t][h*dv + j] / sqrt(mean_j(o^2) + eps) * w[j] * silu(g[t][h*dv + j]) (w NULL = no weight). mode bit 0: the gate comes first,
+ * u = o * silu(g), out = u / sqrt(mean_j(u^2) + eps) * w; bit 1: w has heads * dv entries (one per channel of the row) instead of dv;
+ * bit 2: the gate is sigmoid(g) instead of silu(g).
  * out fp32 and / or out16 dense bf16 [T][heads * dv]. */
 int sllm_seq_headnorm_gate(const float* o, int32_t ldo, const float* g, int32_t ldg, const float* w, int32_t heads, int32_t dv, float eps,
                            float* out, int32_t ldout, void* out16, int32_t T, int32_t mode, sllm_stream_t stream);

@@ -129,6 +129,11 @@ class SeqAttnOpts(C.Structure):
     _fields_ = [("window", _I), ("keep_first", _I), ("softcap", _F), ("slopes", _P), ("values_in_keys", _I), ("logdist", _P), ("cross_values", _I), ("chunk", _I)]
 
 
+class SeqMoeOpts(C.Structure):
+    """sllm_seq_moe_opts: groups of experts and how many are kept / factor on the weights / clamp limits of the experts and the shared one."""
+    _fields_ = [("groups", _I), ("keep", _I), ("scale", _F), ("limit", _F), ("shared_limit", _F)]
+
+
 _B = C.POINTER(SeqBatch)
 SIGNATURES.update({
     "sllm_seq_embed": (C.c_int, [_P, _P, _I, _I, _I, _I, _F, _P, _I, _P]),
@@ -136,9 +141,9 @@ SIGNATURES.update({
     "sllm_seq_hyper_write": (C.c_int, [_P, _I, _I, _I, _P, _P, _P, _P]),
     "sllm_seq_hyper_write_read": (C.c_int, [_P, _I, _I, _I, _P, _P, _P, _P, _P, _I, _F, _P, _P]),
     "sllm_seq_linear": (C.c_int, [_P, _I, _P, _I, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _I, _L, _L, _L, _L, _P, _I, _P, _P]),
-    "sllm_seq_moe_route": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P]),
-    "sllm_seq_moe_expert_act": (C.c_int, [_P, _P, _I, _I, _I, _I, _P, _P, _P]),
-    "sllm_seq_moe_pair_act": (C.c_int, [_P, _P, _I, _I, _I, _P, _P, _P]),
+    "sllm_seq_moe_route": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _P, C.POINTER(SeqMoeOpts), _P]),
+    "sllm_seq_moe_expert_act": (C.c_int, [_P, _P, _I, _I, _I, _I, _P, _P, _F, _P]),
+    "sllm_seq_moe_pair_act": (C.c_int, [_P, _P, _I, _I, _I, _P, _P, _F, _P]),
     "sllm_seq_moe_combine": (C.c_int, [_P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P]),
     "sllm_seq_zero": (C.c_int, [_P, _L, _P]),
     "sllm_seq_act": (C.c_int, [_P, _L, _I, _P]),
@@ -167,7 +172,12 @@ SIGNATURES.update({
     "sllm_seq_normed_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _I, _P]),
     "sllm_seq_head_mix": (C.c_int, [_P, _I, _P, _I, _I, _I, _P, _I, _P, _I, _P]),
     "sllm_seq_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P]),
-    "sllm_seq_moe_act": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P]),
+    "sllm_seq_moe_act": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, C.POINTER(SeqMoeOpts), _P]),
+    "sllm_seq_linear_grouped": (C.c_int, [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
+    "sllm_seq_branch_seam": (C.c_int, [_P, _P, _I, C.POINTER(_P), C.POINTER(_P), C.POINTER(_I), _F, _P, _P, _P, _I, _I, _P]),
+    "sllm_seq_channel_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P]),
+    "sllm_seq_decay_scan": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P, _P, _I, _P, _P]),
+    "sllm_seq_conv_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _P]),
     "sllm_seq_layernorm": (C.c_int, [_P, _I, _P, _P, _F, _P, _I, _P, _I, _I, _P]),
     "sllm_seq_depth_average": (C.c_int, [_P, _P, _P, _I, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
     "sllm_seq_clamped_glu": (C.c_int, [_P, _I, _P, _I, _F, _F, _P, _I, _P, _I, _I, _P]),

@@ -1,7 +1,7 @@
 """Model-shape presets (reference: include/model/config.h:5-17 hard-codes ONE shape; BASELINE.json names five)."""
 from __future__ import annotations
 
-from dataclasses import dataclass, asdict
+from dataclasses import dataclass, asdict, replace
 
 F32, BF16, INT8 = 0, 1, 2
 DTYPE_NAMES = {F32: "f32", BF16: "bf16", INT8: "int8"}
@@ -293,12 +293,19 @@ class GatedFeedForwardConfig:
 @dataclass(frozen=True)
 class ExpertsConfig:
     """Mixture of experts: ``experts`` feed-forwards of width ``ff`` and ``identity`` experts without weights (their output is their
-    input) share one router; a token uses the ``top`` best. ``shared``: width of one more expert that every token uses (0 = none)."""
+    input) share one router; a token uses the ``top`` best. ``shared``: width of one more expert that every token uses (0 = none).
+    ``limit`` / ``shared_limit``: where clamped experts clamp; ``groups`` > 1: only experts of the ``keep`` best groups of neighbours can be
+    chosen; ``scale``: a factor on the weights."""
     experts: int
     identity: int
     top: int
     ff: int
     shared: int = 0
+    limit: float = 0.0
+    shared_limit: float = 0.0
+    groups: int = 0
+    keep: int = 0
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -554,8 +561,140 @@ class LovulixConfig:
                              1.0 if scale is None else float(scale), tuple(layers))
 
 
+@dataclass(frozen=True)
+class ConvRotaryAttentionConfig:
+    """Softmax attention with partial rotary positions (``rot`` None = none), a sliding window, optionally capped scores (``softcap`` 0 =
+    no cap) and a short causal convolution of ``conv`` taps on q, k and v (0 = none)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotaryConfig | None
+    mask: WindowMask
+    softcap: float = 0.0
+    conv: int = 0
+
+
+@dataclass(frozen=True)
+class DecayedAttentionConfig:
+    """Linear attention with a constant decay per head (``decay`` [heads]), optionally with rotary positions on q and k."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: RotaryConfig | None = None
+
+
+@dataclass(frozen=True)
+class NelutarLayerConfig:
+    type: str                   # "parallel" | "parallel_2" | "retention"
+    left: object = None         # ConvRotaryAttentionConfig (parallel, parallel_2)
+    right: object = None        # DeltaRuleConfig (parallel) | DecayedAttentionConfig (parallel_2)
+    mixer: object = None        # DecayedAttentionConfig (retention)
+    left_scale: float = 0.5
+    right_scale: float = 0.5
+    mlp: object = None          # GatedFeedForwardConfig | ExpertsConfig | None
+    weights_of: int | None = None
+
+
+@dataclass(frozen=True)
+class NelutarConfig:
+    """The Nelutar design: parallel layers (one RMS norm feeds the mixer and the feed-forward, a weight per channel on each result), a hashed
+    pair embedding, layers that borrow another layer's weights. Mixers: window attention beside the gated delta rule with a decay per key
+    channel (each result normed over the width), window attention with convolved, normed heads and capped scores beside lightning
+    attention, and retention; feed-forwards: gated, or a mixture of clamped experts with a grouped sigmoid router beside a shared one. Every
+    size and constant that may differ comes from config.json."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    pair_buckets: int
+    pair_mul_prev: int
+    pair_mul_cur: int
+    layers: tuple
+
+    @staticmethod
+    def _rotary(m: dict, i: int):
+        rot = m.get("rot")
+        if not rot or not int(rot.get("dims") or 0):
+            return None
+        rot = RotaryConfig(int(rot["dims"]), float(rot["base"]), None)
+        if rot.dims > int(m["dim"]) or rot.dims % 2:
+            raise ValueError(f"layer {i}: {rot.dims} rotary dimensions do not fit heads of {m['dim']}")
+        return rot
+
+    @staticmethod
+    def _grouped_heads(m: dict, i: int) -> tuple:
+        heads = int(m["heads"])
+        kv_heads = int(m.get("kv_heads") or heads)
+        if heads % kv_heads:
+            raise ValueError(f"layer {i}: {heads} heads do not divide over {kv_heads} key heads")
+        return heads, kv_heads
+
+    @staticmethod
+    def _attention(m: dict, i: int) -> ConvRotaryAttentionConfig:
+        heads, kv_heads = NelutarConfig._grouped_heads(m, i)
+        return ConvRotaryAttentionConfig(heads, kv_heads, int(m["dim"]), int(m["vdim"]), float(m["scale"]), NelutarConfig._rotary(m, i), WindowMask.from_dict(m.get("mask")),
+                                         float(m.get("softcap") or 0.0), int(m.get("conv") or 0))
+
+    @staticmethod
+    def _decayed(m: dict, i: int) -> DecayedAttentionConfig:
+        decay = tuple(float(x) for x in m["decay"])
+        if len(decay) != int(m["heads"]) or not all(0.0 < x <= 1.0 for x in decay):
+            raise ValueError(f"layer {i}: {len(decay)} decays for {m['heads']} heads, each has to lie in (0, 1]")
+        return DecayedAttentionConfig(int(m["heads"]), int(m["dim"]), int(m["vdim"]), decay, NelutarConfig._rotary(m, i))
+
+    @staticmethod
+    def _feed_forward(mlp: dict | None, i: int):
+        if mlp is None:
+            return None
+        if mlp.get("kind", "dense") == "dense":
+            return GatedFeedForwardConfig(int(mlp["ff"]))
+        if mlp["kind"] != "moe":
+            raise ValueError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not part of this design")
+        r, shared, groups = mlp["router"], mlp.get("shared") or {}, mlp["router"].get("groups") or {}
+        scale = r.get("scale")
+        ff = ExpertsConfig(int(r["experts"]), 0, int(r["top"]), int(mlp["expert"]["ff"]), int(shared.get("ff") or 0), float(mlp["expert"]["limit"]),
+                           float(shared.get("limit") or 0.0), int(groups.get("count") or 0), int(groups.get("keep") or 0), 1.0 if scale is None else float(scale))
+        if ff.groups and (ff.experts % ff.groups or not 1 <= ff.keep <= ff.groups):
+            raise ValueError(f"layer {i}: {ff.experts} experts in {ff.groups} groups, {ff.keep} kept")
+        if not 1 <= ff.top <= (ff.experts // ff.groups * ff.keep if ff.groups else ff.experts):
+            raise ValueError(f"layer {i}: {ff.top} of {ff.experts} experts")
+        return ff
+
+    @staticmethod
+    def from_dict(c: dict) -> "NelutarConfig":
+        layers = []
+        for i, l in enumerate(c["layers"]):
+            m, kind, src = l["mixer"], l["type"], l.get("weights_of")
+            common = dict(mlp=NelutarConfig._feed_forward(l.get("mlp"), i), weights_of=None if src is None else int(src))
+            if kind == "parallel":
+                heads, kv_heads = NelutarConfig._grouped_heads(m["right"], i)
+                right = DeltaRuleConfig(heads, kv_heads, int(m["right"]["dim"]), int(m["right"]["vdim"]), int(m["right"].get("conv") or 1))
+                layer = NelutarLayerConfig(kind, left=NelutarConfig._attention(m["left"], i), right=right, **common)
+            elif kind == "parallel_2":
+                layer = NelutarLayerConfig(kind, left=NelutarConfig._attention(m["left"], i), right=NelutarConfig._decayed(m["right"], i),
+                                           left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]), **common)
+            elif kind == "retention":
+                layer = NelutarLayerConfig(kind, mixer=NelutarConfig._decayed(m, i), **common)
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            if layer.weights_of is not None:
+                j = layer.weights_of
+                if not 0 <= j < len(c["layers"]) or j == i or c["layers"][j].get("weights_of") is not None:
+                    raise ValueError(f"layer {i}: weights_of {j} must name a layer with tensors of its own")
+            layers.append(layer)
+        for i, layer in enumerate(layers):
+            if layer.weights_of is not None and layer != replace(layers[layer.weights_of], weights_of=layer.weights_of):
+                raise ValueError(f"layer {i} uses the weights of layer {layer.weights_of} and has to be described like it")
+        pair = (c.get("embedding") or {}).get("bigram") or {}
+        return NelutarConfig(c["architecture"], int(c["vocab"]), int(c["width"]), float((c.get("norm") or {}).get("eps", 1e-6)), int(pair.get("buckets") or 0),
+                             int(pair.get("mul_prev") or 0), int(pair.get("mul_cur") or 0), tuple(layers))
+
+
 CONFIG_READERS = {"Munazen": MunazenConfig.from_dict, "Sopetar": SopetarConfig.from_dict, "Vasosun": VasosunConfig.from_dict,
-                  "Kodezen": KodezenConfig.from_dict, "Lovulix": LovulixConfig.from_dict}
+                  "Kodezen": KodezenConfig.from_dict, "Lovulix": LovulixConfig.from_dict, "Nelutar": NelutarConfig.from_dict}
 
 
 def read_model_config(model_dir: str):

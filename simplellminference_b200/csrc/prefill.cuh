@@ -38,6 +38,10 @@ struct PfGemmArgs {
     int32_t bn;           // 0 = choose; 128 / 256 = force the N tile
     const float* bias;    // STORE / RESID / ACCUM: fp32 [N] added to every row of C (once, whatever the split of K), or NULL
     const int32_t* rows_dev;   // device memory or NULL: only the first *rows_dev rows of A (at most T) are multiplied — a count an earlier kernel left
+    // Grouped product (STORE, tiled = 0, no bias): `groups` matrices W [groups][N][K] one behind the other, A [groups][T][K], out [groups][T][ld_out],
+    // rows_dev [groups] — as many row tiles per group as its count asks for, in ONE launch. 0 or 1 = the plain product. rows_hint: rows a group
+    // is expected to hold (for the choice of the tile only).
+    int32_t groups, rows_hint;
 };
 
 struct PfCache;   // tensor-map cache (one CUtensorMap per weight matrix and tile shape), owned by the engine

@@ -57,6 +57,7 @@ struct PfDev {           // kernel-side view of PfGemmArgs
     uint16_t* s_out; int32_t I_loc;
     const float* bias;
     const int32_t* rows_dev;   // the row tiles beyond ceil(*rows_dev / tile rows) are skipped by every role alike
+    int32_t groups;            // matrices one behind the other, each with its own count in rows_dev; T and N are then those of one group
 };
 
 // ------------------------------------------------------------------------------------------ PTX -------
@@ -347,22 +348,36 @@ __global__ void __launch_bounds__(kPfThreads, 1) pf_gemm_kernel(const __grid_con
     // stream) are visible after the wait. The next kernel may start ITS set-up as soon as every CTA here is past this point.
     pdl_wait();
     pdl_launch_dependents();
-    // a row count left by an earlier kernel (tokens routed to one expert): every thread reads the same number, so the three roles walk the
-    // same work units; with no rows at all the kernel only tears down
-    int m_tiles = p.m_tiles;
-    if (p.rows_dev) m_tiles = min(m_tiles, (*p.rows_dev + BM - 1) / BM);
-    const int nunits = m_tiles * p.n_tiles * p.ksplit;
+    // row counts left by an earlier kernel (tokens routed to an expert): every thread reads the same numbers, so the three roles walk the
+    // same work units (all of group 0, then all of group 1, ...); with no rows at all the kernel only tears down
+    struct Walk {
+        const PfDev& p;
+        int g, base, m_tiles;                             // group at hand, its first work unit, its row tiles
+        __device__ __forceinline__ int tiles() const {
+            return p.rows_dev ? min(p.m_tiles, (p.rows_dev[g] + BM - 1) / BM) : p.m_tiles;
+        }
+        __device__ __forceinline__ explicit Walk(const PfDev& q) : p(q), g(0), base(0) { m_tiles = tiles(); }
+        __device__ __forceinline__ bool reach(int unit) {  // units come in ascending order
+            while (unit - base >= m_tiles * p.n_tiles * p.ksplit) {
+                base += m_tiles * p.n_tiles * p.ksplit;
+                if (++g >= p.groups) return false;
+                m_tiles = tiles();
+            }
+            return true;
+        }
+    };
+    Walk walk(p);
 
     if (warp == 0) {
         if (lane == 0) {   // ===== TMA producer =====
             int stage = 0;
             uint32_t phase = 0;
-            for (int unit = worker; unit < nunits; unit += nworkers) {
-                const int tile = unit / p.ksplit, part = unit - tile * p.ksplit;
+            for (int unit = worker; walk.reach(unit); unit += nworkers) {
+                const int tile = (unit - walk.base) / p.ksplit, part = (unit - walk.base) - tile * p.ksplit;
                 const int kb0 = (p.nkb * part) / p.ksplit, kb1 = (p.nkb * (part + 1)) / p.ksplit;
-                const int m_tile = tile % m_tiles, n_tile = tile / m_tiles;   // consecutive workers share the weight tile (L2)
-                const int row0 = m_tile * BM + (int)rank * kPfBM;                  // this CTA's 128 rows of A
-                const int n0 = n_tile * BN + (int)rank * b_rows;                   // this CTA's rows of W
+                const int m_tile = tile % walk.m_tiles, n_tile = tile / walk.m_tiles;   // consecutive workers share the weight tile (L2)
+                const int row0 = walk.g * p.T + m_tile * BM + (int)rank * kPfBM;   // this CTA's 128 rows of A
+                const int n0 = walk.g * p.N + n_tile * BN + (int)rank * b_rows;    // this CTA's rows of W
                 for (int kb = kb0; kb < kb1; ++kb) {
                     mb_wait(empty + stage, phase ^ 1);
                     const int ks = kb / p.kb_per_seg, kk = kb - ks * p.kb_per_seg;
@@ -390,8 +405,8 @@ __global__ void __launch_bounds__(kPfThreads, 1) pf_gemm_kernel(const __grid_con
             const uint32_t idesc = umma_idesc_bf16(BM, BN);
             int stage = 0, acc = 0;
             uint32_t phase = 0, acc_phase = 0;
-            for (int unit = worker; unit < nunits; unit += nworkers) {
-                const int part = unit % p.ksplit;
+            for (int unit = worker; walk.reach(unit); unit += nworkers) {
+                const int part = (unit - walk.base) % p.ksplit;
                 const int kb0 = (p.nkb * part) / p.ksplit, kb1 = (p.nkb * (part + 1)) / p.ksplit;
                 mb_wait(tempty + acc, acc_phase ^ 1);   // the epilogue has drained this accumulator
                 tc_fence_after();
@@ -419,10 +434,11 @@ __global__ void __launch_bounds__(kPfThreads, 1) pf_gemm_kernel(const __grid_con
         int acc = 0;
         uint32_t acc_phase = 0;
         const uint32_t tempty_leader[2] = {PAIR ? mapa_u32(tempty, 0) : 0u, PAIR ? mapa_u32(tempty + 1, 0) : 0u};
-        for (int unit = worker; unit < nunits; unit += nworkers) {
-            const int tile = unit / p.ksplit;
-            const int m_tile = tile % m_tiles, n_tile = tile / m_tiles;
+        for (int unit = worker; walk.reach(unit); unit += nworkers) {
+            const int tile = (unit - walk.base) / p.ksplit;
+            const int m_tile = tile % walk.m_tiles, n_tile = tile / walk.m_tiles;
             const int t = m_tile * BM + (int)rank * kPfBM + row;
+            const int t_out = walk.g * p.T + t;
             mb_wait(tfull + acc, acc_phase);
             tc_fence_after();
 #pragma unroll 1
@@ -431,15 +447,15 @@ __global__ void __launch_bounds__(kPfThreads, 1) pf_gemm_kernel(const __grid_con
                 tc_ld32(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(acc * 256 + c0), v);
                 const int n0 = n_tile * BN + c0;
                 if (t < p.T && n0 < p.N) {
-                    if (p.bias && unit % p.ksplit == 0) {   // the bias rides on the first share of K
+                    if (p.bias && (unit - walk.base) % p.ksplit == 0) {   // the bias rides on the first share of K
 #pragma unroll
                         for (int i = 0; i < 32; ++i)
                             if (n0 + i < p.n_valid) v[i] = __float_as_uint(__uint_as_float(v[i]) + p.bias[n0 + i]);
                     }
                     if (p.epilogue == PF_EPI_QKV) epi_qkv(p, t, n0, v);
                     else if (p.epilogue == PF_EPI_GATEUP) epi_gateup(p, t, n0, v);
-                    else if (p.ksplit > 1) epi_red_add(p, t, n0, v);
-                    else epi_store(p, t, n0, v, p.epilogue == PF_EPI_RESID);
+                    else if (p.ksplit > 1) epi_red_add(p, t_out, n0, v);
+                    else epi_store(p, t_out, n0, v, p.epilogue == PF_EPI_RESID);
                 }
             }
             tc_fence_before();
@@ -502,7 +518,7 @@ static int launch(const CUtensorMap& tmA, const CUtensorMap& tmB, const PfDev& p
         SLLM_CUDA(cudaFuncSetAttribute(pf_gemm_kernel<PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kPfSmem));
         configured = true;
     }
-    const int workers = std::min(PAIR ? sm_count() / 2 : sm_count(), p.m_tiles * p.n_tiles * p.ksplit);
+    const int workers = (int)std::min<long long>(PAIR ? sm_count() / 2 : sm_count(), (long long)p.m_tiles * p.n_tiles * p.ksplit * p.groups);
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3(PAIR ? 2 * workers : workers);
     cfg.blockDim = dim3(kPfThreads);
@@ -525,7 +541,7 @@ static int launch(const CUtensorMap& tmA, const CUtensorMap& tmB, const PfDev& p
 // Host-side plan of one GEMM: cluster shape, N extent of a tile, K split, k-blocks. Pure arithmetic (no device access beyond the
 // cached SM count), exposed as sllm_prefill_gemm_plan for tests.
 struct PfPlan { int pair, bn, ksplit, m_tiles, n_tiles, nkb, kb_per_seg, seg_elems, R; TileGeom g; };
-static PfPlan pf_plan(int T, int N, int K, int tiled, int epilogue, int bn_forced) {
+static PfPlan pf_plan(int T, int N, int K, int tiled, int epilogue, int bn_forced, int groups = 1) {
     PfPlan pl{};
     // more than one 128-row block of tokens: two SMs share a 256-row tile (tcgen05 cta_group::2)
     pl.pair = g_tune_pf_pair >= 0 ? (g_tune_pf_pair != 0) : (T > kPfBM);
@@ -554,7 +570,7 @@ static PfPlan pf_plan(int T, int N, int K, int tiled, int epilogue, int bn_force
         for (int b = 256; b >= 64; b -= 32) {
             for (int sp = 1; sp <= max_split; ++sp) {
                 if (sp > 1 && pl.nkb / sp < 8) break;   // keep at least 8 k-blocks per work unit
-                const long units = (long)pl.m_tiles * ((N + b - 1) / b) * sp;
+                const long units = (long)pl.m_tiles * ((N + b - 1) / b) * sp * groups;
                 const int a_rows = (!pl.pair && T < kPfBM) ? (T + 7) / 8 * 8 : kPfBM;   // operand rows a CTA really ingests per k-block
                 const double unit_cost = (double)((pl.nkb + sp - 1) / sp) * (a_rows + (pl.pair ? b / 2 : b)) + 10.0 * b;
                 const double c = (double)((units + workers - 1) / workers) * unit_cost;
@@ -572,7 +588,10 @@ static PfPlan pf_plan(int T, int N, int K, int tiled, int epilogue, int bn_force
 int pf_gemm(PfCache* cache, const PfGemmArgs& a, cudaStream_t st) {
     SLLM_REQUIRE(cache && a.A && a.W && a.T > 0 && a.N > 0 && a.K > 0, SLLM_EINVAL, "pf_gemm: bad argument");
     SLLM_REQUIRE(a.K % 8 == 0, SLLM_ENOTSUP, "pf_gemm: K=%d must be a multiple of 8", a.K);
-    const PfPlan pl = pf_plan(a.T, a.N, a.K, a.tiled, a.epilogue, a.bn);
+    const int groups = std::max(1, a.groups);
+    SLLM_REQUIRE(groups == 1 || (!a.tiled && a.epilogue == PF_EPI_STORE && !a.bias && a.n_valid == a.N), SLLM_EINVAL, "pf_gemm: a grouped product only stores");
+    PfPlan pl = pf_plan(groups > 1 && a.rows_hint > 0 ? std::min(a.rows_hint, a.T) : a.T, a.N, a.K, a.tiled, a.epilogue, a.bn, groups);
+    if (groups > 1) pl.m_tiles = (a.T + (pl.pair ? 2 : 1) * kPfBM - 1) / ((pl.pair ? 2 : 1) * kPfBM);   // the most a group can hold
     const bool pair = pl.pair != 0;
     const int bn = pl.bn, ksplit = pl.ksplit;
     const TileGeom g = pl.g;
@@ -587,17 +606,18 @@ int pf_gemm(PfCache* cache, const PfGemmArgs& a, cudaStream_t st) {
     p.pos0 = a.pos0; p.sin_t = a.sin_t; p.cos_t = a.cos_t; p.s_out = a.s_out; p.I_loc = a.I_loc;
     p.bias = (a.epilogue == PF_EPI_STORE || a.epilogue == PF_EPI_RESID || a.epilogue == PF_EPI_ACCUM) ? a.bias : nullptr;
     p.rows_dev = a.rows_dev;
+    p.groups = groups;
 
     CUtensorMap tmA;
     {
-        const cuuint64_t dims[2] = {(cuuint64_t)a.K, (cuuint64_t)a.T};
+        const cuuint64_t dims[2] = {(cuuint64_t)a.K, (cuuint64_t)a.T * groups};
         const cuuint64_t strides[1] = {(cuuint64_t)a.K * 2};
         p.a_rows = (!pair && a.T < kPfBM) ? (a.T + 7) / 8 * 8 : kPfBM;
         const cuuint32_t box[2] = {kPfBK, (cuuint32_t)p.a_rows};
         if (int rc = encode(&tmA, a.A, 2, dims, strides, box)) return rc;
     }
     const int box_rows = pair ? bn / 2 : bn;   // W rows one CTA stages per k-block
-    const auto key = std::make_tuple(a.W, a.N, a.K, a.tiled, box_rows);
+    const auto key = std::make_tuple(a.W, a.N * groups, a.K, a.tiled, box_rows);
     auto it = cache->weights.find(key);
     if (it == cache->weights.end()) {
         CUtensorMap tmB;
@@ -607,8 +627,9 @@ int pf_gemm(PfCache* cache, const PfGemmArgs& a, cudaStream_t st) {
             const cuuint32_t box[4] = {kPfBK, (cuuint32_t)g.R, 1, (cuuint32_t)(box_rows / g.R)};
             if (int rc = encode(&tmB, a.W, 4, dims, strides, box)) return rc;
         } else {
-            const cuuint64_t dims[4] = {(cuuint64_t)a.K, (cuuint64_t)a.N, 1, 1};
-            const cuuint64_t strides[3] = {(cuuint64_t)a.K * 2, (cuuint64_t)a.K * 2 * a.N, (cuuint64_t)a.K * 2 * a.N};
+            const cuuint64_t rows = (cuuint64_t)a.N * groups;
+            const cuuint64_t dims[4] = {(cuuint64_t)a.K, rows, 1, 1};
+            const cuuint64_t strides[3] = {(cuuint64_t)a.K * 2, (cuuint64_t)a.K * 2 * rows, (cuuint64_t)a.K * 2 * rows};
             const cuuint32_t box[4] = {kPfBK, (cuuint32_t)box_rows, 1, 1};
             if (int rc = encode(&tmB, a.W, 4, dims, strides, box)) return rc;
         }

@@ -10,6 +10,12 @@
 //     S <- g S + dt B x^T;  y = S^T C + D x,   dt = softplus(a + dt_bias), g = exp(-exp(A_log) dt)
 // with B in the place of k, C in the place of q (neither made a unit vector), x in the place of v, and the heads of a group sharing B and C.
 //
+// Two more forms of the kernel: the delta rule whose decay is a vector per head (one number per key channel, acting on the rows of S), and
+// linear attention with a constant decay per head,
+//     S <- decay S + k v^T;  o = S^T q,
+// whose queries and keys may be rotated by their position and scaled (retention) and whose q, k and v may pass silu (lightning attention)
+// as they arrive in shared memory.
+//
 // The convolution keeps its last taps-1 inputs per sequence in a ring (position p at row p % (taps-1)); the recurrence kernel, which
 // runs after the convolution has read the ring, stores the portion's last inputs there.
 #include <cstdlib>
@@ -47,6 +53,9 @@ struct DeltaArgs {
     const float* conv_x; int ldx, channels, taps; float* ring;   // inputs of the convolution, stored to the ring for the next step (NULL = not)
     int chunk, PP, CB, vec;
     const float* skip;                                  // state-space form: [heads] weight of the input added to the output (NULL = none)
+    const float *decay, *rate;                          // constant decay: [heads] the decay and minus its logarithm
+    const float2* angles; int n_freq, layout;           // constant decay: (cos, sin) [T][n_freq] that turn q and k (NULL = not), pairs as in sllm_seq_rotary_kv
+    int silu;                                           // constant decay: q, k and v pass silu
     float* ws; int nrange;                              // state-space form in three passes: per range and head [dk][dv] states, then the sums of dt
 };
 
@@ -74,11 +83,13 @@ __device__ __forceinline__ void delta_cp4(void* dst, const void* src, bool take)
 
 // CTA = (segment, head, block of CB value columns); thread = (value column j, piece `part` of the key channels), part = tid % PP
 // kForm 0: the delta rule. 1: the state-space form (no correction by the old state, no unit vectors, the step size multiplies the input)
-// over whole portions; 2 / 3: its first and third pass over ranges (2: from zero, no outputs; 3: from the range's start state, no state store)
+// over whole portions; 2 / 3: its first and third pass over ranges (2: from zero, no outputs; 3: from the range's start state, no state store).
+// 4: the delta rule with a decay per key channel. 5 / 6 / 7: as 1 / 2 / 3 with a constant decay per head (qscale then multiplies k).
 template <int kDeltaKP, int kMaxThreads, int kForm>
 __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
     constexpr int kDeltaRS = kDeltaKP + 4;
-    constexpr bool kSsd = kForm != 0, kRanges = kForm >= 2;
+    constexpr bool kChannel = kForm == 4, kFixed = kForm >= 5, kSsd = kForm != 0 && !kChannel;
+    constexpr bool kFromZero = kForm == 2 || kForm == 6, kFromStart = kForm == 3 || kForm == 7, kRanges = kFromZero || kFromStart;
     extern __shared__ __align__(16) float dsm[];
     const sllm_seq_batch& b = p.b;
     const int seg = kRanges ? blockIdx.x / p.nrange : blockIdx.x, rg = kRanges ? blockIdx.x % p.nrange : 0;
@@ -92,17 +103,18 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     // two stages of inputs (the next chunk of tokens travels while this one is walked), then what both share
     const int CBp = (CB + 3) & ~3;                     // every array of a stage starts at a 16-byte boundary
-    const int stage_floats = C * (2 * RS + CBp + 4);   // per token: k and q [RS] each, v [CB], the two logits
+    const int stage_floats = C * ((kChannel ? 3 : 2) * RS + CBp + 4);   // per token: k and q [RS] each, v [CB], the two logits; a decay per channel: [RS] more
     float* s_o = dsm + 2 * stage_floats;               // [C][CB]
     float* s_beta = s_o + C * CB;                      // [C]
     float* s_g = s_beta + C;                           // [C]
     float* s_kq = s_g + C;                             // [C] k . q of the unit vectors
-    const bool vec = p.vec;                            // 16-byte copies of q / k: dk a multiple of 4, rows 16-byte aligned
+    const bool vec = p.vec;                            // 16-byte copies of q / k (and the channels' steps): dk a multiple of 4, rows 16-byte aligned
     auto issue = [&](int c0, int stage) {
         float* d_k = dsm + stage * stage_floats;
         float* d_q = d_k + C * RS;
         float* d_v = d_q + C * RS;
         float* d_l = d_v + C * CBp;                    // [C][2] logits of beta and of the step
+        float* d_a = d_l + C * 4;                      // [C][RS] logits of the channels' steps
         const int n = min(C, len - c0), groups = PP * kDeltaKP / 4;
         for (int i = threadIdx.x; i < n * groups; i += blockDim.x) {               // channels beyond dk are zeros
             const int tok = i / groups, kr = (i % groups) * 4;
@@ -110,6 +122,13 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
             const int at = tok * RS + (kr / kDeltaKP) * kDeltaRS + kr % kDeltaKP;
             const float* ks = p.k + t * p.ldk + (size_t)kvh * dk;
             const float* qs = p.q + t * p.ldq + (size_t)kvh * dk;
+            if (kChannel) {
+                const float* as = p.al + t * p.lda + (size_t)h * dk;
+                if (vec) delta_cp16(d_a + at, kr < dk ? as + kr : as, kr < dk);
+                else
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) delta_cp4(d_a + at + e, kr + e < dk ? as + kr + e : as, kr + e < dk);
+            }
             if (vec) {
                 delta_cp16(d_k + at, kr < dk ? ks + kr : ks, kr < dk);
                 delta_cp16(d_q + at, kr < dk ? qs + kr : qs, kr < dk);
@@ -126,8 +145,9 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
             const float* vs = p.v + (size_t)(start + c0 + i / CB) * p.ldv + (size_t)h * dv;
             delta_cp4(d_v + i, col < dv ? vs + col : vs, col < dv);
         }
-        for (int i = threadIdx.x; i < 2 * n; i += blockDim.x) {
+        for (int i = threadIdx.x; i < (kFixed ? 0 : 2 * n); i += blockDim.x) {
             const size_t t = (size_t)(start + c0 + (i >> 1));
+            if (kChannel && (i & 1)) continue;
             delta_cp4(d_l + i, (i & 1) ? p.al + t * p.lda + h : p.bl + t * p.ldb + h, true);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -137,10 +157,10 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
 #pragma unroll
     for (int x = 0; x < kDeltaKP; ++x) {
         const int kr = part * kDeltaKP + x;
-        S[x] = (kForm != 2 && live && kr < dk) ? st[(size_t)kr * dv + j] : 0.0f;
+        S[x] = (!kFromZero && live && kr < dk) ? st[(size_t)kr * dv + j] : 0.0f;
     }
     float dt_sum = 0.0f;
-    const float rate = expf(p.A_log[h]), bias = p.dt_bias[h];
+    const float rate = kFixed ? 0.0f : expf(p.A_log[h]), bias = (kFixed || kChannel) ? 0.0f : p.dt_bias[h], decay = kFixed ? p.decay[h] : 0.0f;
     const float skip = (kSsd && p.skip) ? p.skip[h] : 0.0f;
     issue(0, 0);
     int stage = 0;
@@ -153,13 +173,50 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
         float* s_q = s_k + C * RS;                     // [C][RS]
         const float* s_v = s_q + C * RS;               // [C][CB]
         const float* s_l = s_v + C * CBp;              // [C][2]
-        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        float* s_a = dsm + stage * stage_floats + C * (2 * RS + CBp + 4);   // [C][RS]
+        for (int i = threadIdx.x; i < (kFixed ? 0 : n); i += blockDim.x) {
+            if (kChannel) {
+                s_beta[i] = seq_sigmoid(s_l[2 * i]);
+                continue;
+            }
             const float dt = seq_softplus(s_l[2 * i + 1] + bias);
             s_beta[i] = kSsd ? dt : seq_sigmoid(s_l[2 * i]);
             s_g[i] = expf(-rate * dt);
         }
+        if (kFixed && p.silu)
+            for (int i = threadIdx.x; i < n * CB; i += blockDim.x) {
+                float* v = dsm + stage * stage_floats + 2 * C * RS + i;
+                *v = *v * seq_sigmoid(*v);
+            }
         for (int tok = warp; tok < n; tok += nwarps) {                             // unit vectors: a warp per token
             float sk = 0.0f, sq = 0.0f, skq = 0.0f;
+            if (kChannel)
+                for (int kr = lane; kr < dk; kr += 32) {
+                    const int at = tok * RS + (kr / kDeltaKP) * kDeltaRS + kr % kDeltaKP;
+                    s_a[at] = expf(-rate * seq_softplus(s_a[at] + p.dt_bias[(size_t)h * dk + kr]));
+                }
+            if (kFixed) {                                                           // silu, rotation and the keys' factor, in place
+                for (int kr = lane; kr < dk && p.silu; kr += 32) {
+                    const int at = tok * RS + (kr / kDeltaKP) * kDeltaRS + kr % kDeltaKP;
+                    s_k[at] = s_k[at] * seq_sigmoid(s_k[at]);
+                    s_q[at] = s_q[at] * seq_sigmoid(s_q[at]);
+                }
+                __syncwarp();
+                for (int i = lane; i < p.n_freq; i += 32) {
+                    const int ka = p.layout == 0 ? 2 * i : i, kb = p.layout == 0 ? 2 * i + 1 : i + p.n_freq;
+                    const int ia = tok * RS + (ka / kDeltaKP) * kDeltaRS + ka % kDeltaKP, ib = tok * RS + (kb / kDeltaKP) * kDeltaRS + kb % kDeltaKP;
+                    const float2 a = p.angles[(size_t)(start + c0 + tok) * p.n_freq + i];
+                    const float ku = s_k[ia], kw = s_k[ib], qu = s_q[ia], qw = s_q[ib];
+                    s_k[ia] = ku * a.x - kw * a.y;
+                    s_k[ib] = kw * a.x + ku * a.y;
+                    s_q[ia] = qu * a.x - qw * a.y;
+                    s_q[ib] = qw * a.x + qu * a.y;
+                }
+                __syncwarp();
+                if (p.qscale != 1.0f)
+                    for (int kr = lane; kr < dk; kr += 32) s_k[tok * RS + (kr / kDeltaKP) * kDeltaRS + kr % kDeltaKP] *= p.qscale;
+                __syncwarp();
+            }
             for (int kr = lane; kr < PP * kDeltaKP; kr += 32) {
                 const int at = tok * RS + (kr / kDeltaKP) * kDeltaRS + kr % kDeltaKP;
                 sk = fmaf(s_k[at], s_k[at], sk);
@@ -184,9 +241,9 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
         // OLD state run side by side (one pass over the piece, ONE round of shuffles for the two sums), and k . q is a number per token:
         // the serial chain of a token holds one reduction instead of two.
         for (int i = 0; i < n; ++i) {
-            const float g = s_g[i], beta = s_beta[i], kq = s_kq[i];
+            const float g = kFixed ? decay : (kChannel ? 1.0f : s_g[i]), beta = kFixed ? 1.0f : s_beta[i], kq = s_kq[i];
             const float4* kk = reinterpret_cast<const float4*>(s_k + i * RS + part * kDeltaRS);
-            if (kForm == 2) {                                                       // the end state only
+            if (kFromZero) {                                                        // the end state only
                 dt_sum += beta;
                 const float u = beta * (live ? s_v[i * CB + jl] : 0.0f);
 #pragma unroll
@@ -200,6 +257,17 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
                 continue;
             }
             const float4* qq = reinterpret_cast<const float4*>(s_q + i * RS + part * kDeltaRS);
+            if (kChannel) {                                                         // the rows of the old state decay first
+                const float4* gg = reinterpret_cast<const float4*>(s_a + i * RS + part * kDeltaRS);
+#pragma unroll
+                for (int x = 0; x < kDeltaKP; x += 4) {
+                    const float4 gv = gg[x >> 2];
+                    S[x] *= gv.x;
+                    S[x + 1] *= gv.y;
+                    S[x + 2] *= gv.z;
+                    S[x + 3] *= gv.w;
+                }
+            }
             float kr[kDeltaKP];
             float d4[4] = {0.0f, 0.0f, 0.0f, 0.0f}, e4[4] = {0.0f, 0.0f, 0.0f, 0.0f};   // four running sums each: no long chain of dependent multiply-adds
 #pragma unroll
@@ -222,25 +290,25 @@ __global__ void __launch_bounds__(kMaxThreads) seq_delta_kernel(DeltaArgs p) {
             const float u = kSsd ? beta * vin : beta * (vin - g * dot);
             if (live && part == 0) s_o[i * CB + jl] = fmaf(u, kq, g * dq) + skip * vin;
 #pragma unroll
-            for (int x = 0; x < kDeltaKP; ++x) S[x] = fmaf(kr[x], u, g * S[x]);
+            for (int x = 0; x < kDeltaKP; ++x) S[x] = fmaf(kr[x], u, kChannel ? S[x] : g * S[x]);
         }
         __syncthreads();
-        if (kForm != 2)
+        if (!kFromZero)
         for (int i = threadIdx.x; i < n * CB; i += blockDim.x) {
             const int col = blockIdx.z * CB + i % CB;
             if (col < dv) p.o[(size_t)(start + c0 + i / CB) * p.ldo + (size_t)h * dv + col] = s_o[i];
         }
     }
-    if (kForm != 3 && live) {
+    if (!kFromStart && live) {
 #pragma unroll
         for (int x = 0; x < kDeltaKP; ++x) {
             const int kr = part * kDeltaKP + x;
             if (kr < dk) st[(size_t)kr * dv + j] = S[x];
         }
     }
-    if (kForm == 2 && threadIdx.x == 0 && blockIdx.z == 0)
+    if (kFromZero && threadIdx.x == 0 && blockIdx.z == 0)
         p.ws[ssd_range_count(b.n_qtiles, b.nseg) * p.heads * dk * dv + ssd_range_id(b, seg, rg) * p.heads + h] = dt_sum;
-    if (kForm != 2 && p.ring && p.taps > 1 && r0 + len == seg_len) {   // the heads of a segment share the job of storing its last inputs of the convolution
+    if (!kFromZero && p.ring && p.taps > 1 && r0 + len == seg_len) {   // the heads of a segment share the job of storing its last inputs of the convolution
         const int seg_start = b.seg_start[seg], pos0 = b.seg_pos0[seg];
         const int keep = min(seg_len, p.taps - 1);
         for (int i = (h * gridDim.z + blockIdx.z) * blockDim.x + threadIdx.x; i < keep * p.channels; i += p.heads * gridDim.z * blockDim.x) {
@@ -256,7 +324,7 @@ __global__ void seq_ssd_carry_kernel(DeltaArgs p) {
     const int seg = blockIdx.z, h = blockIdx.y, per = p.dk * p.dv, e = blockIdx.x * blockDim.x + threadIdx.x;
     if (e >= per) return;
     const int ranges = (b.seg_len[seg] + kSsdRange - 1) / kSsdRange;
-    const float rate = expf(p.A_log[h]);
+    const float rate = p.rate ? p.rate[h] : expf(p.A_log[h]);
     const float* sums = p.ws + ssd_range_count(b.n_qtiles, b.nseg) * p.heads * per;
     float* sp = p.state + ((size_t)b.seg_slot[seg] * p.heads + h) * per + e;
     float S = *sp;
@@ -299,13 +367,21 @@ int sllm_seq_conv_ring(const sllm_seq_batch* b, const float* x, int32_t ldx, int
 
 }  // extern "C"
 
-// both recurrences: `ssd` = the state-space form (skip [heads] or NULL)
-static int delta_run(bool ssd, const float* skip, const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
+// what the forms beyond the plain delta rule and the state-space form bring
+struct DeltaExtra {
+    bool channel = false;                                // the decay's step logits are [heads * dk] per token, dt_bias [heads * dk]
+    const float *decay = nullptr, *rate = nullptr;       // constant decay per head
+    const float* angles = nullptr; int n_freq = 0, layout = 0, silu = 0;
+};
+
+// all recurrences: `ssd` = no correction by the old state (skip [heads] or NULL)
+static int delta_run(bool ssd, const float* skip, const DeltaExtra& ex, const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                      const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias, int32_t heads,
                      int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o, int32_t ldo, const float* conv_x,
                      int32_t ldx, int32_t channels, int32_t taps, float* ring, float* scratch, sllm_stream_t stream) {
     SLLM_REQUIRE(b && b->T > 0 && b->nseg > 0 && b->seg_start && b->seg_len && b->seg_slot && b->seg_pos0, SLLM_EINVAL, "seq_delta_rule: incomplete batch description");
-    SLLM_REQUIRE(q && k && v && beta_logit && step_logit && A_log && dt_bias && state && o, SLLM_EINVAL, "seq_delta_rule / seq_ssd_scan: bad argument");
+    SLLM_REQUIRE(q && k && v && state && o && (ex.decay ? ex.rate != nullptr : beta_logit && step_logit && A_log && dt_bias), SLLM_EINVAL,
+                 "seq_delta_rule / seq_ssd_scan / seq_decay_scan: bad argument");
     SLLM_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0, SLLM_EINVAL, "seq_delta_rule: %d heads over %d key heads", heads, kv_heads);
     SLLM_REQUIRE(!ring || (conv_x && channels > 0 && taps >= 1), SLLM_EINVAL, "seq_delta_rule: the ring needs the convolution's inputs");
     static const int tune_kp = getenv("SLLM_DELTA_KP") ? atoi(getenv("SLLM_DELTA_KP")) : 0;      // measurement aids: 8 / 16 / 32 channels per thread,
@@ -323,7 +399,7 @@ static int delta_run(bool ssd, const float* skip, const sllm_seq_batch* b, const
     if (tune_cb > 0) CB = std::min(dv, tune_cb);
     const int blocks = (dv + CB - 1) / CB;
     const int threads = (CB * PP + 31) / 32 * 32;
-    const int per_tok = 2 * (2 * PP * RSh + ((CB + 3) & ~3) + 4) + CB + 3;      // two stages of inputs, one of outputs
+    const int per_tok = 2 * ((ex.channel ? 3 : 2) * PP * RSh + ((CB + 3) & ~3) + 4) + CB + 3;      // two stages of inputs, one of outputs
     // tokens per stage: every stage costs a round trip to memory and three barriers whatever its size (measured: 12 tokens per stage spent
     // most of the time there), so portions use up to 160 KB of shared memory; steps of single tokens keep the stages small
     static const int tune_chunk = getenv("SLLM_DELTA_CHUNK") ? atoi(getenv("SLLM_DELTA_CHUNK")) : 0;
@@ -340,9 +416,11 @@ static int delta_run(bool ssd, const float* skip, const sllm_seq_batch* b, const
     if (ranges && tune_chunk <= 0) chunk = std::max(4, std::min(chunk, 14336 / per_tok));
     const size_t smem = (size_t)chunk * per_tok * sizeof(float);
     SLLM_REQUIRE(smem <= (size_t)smem_optin_bytes() - 2048, SLLM_ENOTSUP, "seq_delta_rule: one token of a %d x %d head needs %zu bytes of shared memory", dk, dv, smem);
-    const int vec = dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ((uintptr_t)q % 16) == 0 && ((uintptr_t)k % 16) == 0;
+    const int vec = dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ((uintptr_t)q % 16) == 0 && ((uintptr_t)k % 16) == 0 &&
+                    (!ex.channel || (lda % 4 == 0 && ((uintptr_t)step_logit % 16) == 0));
     DeltaArgs p{*b, q, k, v, ldq, ldk, ldv, beta_logit, step_logit, ldb, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state, o, ldo,
-                conv_x, ldx, channels, taps, ring, chunk, PP, CB, vec, skip, scratch, (longest + kSsdRange - 1) / kSsdRange};
+                conv_x, ldx, channels, taps, ring, chunk, PP, CB, vec, skip, ex.decay, ex.rate, (const float2*)ex.angles, ex.n_freq, ex.layout, ex.silu,
+                scratch, (longest + kSsdRange - 1) / kSsdRange};
     SLLM_REQUIRE(!ranges || (long long)b->nseg * p.nrange <= 0x7fffffffLL, SLLM_ENOTSUP, "seq_ssd_scan: %d portions of up to %d ranges", b->nseg, p.nrange);
     const dim3 grid(ranges ? b->nseg * p.nrange : b->nseg, heads, blocks);
 #define SLLM_DELTA_LAUNCH_AS(KPV, MAXT, FORM)                                                                                                             \
@@ -352,15 +430,21 @@ static int delta_run(bool ssd, const float* skip, const sllm_seq_batch* b, const
         ++g_launches;                                                                                                                                     \
         SLLM_LAUNCH_CHECK();                                                                                                                              \
     } while (0)
+#define SLLM_DELTA_RANGES(KPV, MAXT, FIRST, THIRD)                                                                                    \
+    do {                                                                                                                              \
+        SLLM_DELTA_LAUNCH_AS(KPV, MAXT, FIRST);                                                                                       \
+        seq_ssd_carry_kernel<<<dim3((dk * dv + 255) / 256, heads, b->nseg), 256, 0, as_stream(stream)>>>(p);                          \
+        ++g_launches;                                                                                                                 \
+        SLLM_LAUNCH_CHECK();                                                                                                          \
+        SLLM_DELTA_LAUNCH_AS(KPV, MAXT, THIRD);                                                                                       \
+    } while (0)
 #define SLLM_DELTA_LAUNCH(KPV, MAXT)                                                                                                  \
     do {                                                                                                                              \
-        if (ranges) {                                                                                                                 \
-            SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 2);                                                                                       \
-            seq_ssd_carry_kernel<<<dim3((dk * dv + 255) / 256, heads, b->nseg), 256, 0, as_stream(stream)>>>(p);                      \
-            ++g_launches;                                                                                                             \
-            SLLM_LAUNCH_CHECK();                                                                                                      \
-            SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 3);                                                                                       \
-        } else if (ssd) SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 1);                                                                           \
+        if (ex.decay && ranges) SLLM_DELTA_RANGES(KPV, MAXT, 6, 7);                                                                   \
+        else if (ex.decay) SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 5);                                                                        \
+        else if (ranges) SLLM_DELTA_RANGES(KPV, MAXT, 2, 3);                                                                          \
+        else if (ssd) SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 1);                                                                             \
+        else if (ex.channel) SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 4);                                                                      \
         else SLLM_DELTA_LAUNCH_AS(KPV, MAXT, 0);                                                                                      \
     } while (0)
     if (KP == 8) SLLM_DELTA_LAUNCH(8, 1024);
@@ -368,6 +452,7 @@ static int delta_run(bool ssd, const float* skip, const sllm_seq_batch* b, const
     else if (threads <= 256) SLLM_DELTA_LAUNCH(32, 256);
     else SLLM_DELTA_LAUNCH(32, 1024);
 #undef SLLM_DELTA_LAUNCH
+#undef SLLM_DELTA_RANGES
 #undef SLLM_DELTA_LAUNCH_AS
     return SLLM_OK;
 }
@@ -378,7 +463,7 @@ int sllm_seq_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, co
                         int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias, int32_t heads, int32_t kv_heads,
                         int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o, int32_t ldo, const float* conv_x, int32_t ldx,
                         int32_t channels, int32_t taps, float* ring, sllm_stream_t stream) {
-    return delta_run(false, nullptr, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
+    return delta_run(false, nullptr, DeltaExtra{}, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
                      o, ldo, conv_x, ldx, channels, taps, ring, nullptr, stream);
 }
 
@@ -386,8 +471,28 @@ int sllm_seq_ssd_scan(const sllm_seq_batch* b, const float* x, int32_t ldx, cons
                       int32_t lda, const float* A_log, const float* dt_bias, const float* skip, int32_t heads, int32_t groups, int32_t n_state, int32_t dv,
                       float* state, float* y, int32_t ldy, const float* conv_x, int32_t ld_conv, int32_t channels, int32_t taps, float* ring,
                       float* scratch, sllm_stream_t stream) {
-    return delta_run(true, skip, b, C, ldc, B, ldb, x, ldx, step_logit, lda, step_logit, lda, A_log, dt_bias, heads, groups, n_state, dv, 0.0f, 1.0f, state, y, ldy,
+    return delta_run(true, skip, DeltaExtra{}, b, C, ldc, B, ldb, x, ldx, step_logit, lda, step_logit, lda, A_log, dt_bias, heads, groups, n_state, dv, 0.0f, 1.0f, state, y, ldy,
                      conv_x, ld_conv, channels, taps, ring, scratch, stream);
+}
+
+int sllm_seq_channel_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
+                                const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias,
+                                int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o, int32_t ldo,
+                                const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, sllm_stream_t stream) {
+    DeltaExtra ex;
+    ex.channel = true;
+    return delta_run(false, nullptr, ex, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
+                     o, ldo, conv_x, ldx, channels, taps, ring, nullptr, stream);
+}
+
+int sllm_seq_decay_scan(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv, const float* decay,
+                        const float* rate, const float* angles, int32_t n_freq, int32_t layout, int32_t silu, float kscale, int32_t heads, int32_t dk, int32_t dv,
+                        float* state, float* o, int32_t ldo, float* scratch, sllm_stream_t stream) {
+    SLLM_REQUIRE(decay && rate && n_freq >= 0 && 2 * n_freq <= dk && (n_freq == 0 || angles) && (layout == 0 || layout == 1), SLLM_EINVAL, "seq_decay_scan: bad argument");
+    DeltaExtra ex;
+    ex.decay = decay; ex.rate = rate; ex.angles = angles; ex.n_freq = n_freq; ex.layout = layout; ex.silu = silu;
+    return delta_run(true, nullptr, ex, b, q, ldq, k, ldk, v, ldv, nullptr, 0, nullptr, 0, nullptr, nullptr, heads, heads, dk, dv, 0.0f, kscale, state, o, ldo, nullptr, 0, 0,
+                     0, nullptr, scratch, stream);
 }
 
 }  // extern "C"

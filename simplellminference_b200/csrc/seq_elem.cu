@@ -136,6 +136,10 @@ __global__ void seq_gather_rows_kernel(const float* __restrict__ x, int ldx, con
     for (int j = threadIdx.x; j < d; j += blockDim.x) out[(size_t)i * d + j] = src[j];
 }
 
+// mode bits of the norm-and-gate kernels: 1 = the gate multiplies before the root mean square is taken, 2 = a weight per channel of the whole
+// row (else one set shared by the parts), 4 = the gate is sigmoid(g) (else silu(g)); w NULL = no weight
+__device__ __forceinline__ float headnorm_gate_of(float g, int mode) { return (mode & 4) ? seq_sigmoid(g) : g / (1.0f + expf(-g)); }
+
 // one warp per (token, head)
 __global__ void seq_headnorm_gate_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ g, int ldg, const float* __restrict__ w,
                                          int heads, int dv, float eps, float* __restrict__ out, int ldout, uint16_t* __restrict__ out16, int T, int mode) {
@@ -144,20 +148,18 @@ __global__ void seq_headnorm_gate_kernel(const float* __restrict__ o, int ldo, c
     const int t = item / heads, h = item % heads;
     const float* orow = o + (size_t)t * ldo + (size_t)h * dv;
     const float* grow = g + (size_t)t * ldg + (size_t)h * dv;
-    const float* wrow = (mode & 2) ? w + (size_t)h * dv : w;      // a weight per channel of the whole row, or one set shared by the parts
-    const bool gate_first = mode & 1;                             // the gate multiplies before the root mean square is taken
+    const float* wrow = (w && (mode & 2)) ? w + (size_t)h * dv : w;
+    const bool gate_first = mode & 1;
     float ss = 0.0f;
     for (int j = lane; j < dv; j += 32) {
-        const float gv = grow[j];
-        const float v = gate_first ? orow[j] * (gv / (1.0f + expf(-gv))) : orow[j];
+        const float v = gate_first ? orow[j] * headnorm_gate_of(grow[j], mode) : orow[j];
         ss = fmaf(v, v, ss);
     }
     ss = warp_sum(ss);
     const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
     for (int j = lane; j < dv; j += 32) {
-        const float gv = grow[j];
-        const float sg = gv / (1.0f + expf(-gv));
-        const float v = gate_first ? ((orow[j] * sg) * inv) * wrow[j] : ((orow[j] * inv) * wrow[j]) * sg;
+        const float sg = headnorm_gate_of(grow[j], mode), wj = wrow ? wrow[j] : 1.0f;
+        const float v = gate_first ? ((orow[j] * sg) * inv) * wj : ((orow[j] * inv) * wj) * sg;
         if (out) out[(size_t)t * ldout + (size_t)h * dv + j] = v;
         if (out16) out16[(size_t)t * heads * dv + (size_t)h * dv + j] = f32_to_bf16_bits(v);
     }
@@ -166,14 +168,14 @@ __global__ void seq_headnorm_gate_kernel(const float* __restrict__ o, int ldo, c
 // the same with one CTA per (token, part), for parts too wide for a warp (a norm over a few parts of a wide row): the part's gated values
 // wait in registers between the sum of squares and the scaling, kNormPer per thread
 constexpr int kNormPer = 8;
-__global__ void __launch_bounds__(256) seq_headnorm_gate_wide_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ g, int ldg,
+__global__ void __launch_bounds__(1024) seq_headnorm_gate_wide_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ g, int ldg,
                                                                      const float* __restrict__ w, int heads, int dv, float eps, float* __restrict__ out, int ldout,
                                                                      uint16_t* __restrict__ out16, int mode) {
     __shared__ float red[33];
     const int t = blockIdx.x / heads, h = blockIdx.x % heads;
     const float* orow = o + (size_t)t * ldo + (size_t)h * dv;
     const float* grow = g + (size_t)t * ldg + (size_t)h * dv;
-    const float* wrow = (mode & 2) ? w + (size_t)h * dv : w;
+    const float* wrow = (w && (mode & 2)) ? w + (size_t)h * dv : w;
     const bool gate_first = mode & 1;
     float v[kNormPer], sg[kNormPer];
     float ss = 0.0f;
@@ -183,8 +185,7 @@ __global__ void __launch_bounds__(256) seq_headnorm_gate_wide_kernel(const float
         v[i] = 0.0f;
         sg[i] = 0.0f;
         if (j < dv) {
-            const float gv = grow[j];
-            sg[i] = gv / (1.0f + expf(-gv));
+            sg[i] = headnorm_gate_of(grow[j], mode);
             v[i] = gate_first ? orow[j] * sg[i] : orow[j];
             ss = fmaf(v[i], v[i], ss);
         }
@@ -194,7 +195,8 @@ __global__ void __launch_bounds__(256) seq_headnorm_gate_wide_kernel(const float
     for (int i = 0; i < kNormPer; ++i) {
         const int j = threadIdx.x + i * blockDim.x;
         if (j < dv) {
-            const float r = gate_first ? (v[i] * inv) * wrow[j] : ((v[i] * inv) * wrow[j]) * sg[i];
+            const float wj = wrow ? wrow[j] : 1.0f;
+            const float r = gate_first ? (v[i] * inv) * wj : ((v[i] * inv) * wj) * sg[i];
             if (out) out[(size_t)t * ldout + (size_t)h * dv + j] = r;
             if (out16) out16[(size_t)t * heads * dv + (size_t)h * dv + j] = f32_to_bf16_bits(r);
         }
@@ -447,10 +449,11 @@ int sllm_seq_gather_rows(const float* x, int32_t ldx, const int32_t* rows, int32
 
 int sllm_seq_headnorm_gate(const float* o, int32_t ldo, const float* g, int32_t ldg, const float* w, int32_t heads, int32_t dv, float eps, float* out,
                            int32_t ldout, void* out16, int32_t T, int32_t mode, sllm_stream_t stream) {
-    SLLM_REQUIRE(o && g && w && (out || out16) && heads > 0 && dv > 0 && T > 0 && mode >= 0 && mode <= 3, SLLM_EINVAL, "seq_headnorm_gate: bad argument");
+    SLLM_REQUIRE(o && g && (out || out16) && heads > 0 && dv > 0 && T > 0 && mode >= 0 && mode <= 7, SLLM_EINVAL, "seq_headnorm_gate: bad argument");
     const int items = T * heads;
-    if (dv >= 512 && dv <= 256 * kNormPer)       // a warp per part would walk such a part in 16 and more rounds, twice
-        seq_headnorm_gate_wide_kernel<<<items, 256, 0, as_stream(stream)>>>(o, ldo, g, ldg, w, heads, dv, eps, out, ldout, (uint16_t*)out16, mode);
+    if (dv >= 512 && dv <= 1024 * kNormPer)       // a warp per part would walk such a part in 16 and more rounds, twice
+        seq_headnorm_gate_wide_kernel<<<items, std::max(256, ((dv + kNormPer - 1) / kNormPer + 31) / 32 * 32), 0, as_stream(stream)>>>(o, ldo, g, ldg, w, heads, dv, eps, out, ldout,
+                                                                                                                    (uint16_t*)out16, mode);
     else
         seq_headnorm_gate_kernel<<<(items + 3) / 4, 128, 0, as_stream(stream)>>>(o, ldo, g, ldg, w, heads, dv, eps, out, ldout, (uint16_t*)out16, T, mode);
     ++g_launches;

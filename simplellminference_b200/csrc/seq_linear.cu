@@ -19,9 +19,10 @@ struct LinArgs {
     int lda, ldw, ldc, T, N, K, w_dtype, accumulate, round_a;
     float alpha;
     long long a_bs, w_bs, bias_bs, c_bs;
-    const int32_t* rows_dev;   // device memory or NULL: rows from *rows_dev on are not computed (tile body and tensor cores)
+    const int32_t* rows_dev;   // device memory or NULL: rows from rows_dev[b * rows_bs] on are not computed (tile body and tensor cores)
     const int32_t* w_index;    // rows body, device memory or NULL: product b of the batch uses matrix w_index[b] (W + w_index[b] * w_bs); -1 = no matrix, zeros
     int a_div;                 // rows body: product b reads the activations of batch element b / a_div (0 or 1: its own)
+    int rows_bs;               // tile body: 1 = a row count per product of the batch
 };
 
 constexpr int kRowsMax = 8;
@@ -140,7 +141,7 @@ __global__ void __launch_bounds__(256) seq_linear_tile_kernel(LinArgs p) {
     const float* bias = p.bias ? p.bias + (size_t)b * p.bias_bs : nullptr;
     float* C = p.C + (size_t)b * p.c_bs;
     const int m0 = blockIdx.y * kTM, n0 = blockIdx.x * kTN;
-    if (p.rows_dev && m0 >= *p.rows_dev) return;
+    if (p.rows_dev && m0 >= p.rows_dev[b * p.rows_bs]) return;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;   // loader: row lr of the tile, k columns lk .. lk+3
     float acc[4][4];
@@ -242,7 +243,7 @@ extern "C" int sllm_seq_linear_indexed(const float* A, int32_t lda, int64_t a_bs
     SLLM_REQUIRE(A && W && C && w_index && batch > 0 && batch <= 65535 && N > 0 && K > 0 && a_div >= 1, SLLM_EINVAL, "seq_linear_indexed: bad argument");
     SLLM_REQUIRE(lda >= K && ldw >= K && ldc >= N, SLLM_EINVAL, "seq_linear_indexed: row strides shorter than the rows");
     SLLM_REQUIRE(w_dtype == SLLM_F32 || w_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_linear_indexed: fp32 or bf16 weights");
-    LinArgs p{A, W, nullptr, C, lda, ldw, ldc, 1, N, K, w_dtype, 0, round_a, 1.0f, a_bs, w_bs, 0, c_bs, nullptr, w_index, a_div};
+    LinArgs p{A, W, nullptr, C, lda, ldw, ldc, 1, N, K, w_dtype, 0, round_a, 1.0f, a_bs, w_bs, 0, c_bs, nullptr, w_index, a_div, 0};
     return launch_rows(p, batch, as_stream(stream));
 }
 
@@ -258,7 +259,7 @@ extern "C" int sllm_seq_linear(const float* A, int32_t lda, const void* W, int32
     SLLM_REQUIRE(lda >= K && ldw >= K && ldc >= N, SLLM_EINVAL, "seq_linear: row strides shorter than the rows");
     SLLM_REQUIRE(w_dtype == SLLM_F32 || w_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_linear: fp32 or bf16 weights");
     cudaStream_t st = as_stream(stream);
-    LinArgs p{A, W, bias, C, lda, ldw, ldc, T, N, K, w_dtype, accumulate, round_a, alpha, a_bs, w_bs, bias_bs, c_bs, rows_dev, nullptr, 0};
+    LinArgs p{A, W, bias, C, lda, ldw, ldc, T, N, K, w_dtype, accumulate, round_a, alpha, a_bs, w_bs, bias_bs, c_bs, rows_dev, nullptr, 0, 0};
     if (T <= kRowsMax) return launch_rows(p, batch, st);
     // tensor cores: bf16 weights, a dense bf16 copy of A, rows that TMA can address (16-byte multiples) and enough work to fill tiles
     if (a16 && sllm_seq_linear_on_tensor_cores(T, N, K, w_dtype, ldw, batch, round_a) && ((uintptr_t)W % 16) == 0) {
@@ -288,6 +289,32 @@ extern "C" int sllm_seq_linear(const float* A, int32_t lda, const void* W, int32
         return SLLM_OK;
     }
     dim3 grid((N + kTN - 1) / kTN, (T + kTM - 1) / kTM, batch);
+    if (w_dtype == SLLM_BF16) seq_linear_tile_kernel<SLLM_BF16><<<grid, 256, 0, st>>>(p);
+    else seq_linear_tile_kernel<SLLM_F32><<<grid, 256, 0, st>>>(p);
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    return SLLM_OK;
+}
+
+extern "C" int sllm_seq_linear_grouped(const void* A, int32_t a_bf16, const void* W, int32_t w_dtype, float* C, const int32_t* counts, int32_t groups, int32_t cap,
+                                       int32_t rows_hint, int32_t N, int32_t K, sllm_stream_t stream) {
+    SLLM_REQUIRE(A && W && C && counts && groups > 0 && cap > 0 && N > 0 && K > 0, SLLM_EINVAL, "seq_linear_grouped: bad argument");
+    SLLM_REQUIRE(w_dtype == SLLM_F32 || w_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_linear_grouped: fp32 or bf16 weights");
+    SLLM_REQUIRE(groups <= 65535, SLLM_ENOTSUP, "seq_linear_grouped: %d groups", groups);
+    cudaStream_t st = as_stream(stream);
+    if (a_bf16) {        // bf16 rows: ONE tensor-core launch that walks every group's row tiles
+        SLLM_REQUIRE(w_dtype == SLLM_BF16 && K % 8 == 0 && K >= 64 && N >= 64 && N % 4 == 0 && ((uintptr_t)A % 16) == 0 && ((uintptr_t)W % 16) == 0, SLLM_ENOTSUP,
+                     "seq_linear_grouped: %d x %d does not fit the tensor-core tiles", N, K);
+        SLLM_REQUIRE((long long)groups * cap < 0x7fffffffLL && (long long)groups * N < 0x7fffffffLL, SLLM_ENOTSUP, "seq_linear_grouped: too many rows");
+        static PfCache* cache = pf_cache_create();
+        PfGemmArgs a{};
+        a.A = A; a.W = W; a.T = cap; a.N = N; a.K = K; a.epilogue = PF_EPI_STORE; a.out = C; a.ld_out = N; a.n_valid = N; a.rows_dev = counts;
+        a.groups = groups; a.rows_hint = rows_hint;
+        return pf_gemm(cache, a, st);
+    }
+    LinArgs p{(const float*)A, W, nullptr, C, K, K, N, cap, N, K, w_dtype, 0, w_dtype == SLLM_BF16, 1.0f, (long long)cap * K, (long long)N * K, 0, (long long)cap * N,
+              counts, nullptr, 0, 1};
+    dim3 grid((N + kTN - 1) / kTN, (cap + kTM - 1) / kTM, groups);
     if (w_dtype == SLLM_BF16) seq_linear_tile_kernel<SLLM_BF16><<<grid, 256, 0, st>>>(p);
     else seq_linear_tile_kernel<SLLM_F32><<<grid, 256, 0, st>>>(p);
     ++g_launches;

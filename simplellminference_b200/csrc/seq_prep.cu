@@ -10,6 +10,9 @@
 // values optionally blended as in (1); the keys of a token's heads may be stored side by side, and the queries may leave as the mixed
 // bf16 operand rows of attention whose scores are mixed over the heads before the softmax;
 // (6) sllm_seq_angles — cos and sin of every token's position times every frequency, once per step for all layers that turn alike.
+// (7) sllm_seq_conv_rotary_kv — every query, key and value head through a short causal convolution (optional), queries and keys then turned by
+// the step's angles and (optionally) divided by their root mean square; keys and values written to their pools, the convolution's last
+// inputs to their ring in steps of single tokens.
 // All arithmetic is fp32 (angles in double); the pools hold fp32 or bf16.
 #include "seq_common.cuh"
 
@@ -324,6 +327,120 @@ __global__ void __launch_bounds__(256) seq_wide_normed_rotary_kv_kernel(sllm_seq
     }
 }
 
+struct ConvRotaryArgs {
+    sllm_seq_batch b;
+    const float *q, *k, *v; int ldq, ldk, ldv;           // projections: q [heads][dk], k [kv_heads][dk], v [kv_heads][dv] per token
+    int heads, kv_heads, dk, dv;
+    const float* conv_w; int taps; float* ring;          // [taps][channels] (oldest first), channels = q, k, v in this order; ring [slots][taps-1][channels]; NULL = no convolution
+    int store_ring;                                      // every portion is one token: the token's inputs go to the ring here
+    const float2* angles; int n_freq, layout;            // (cos, sin) [T][n_freq]
+    int unit; float eps;                                 // 1: queries and keys divided by their root mean square after they turned
+    float* q_out; int ldqo;                              // may be q itself when there is no convolution
+    void *k_pool, *v_pool;
+    int tile, vec;                                       // tokens a warp walks; 16-byte accesses
+};
+
+// grid (ceil(T / tile), ceil(items / 4)), 4 warps: warp = one head of q, k or v over a tile of tokens; the head's row of the token at hand
+// sits in shared memory while its pairs turn
+template <typename KV>
+__global__ void __launch_bounds__(128) seq_conv_rotary_kv_kernel(ConvRotaryArgs p) {
+    extern __shared__ __align__(16) float cr_sm[];       // [4][max(dk, dv)]
+    const sllm_seq_batch& b = p.b;
+    const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= p.heads + 2 * p.kv_heads) return;
+    const bool is_q = item < p.heads, is_v = item >= p.heads + p.kv_heads;
+    const int g = is_q ? item : (is_v ? item - p.heads - p.kv_heads : item - p.heads), width = is_v ? p.dv : p.dk;
+    const float* src = (is_q ? p.q : (is_v ? p.v : p.k)) + (size_t)g * width;
+    const int ld = is_q ? p.ldq : (is_v ? p.ldv : p.ldk);
+    const int channels = (p.heads + p.kv_heads) * p.dk + p.kv_heads * p.dv;
+    const int ch0 = is_q ? g * p.dk : (is_v ? (p.heads + p.kv_heads) * p.dk + g * p.dv : (p.heads + g) * p.dk);   // the head's first channel of the convolution
+    float* row = cr_sm + (threadIdx.x >> 5) * ((max(p.dk, p.dv) + 3) & ~3);
+    const int t1 = min(b.T, (int)(blockIdx.x + 1) * p.tile);
+    for (int t = blockIdx.x * p.tile; t < t1; ++t) {
+        const int pos = b.tok_pos[t], slot = b.tok_slot[t];
+        const int page = b.block_table[(size_t)slot * b.max_pages + pos / b.page_len], in_page = pos % b.page_len;
+        // the input row `back` positions before the token: a row of this step, a row of the ring, or (before the start) nothing
+        auto earlier = [&](int back) -> const float* {
+            if (pos - back < 0) return nullptr;
+            if (back == 0 || (t - back >= 0 && b.tok_slot[t - back] == slot)) return src + (size_t)(t - back) * ld;
+            return p.ring + ((size_t)slot * (p.taps - 1) + (pos - back) % (p.taps - 1)) * channels + ch0;
+        };
+        float* keep = p.store_ring ? p.ring + ((size_t)slot * (p.taps - 1) + pos % (p.taps - 1)) * channels + ch0 : nullptr;
+        float ss = 0.0f;
+        if (p.vec) {
+            for (int j = 4 * lane; j < width; j += 128) {
+                const float4 own = *reinterpret_cast<const float4*>(src + (size_t)t * ld + j);
+                float4 a = own;
+                if (p.conv_w) {
+                    const float4 w0 = *reinterpret_cast<const float4*>(p.conv_w + (size_t)(p.taps - 1) * channels + ch0 + j);
+                    a = make_float4(w0.x * own.x, w0.y * own.y, w0.z * own.z, w0.w * own.w);
+                    for (int back = 1; back < p.taps; ++back) {
+                        const float* e = earlier(back);
+                        if (!e) break;
+                        const float4 x = *reinterpret_cast<const float4*>(e + j), w = *reinterpret_cast<const float4*>(p.conv_w + (size_t)(p.taps - 1 - back) * channels + ch0 + j);
+                        a = make_float4(fmaf(w.x, x.x, a.x), fmaf(w.y, x.y, a.y), fmaf(w.z, x.z, a.z), fmaf(w.w, x.w, a.w));
+                    }
+                    if (keep) *reinterpret_cast<float4*>(keep + j) = own;      // the oldest row of the ring, read above by this thread
+                }
+                *reinterpret_cast<float4*>(row + j) = a;
+                ss = fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, ss))));
+            }
+        } else {
+            for (int j = lane; j < width; j += 32) {
+                const float own = src[(size_t)t * ld + j];
+                float a = own;
+                if (p.conv_w) {
+                    a = p.conv_w[(size_t)(p.taps - 1) * channels + ch0 + j] * own;
+                    for (int back = 1; back < p.taps; ++back) {
+                        const float* e = earlier(back);
+                        if (!e) break;
+                        a = fmaf(p.conv_w[(size_t)(p.taps - 1 - back) * channels + ch0 + j], e[j], a);
+                    }
+                    if (keep) keep[j] = own;
+                }
+                row[j] = a;
+                ss = fmaf(a, a, ss);
+            }
+        }
+        __syncwarp();
+        if (!is_v && p.n_freq) {
+            for (int i = lane; i < p.n_freq; i += 32) {
+                const int ia = p.layout == 0 ? 2 * i : i, ib = p.layout == 0 ? 2 * i + 1 : i + p.n_freq;
+                const float2 a = p.angles[(size_t)t * p.n_freq + i];
+                const float u = row[ia], w = row[ib];
+                row[ia] = u * a.x - w * a.y;
+                row[ib] = w * a.x + u * a.y;
+            }
+            __syncwarp();
+        }
+        float inv = 1.0f;
+        if (!is_v && p.unit) {
+            if (p.n_freq) {                              // of the turned row, as defined
+                ss = 0.0f;
+                for (int j = lane; j < width; j += 32) ss = fmaf(row[j], row[j], ss);
+            }
+            inv = 1.0f / sqrtf(warp_sum(ss) / (float)width + p.eps);
+        }
+        KV* pool = reinterpret_cast<KV*>(is_v ? p.v_pool : p.k_pool);
+        const size_t dst = is_q ? 0 : seq_pool_row(page, p.kv_heads, g, b.page_len, in_page, width);
+        float* qrow = p.q_out + (size_t)t * p.ldqo + (size_t)g * width;
+        if (p.vec) {
+            for (int j = 4 * lane; j < width; j += 128) {
+                const float4 a = *reinterpret_cast<const float4*>(row + j);
+                const float4 o = make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+                if (is_q) *reinterpret_cast<float4*>(qrow + j) = o;
+                else seq_st4(pool + dst + j, o);
+            }
+        } else {
+            for (int j = lane; j < width; j += 32) {
+                if (is_q) qrow[j] = row[j] * inv;
+                else seq_st(pool, dst + j, row[j] * inv);
+            }
+        }
+        __syncwarp();                                    // the row is free for the next token
+    }
+}
+
 // thread = (token, head, column): out[t][h][c] = sum_g mix[h][g] * in[t][(h / group) * heads + g][c], group = heads / kv_heads: `in` holds,
 // for every key/value head, the result of EVERY query head's weights on that head's values
 __global__ void seq_head_mix_kernel(const float* __restrict__ in, int ldi, const float* __restrict__ mix, int heads, int kv_heads, int dv,
@@ -445,6 +562,32 @@ int sllm_seq_wide_normed_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ld
     if (kv_dtype == SLLM_F32) SLLM_WIDE_LAUNCH(float);
     else SLLM_WIDE_LAUNCH(uint16_t);
 #undef SLLM_WIDE_LAUNCH
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    return SLLM_OK;
+}
+
+int sllm_seq_conv_rotary_kv(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t dk, const float* k, int32_t ldk, int32_t kv_heads,
+                            const float* v, int32_t ldv, int32_t dv, const float* conv_w, int32_t taps, float* ring, const float* angles, int32_t n_freq,
+                            int32_t layout, int32_t unit, float eps, float* q_out, int32_t ldqo, void* k_pool, void* v_pool, int32_t kv_dtype,
+                            sllm_stream_t stream) {
+    SLLM_REQUIRE(b && b->T > 0 && b->tok_slot && b->tok_pos && b->block_table, SLLM_EINVAL, "seq_conv_rotary_kv: incomplete batch description");
+    SLLM_REQUIRE(q && k && v && q_out && k_pool && v_pool && heads > 0 && kv_heads > 0 && dk > 0 && dv > 0, SLLM_EINVAL, "seq_conv_rotary_kv: bad argument");
+    SLLM_REQUIRE(n_freq >= 0 && 2 * n_freq <= dk && (n_freq == 0 || angles), SLLM_EINVAL, "seq_conv_rotary_kv: %d rotary pairs do not fit %d dimensions", n_freq, dk);
+    SLLM_REQUIRE(layout == 0 || layout == 1, SLLM_EINVAL, "seq_conv_rotary_kv: layout 0 (interleaved) or 1 (halves)");
+    SLLM_REQUIRE(!conv_w || (taps >= 1 && (taps == 1 || ring) && q_out != q), SLLM_EINVAL, "seq_conv_rotary_kv: a convolution needs its ring and an output of its own");
+    SLLM_REQUIRE(kv_dtype == SLLM_F32 || kv_dtype == SLLM_BF16, SLLM_ENOTSUP, "seq_conv_rotary_kv: fp32 or bf16 pools");
+    SLLM_REQUIRE(dk <= 2048 && dv <= 2048, SLLM_ENOTSUP, "seq_conv_rotary_kv: heads of %d / %d", dk, dv);
+    auto aligned = [](const void* x) { return x == nullptr || ((uintptr_t)x % 16) == 0; };
+    const int vec = dk % 4 == 0 && dv % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && ldqo % 4 == 0 && aligned(q) && aligned(k) && aligned(v) &&
+                    aligned(conv_w) && aligned(ring) && aligned(q_out) && aligned(k_pool) && aligned(v_pool);
+    const int tile = b->T >= 512 ? 8 : 1;
+    ConvRotaryArgs p{*b, q, k, v, ldq, ldk, ldv, heads, kv_heads, dk, dv, conv_w, taps, conv_w && taps > 1 ? ring : nullptr, conv_w && taps > 1 && b->T == b->nseg,
+                     (const float2*)angles, n_freq, layout, unit, eps, q_out, ldqo, k_pool, v_pool, tile, vec};
+    const dim3 grid((b->T + tile - 1) / tile, (heads + 2 * kv_heads + 3) / 4);
+    const size_t smem = 4 * (size_t)((std::max(dk, dv) + 3) & ~3) * sizeof(float);
+    if (kv_dtype == SLLM_F32) seq_conv_rotary_kv_kernel<float><<<grid, 128, smem, as_stream(stream)>>>(p);
+    else seq_conv_rotary_kv_kernel<uint16_t><<<grid, 128, smem, as_stream(stream)>>>(p);
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     return SLLM_OK;

@@ -4,7 +4,8 @@
 // The same seam serves pre-norm layers: the sum may take y as it is (no norm on the sublayer's output), and the norm in front of the
 // next sublayer may carry a weight per channel stored as its distance from a constant, n = g_pre * (offset + w[c]) * x / rms(x); and layers
 // whose only norm sits on the sublayer's OUTPUT, with a weight per channel: x <- x + g_post * w[c] * y / rms(y), the next sublayer reading x
-// itself (the seam then leaves x as bf16 operand rows).
+// itself (the seam then leaves x as bf16 operand rows). Layers whose sublayers run side by side on one norm's output have a seam of their
+// own (sllm_seq_branch_seam): the sum of several branches, each normed or not, with a weight per channel, then the next layer's norm.
 //
 // The convolution reaches taps-1 tokens back. Inside a portion those are rows of this step: a CTA (one per token) recomputes the
 // residual sum and the norm of its predecessors from the sublayer's input and output (x is therefore read from one buffer and written to
@@ -286,9 +287,156 @@ __global__ void seq_seam_conv_kernel(SeamArgs p, const float* __restrict__ scale
     }
 }
 
+
+// ---- the seam of a layer whose sublayers run side by side -------------------------------------------------------------------------------
+// x <- x + sum_i gain_i * (branch i, or branch i / rms(branch i)), gain_i a weight per channel (a layer scale, a constant factor and a norm's
+// weight are one product), then h = w * x / rms(x) for the next layer, fp32 and / or as bf16 operand rows. CTA = token; the row and its
+// branches stay in registers, E channels at a time, R groups per thread; the branches' root mean squares are ONE reduction.
+constexpr int kMaxBranches = 4;
+struct BranchSeamArgs {
+    const float* x_in; float* x_out;                 // may be the same rows: a CTA owns its row
+    int n; const float* y[kMaxBranches]; const float* gain[kMaxBranches]; int normed[kMaxBranches];
+    float eps;
+    const float* norm_w; float* h; uint16_t* h16;    // norm_w NULL = only the sum
+    int d;
+};
+
+template <int E, int R>
+__global__ void __launch_bounds__(E * R <= 8 ? 1024 : 512) seq_branch_seam_kernel(BranchSeamArgs p) {
+    __shared__ float s_part[kMaxBranches][33];
+    __shared__ float red[33];
+    const int groups = p.d / E, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    const size_t r = (size_t)blockIdx.x * p.d;
+    auto load = [&](const float* src, int j, float (&v)[E]) {
+        if (E == 4) {
+            const float4 f = *reinterpret_cast<const float4*>(src + 4 * j);
+            v[0] = f.x; v[1 % E] = f.y; v[2 % E] = f.z; v[3 % E] = f.w;
+        } else {
+            v[0] = src[j];
+        }
+    };
+    float x[R][E], y[kMaxBranches][R][E];
+    float ss[kMaxBranches];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+#pragma unroll
+        for (int e = 0; e < E; ++e) x[i][e] = 0.0f;
+        if (j < groups) load(p.x_in + r, j, x[i]);
+    }
+#pragma unroll
+    for (int k = 0; k < kMaxBranches; ++k) {
+        ss[k] = 0.0f;
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int j = threadIdx.x + i * blockDim.x;
+#pragma unroll
+            for (int e = 0; e < E; ++e) y[k][i][e] = 0.0f;
+            if (k < p.n && j < groups) load(p.y[k] + r, j, y[k][i]);
+#pragma unroll
+            for (int e = 0; e < E; ++e) ss[k] = fmaf(y[k][i][e], y[k][i][e], ss[k]);
+        }
+    }
+    bool any = false;
+    for (int k = 0; k < p.n; ++k) any |= p.normed[k] != 0;
+    if (any) {                                           // the same answer in every thread
+#pragma unroll
+        for (int k = 0; k < kMaxBranches; ++k) {
+            const float v = warp_sum(ss[k]);
+            if (lane == 0) s_part[k][warp] = v;
+        }
+        __syncthreads();
+        if (warp < kMaxBranches) {
+            const float v = warp_sum(lane < nwarps ? s_part[warp][lane] : 0.0f);
+            if (lane == 0) s_part[warp][32] = v;
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int k = 0; k < kMaxBranches; ++k) {
+        if (k >= p.n) continue;
+        const float inv = p.normed[k] ? 1.0f / sqrtf(s_part[k][32] / (float)p.d + p.eps) : 1.0f;
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+            const int j = threadIdx.x + i * blockDim.x;
+            if (j >= groups) continue;
+            float g[E];
+            load(p.gain[k], j, g);
+#pragma unroll
+            for (int e = 0; e < E; ++e) x[i][e] = fmaf(y[k][i][e] * inv, g[e], x[i][e]);
+        }
+    }
+    float sx = 0.0f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+#pragma unroll
+        for (int e = 0; e < E; ++e) sx = fmaf(x[i][e], x[i][e], sx);     // channels beyond the row are zeros
+        if (j >= groups) continue;
+        if (E == 4) *reinterpret_cast<float4*>(p.x_out + r + 4 * j) = make_float4(x[i][0], x[i][1 % E], x[i][2 % E], x[i][3 % E]);
+        else p.x_out[r + j] = x[i][0];
+    }
+    if (!p.norm_w) return;
+    const float inv = 1.0f / sqrtf(block_sum(sx, red) / (float)p.d + p.eps);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = threadIdx.x + i * blockDim.x;
+        if (j >= groups) continue;
+        float w[E];
+        load(p.norm_w, j, w);
+#pragma unroll
+        for (int e = 0; e < E; ++e) w[e] = (x[i][e] * inv) * w[e];
+        if (E == 4) {
+            if (p.h) *reinterpret_cast<float4*>(p.h + r + 4 * j) = make_float4(w[0], w[1 % E], w[2 % E], w[3 % E]);
+            if (p.h16) *reinterpret_cast<uint2*>(p.h16 + r + 4 * j) = make_uint2(pack_bf16(w[0], w[1 % E]), pack_bf16(w[2 % E], w[3 % E]));
+        } else {
+            if (p.h) p.h[r + j] = w[0];
+            if (p.h16) p.h16[r + j] = f32_to_bf16_bits(w[0]);
+        }
+    }
+}
+
 }  // namespace sllm
 
 using namespace sllm;
+
+extern "C" int sllm_seq_branch_seam(const float* x_in, float* x_out, int32_t n, const float* const* y, const float* const* gain, const int32_t* normed, float eps,
+                                    const float* norm_w, float* h, void* h16, int32_t T, int32_t d, sllm_stream_t stream) {
+    SLLM_REQUIRE(x_in && x_out && T > 0 && d > 0 && n >= 0 && (n == 0 || (y && gain && normed)), SLLM_EINVAL, "seq_branch_seam: bad argument");
+    SLLM_REQUIRE(n <= kMaxBranches, SLLM_ENOTSUP, "seq_branch_seam: %d branches beyond %d", n, kMaxBranches);
+    SLLM_REQUIRE(!norm_w || h || h16, SLLM_EINVAL, "seq_branch_seam: no output for the normed rows");
+    SLLM_REQUIRE(d <= 16384, SLLM_ENOTSUP, "seq_branch_seam: rows of %d floats beyond 16384", d);
+    BranchSeamArgs p{};
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    bool vec = d % 4 == 0 && aligned(x_in) && aligned(x_out) && aligned(norm_w) && aligned(h) && aligned(h16);
+    for (int i = 0; i < n; ++i) {
+        SLLM_REQUIRE(y[i] && gain[i], SLLM_EINVAL, "seq_branch_seam: branch %d is missing", i);
+        p.y[i] = y[i]; p.gain[i] = gain[i]; p.normed[i] = normed[i];
+        vec = vec && aligned(y[i]) && aligned(gain[i]);
+    }
+    p.x_in = x_in; p.x_out = x_out; p.n = n; p.eps = eps; p.norm_w = norm_w; p.h = h; p.h16 = (uint16_t*)h16; p.d = d;
+    // many tokens: CTAs of 256 threads with up to four groups of channels each; few: a thread per group of channels (at least a warp per branch)
+    const int items = vec ? d / 4 : d;
+    int cta = T >= 64 ? std::max(std::min(items, 256), (items + 3) / 4) : items;
+    cta = std::min(items > 2048 ? 512 : 1024, std::max(128, (cta + 31) / 32 * 32));
+    const int per = (items + cta - 1) / cta;
+    SLLM_REQUIRE(per <= (vec ? 8 : 32), SLLM_ENOTSUP, "seq_branch_seam: rows of %d floats", d);
+    cudaStream_t st = as_stream(stream);
+#define SLLM_BRANCH_LAUNCH(E, R) seq_branch_seam_kernel<E, R><<<T, cta, 0, st>>>(p)
+    if (vec) {
+        if (per == 1) SLLM_BRANCH_LAUNCH(4, 1);
+        else if (per == 2) SLLM_BRANCH_LAUNCH(4, 2);
+        else if (per <= 4) SLLM_BRANCH_LAUNCH(4, 4);
+        else SLLM_BRANCH_LAUNCH(4, 8);
+    } else {
+        if (per <= 4) SLLM_BRANCH_LAUNCH(1, 4);
+        else SLLM_BRANCH_LAUNCH(1, 32);
+    }
+#undef SLLM_BRANCH_LAUNCH
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    return SLLM_OK;
+}
 
 extern "C" int sllm_seq_seam(const sllm_seq_batch* b, const float* x_in, float* x_out, const float* y, float post_g, int32_t has_pre, float pre_g,
                              float eps, const float* conv_w, int32_t taps, const float* ring, float* h, void* h16, float* stash, float* flush_ring,

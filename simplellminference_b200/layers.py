@@ -9,7 +9,10 @@ expert every token uses);
 state-space duality (Mamba-2) and the selective scan (Mamba) behind short convolutions; softmax attention whose queries and keys pass a
 convolution and a per-head norm, whose values are the keys before the norm, and whose weights are mixed over the heads after the softmax;
 a feed-forward with biases and the exact gelu; chunked softmax attention with whole-projection norms on queries and keys, scores mixed over
-the heads before the softmax, a sink, blended values and a gate per channel. A mechanism says which per-sequence state it needs
+the heads before the softmax, a sink, blended values and a gate per channel; window softmax attention with partial rotary positions whose
+heads may pass a convolution first and be divided by their root mean square afterwards; the gated delta rule with a decay per key channel;
+linear attention with a constant decay per head (retention, lightning attention); mixers and feed-forwards side by side on one input, each on a
+stream of its own. A mechanism says which per-sequence state it needs
 (``state_spec``); the engine's state manager owns that memory and hands it to ``forward`` — no mechanism keeps a cache of its own.
 
 Additive to the reference, whose only model is the Llama forward of source/model/model.cpp:40-140."""
@@ -86,10 +89,18 @@ class FusedLinear:
         else:
             self.bias = None
 
-    def __call__(self, step, a_ptr, lda, c_ptr, ldc, alpha=1.0, accumulate=False, a16_ready=False):
+    def __call__(self, step, a_ptr, lda, c_ptr, ldc, alpha=1.0, accumulate=False, a16_ready=False, a16=None):
+        """``a16``: dense bf16 rows [T][K] of the input that the caller keeps (only where ``takes_rows16`` says so; the fp32 rows are not read)."""
+        if a16 is not None:
+            self.ops.linear(a16.data_ptr(), self.K, self.w, self.K, self.bias, c_ptr, ldc, step.T, self.N, self.K, step.st, accumulate=accumulate, scratch=a16, a16_ready=True)
+            return
         scratch = step.gemm_scratch(self.K, self.N)
         self.ops.linear(a_ptr, lda, self.w, self.K, self.bias, c_ptr, ldc, step.T, self.N, self.K, step.st, alpha=alpha, accumulate=accumulate,
                         scratch=scratch, a16_ready=a16_ready and scratch is not None)
+
+    def takes_rows16(self, step) -> bool:
+        """Whether this step's product runs on the tensor cores and can read bf16 rows kept by the caller (``a16``)."""
+        return step.engine.tensor_cores and self.ops.on_tensor_cores(step.T, self.N, self.K) and self.w.data_ptr() % 16 == 0
 
     def operand_rows(self, step):
         """Where a kernel that produces this product's input may leave it as bf16 rows [T][K] (then call with ``a16_ready``), or None when
@@ -125,6 +136,14 @@ class GatedRotaryAttention:
         ws = step.scratch("attn_ws", step.T * c.heads * step.nsplit * (c.vdim + 2))
         ops.attention(step.b, q, ld, c.heads, c.kv_heads, c.dim, c.vdim, c.scale, state["k"], state["v"], step.nsplit, ws, step.st)
         ops.attention_finish(step.b, ws, step.nsplit, c.heads, c.vdim, self.vfreq, self.layout, g, ld, out, self.width, step.st)
+
+
+def rotary_frequencies(rot, device):
+    """(their values as a key, the device array) of a rotation without scaling; an empty key and None when there is none."""
+    if rot is None:
+        return (), None
+    key = tuple(rot.base ** (-2.0 * i / rot.dims) for i in range(rot.dims // 2))
+    return key, torch.tensor(key, dtype=torch.float64, device=device)
 
 
 def distance_slopes(heads: int, span: float = 8.0):
@@ -371,6 +390,103 @@ class GatedDeltaRule:
         ops.delta_rule(step.b, u.data_ptr(), C, u.data_ptr() + nk * F32B, C, u.data_ptr() + 2 * nk * F32B, C, bl, ld, al, ld, self.a_log, self.dt_bias,
                        c.heads, c.kv_heads, c.dim, c.vdim, self.unit_eps, c.dim ** -0.5, state["S"], o, self.width, q, ld, C, c.conv, ring, step.st)
         ops.headnorm_gate(o.data_ptr(), self.width, g, ld, self.norm_w, c.heads, c.vdim, self.eps, out, self.width, T, step.st)
+
+
+class ChannelDeltaRule:
+    """Gated delta rule with a decay per head and key channel: as ``GatedDeltaRule`` (short convolutions and silu on q, k and v, unit vectors,
+    beta = sigmoid(W_b h), the state S per head), with S <- diag(g) S in the place of g S,
+    g = exp(-exp(A_log_h) softplus(W_a2 (W_a1 h) + dt_bias)) laid out [heads][dim]; the result is RMS-normed per head (weight ``norm`` shared by
+    the heads), gated by sigmoid(W_g2 (W_g1 h)) and projected. State per sequence: S [heads][dim][vdim] and the convolution's last taps-1
+    inputs (a ring indexed by position), fp32."""
+
+    unit_eps = 1e-6
+
+    def __init__(self, cfg, w, pre, ops, device, eps):
+        self.cfg, self.ops, self.eps = cfg, ops, eps
+        # q, k, v first and adjacent: one convolution runs over all their channels
+        self.inputs = [(w[pre + n], None) for n in ("q", "k", "v", "b", "a1", "g1")]
+        self.conv_w = torch.cat([w[pre + n + ".conv"].float() for n in ("q", "k", "v")], dim=0).contiguous()     # [channels][taps]
+        self.channels = int(self.conv_w.shape[0])
+        if int(self.conv_w.shape[1]) != cfg.conv:
+            raise ValueError(f"{pre}q.conv holds {int(self.conv_w.shape[1])} taps, the configuration says {cfg.conv}")
+        self.a2, self.g2 = (FusedLinear([(w[pre + n], None)], ops, device) for n in ("a2", "g2"))
+        self.a_log = w[pre + "A_log"].float().contiguous()
+        self.dt_bias = w[pre + "dt_bias"].float().contiguous()
+        if self.a2.N != cfg.heads * cfg.dim or tuple(self.dt_bias.shape) != (self.a2.N,):
+            raise ValueError(f"{pre}a2 / dt_bias have {self.a2.N} / {tuple(self.dt_bias.shape)} entries for {cfg.heads} heads of {cfg.dim} key channels")
+        self.norm_w = w[pre + "norm"].float().contiguous()
+        self.out = FusedLinear([(w[pre + "o"], w.get(pre + "o.b"))], ops, device)
+        self.width = cfg.heads * cfg.vdim
+
+    def state_spec(self):
+        c = self.cfg
+        slots = [("S", (c.heads, c.dim, c.vdim))]
+        if c.conv > 1:
+            slots.append(("ring", (c.conv - 1, self.channels)))
+        return {"pages": [], "slots": slots}
+
+    def forward(self, step, cols, ld, state, out):
+        c, ops, T, C = self.cfg, self.ops, step.T, self.channels
+        q, k, v, bl, a1, g1 = cols
+        u = step.scratch("delta_qkv", T * C)
+        ring = state.get("ring")
+        ops.conv_ring(step.b, q, ld, C, c.conv, self.conv_w, ring, 1, u, C, step.st)
+        al = step.scratch("delta_steps", T * self.a2.N)
+        self.a2(step, a1, ld, al.data_ptr(), self.a2.N)
+        gate = step.scratch("delta_gate", T * self.width)
+        self.g2(step, g1, ld, gate.data_ptr(), self.width)
+        nk = c.kv_heads * c.dim
+        o = step.scratch("delta_o", T * self.width)
+        ops.channel_delta_rule(step.b, u.data_ptr(), C, u.data_ptr() + nk * F32B, C, u.data_ptr() + 2 * nk * F32B, C, bl, ld, al.data_ptr(), self.a2.N, self.a_log,
+                               self.dt_bias, c.heads, c.kv_heads, c.dim, c.vdim, self.unit_eps, c.dim ** -0.5, state["S"], o, self.width, q, ld, C, c.conv, ring,
+                               step.st)
+        rows16 = self.out.operand_rows(step)
+        ops.headnorm_gate(o.data_ptr(), self.width, gate.data_ptr(), self.width, self.norm_w, c.heads, c.vdim, self.eps, None if rows16 is not None else out, self.width, T,
+                          step.st, out16=rows16, sigmoid_gate=True)
+        return rows16 is not None
+
+
+class DecayedAttention:
+    """Linear attention with a constant decay per head and no softmax: S <- decay_h S + k v^T, o = S^T q. ``silu``: q, k and v pass silu first
+    (lightning attention); ``cfg.rot``: q and k turn by their position (pairs by ``layout``); k is multiplied by ``kscale`` afterwards
+    (retention). The result is RMS-normed per head without a weight, or (``row_norm``) over all heads together with the weight ``norm``,
+    multiplied by silu (``sigmoid_gate``: sigmoid) of W_g h and projected. State per sequence: S [heads][dim][vdim], fp32."""
+
+    scan_range = 128     # tokens of a range of the kernel's three-pass form (kSsdRange of csrc/seq_delta.cu)
+
+    def __init__(self, cfg, w, pre, ops, device, eps, silu=False, layout=1, kscale=1.0, row_norm=False, sigmoid_gate=False):
+        self.cfg, self.ops, self.eps = cfg, ops, eps
+        self.silu, self.layout, self.kscale, self.row_norm, self.sigmoid_gate = silu, layout, kscale, row_norm, sigmoid_gate
+        self.inputs = [(w[pre + n], None) for n in ("q", "k", "v", "g")]
+        self.decay = torch.tensor(cfg.decay, dtype=torch.float32, device=device)
+        self.rate = torch.tensor([-math.log(x) for x in cfg.decay], dtype=torch.float32, device=device)
+        self.freq_key, self.freq = rotary_frequencies(cfg.rot, device)
+        self.norm_w = w[pre + "norm"].float().contiguous() if row_norm else None
+        self.out = FusedLinear([(w[pre + "o"], w.get(pre + "o.b"))], ops, device)
+        self.width = cfg.heads * cfg.vdim
+
+    def state_spec(self):
+        c = self.cfg
+        return {"pages": [], "slots": [("S", (c.heads, c.dim, c.vdim))]}
+
+    def prepare(self, step):
+        return step.angles(self.freq_key, self.freq) if self.freq_key else None
+
+    def forward(self, step, cols, ld, state, out):
+        c, ops, T = self.cfg, self.ops, step.T
+        q, k, v, g = cols
+        o = step.scratch("decay_o", T * self.width)
+        # a portion longer than a range of the scan: per range and head its end state from zero and its token count (three passes)
+        ws = None
+        if T - step.nseg + 1 > self.scan_range:
+            ws = step.scratch("decay_ranges", (step.b.n_qtiles // 4 + step.nseg + 1) * c.heads * (c.dim * c.vdim + 1))
+        ops.decay_scan(step.b, q, ld, k, ld, v, ld, self.decay, self.rate, self.prepare(step), len(self.freq_key), self.layout, self.silu, self.kscale, c.heads, c.dim,
+                       c.vdim, state["S"], o, self.width, step.st, scratch=ws)
+        rows16 = self.out.operand_rows(step)
+        heads, width = (1, self.width) if self.row_norm else (c.heads, c.vdim)
+        ops.headnorm_gate(o.data_ptr(), self.width, g, ld, self.norm_w, heads, width, self.eps, None if rows16 is not None else out, self.width, T, step.st, out16=rows16,
+                          sigmoid_gate=self.sigmoid_gate)
+        return rows16 is not None
 
 
 class StateSpaceDuality:
@@ -627,9 +743,60 @@ class ScoreMixingAttention:
         return rows16 is not None
 
 
+class ConvRotaryAttention:
+    """Softmax attention over a paged cache with grouped query heads: q, k and v may pass a short causal convolution per channel (``cfg.conv`` > 0;
+    tensors ``q.conv`` / ``k.conv`` / ``v.conv``, no bias) directly after their projections; q and k turn by their position on the first
+    ``rot.dims`` dimensions of each head (pairs by ``layout``) and, with ``unit_heads``, are then divided by their root mean square (no
+    weight); scores may be capped, cap * tanh(q.k * scale / cap); a sliding window. State per sequence: the k and v pools and the
+    convolution's last taps-1 inputs (a ring indexed by position)."""
+
+    def __init__(self, cfg, w, pre, ops, device, eps, layout=0, unit_heads=False):
+        self.cfg, self.ops, self.eps, self.layout, self.unit_heads = cfg, ops, eps, layout, unit_heads
+        self.inputs = [(w[pre + n], w.get(pre + n + ".b")) for n in ("q", "k", "v")]      # adjacent: one convolution runs over all their channels
+        self.channels = (cfg.heads + cfg.kv_heads) * cfg.dim + cfg.kv_heads * cfg.vdim
+        self.conv_w = None
+        if cfg.conv:
+            taps = torch.cat([w[pre + n + ".conv"].float() for n in ("q", "k", "v")], dim=0)
+            if tuple(taps.shape) != (self.channels, cfg.conv):
+                raise ValueError(f"{pre}q.conv / k.conv / v.conv hold {tuple(taps.shape)}, the configuration says {(self.channels, cfg.conv)}")
+            self.conv_w = taps.t().contiguous()                                            # [taps][channels]
+        self.freq_key, self.freq = rotary_frequencies(cfg.rot, device)
+        self.opts = ops.attention_options(cfg.mask.size, cfg.mask.keep_first, cfg.softcap)
+        self.out = FusedLinear([(w[pre + "o"], w.get(pre + "o.b"))], ops, device)
+        self.width = cfg.heads * cfg.vdim
+
+    def state_spec(self):
+        c = self.cfg
+        slots = [("ring", (c.conv - 1, self.channels))] if c.conv > 1 else []
+        return {"pages": [("k", c.kv_heads, c.dim), ("v", c.kv_heads, c.vdim)], "slots": slots}
+
+    def prepare(self, step):
+        return step.angles(self.freq_key, self.freq) if self.freq_key else None
+
+    def forward(self, step, cols, ld, state, out):
+        c, ops, T = self.cfg, self.ops, step.T
+        q, k, v = cols
+        ring = state.get("ring")
+        qo, ldq = q, ld
+        if self.conv_w is not None:
+            ldq = c.heads * c.dim
+            qo = step.scratch("attn_q", T * ldq).data_ptr()
+        ops.conv_rotary_kv(step.b, q, ld, c.heads, c.dim, k, ld, c.kv_heads, v, ld, c.vdim, self.conv_w, c.conv, ring, self.prepare(step), len(self.freq_key), self.layout,
+                           self.unit_heads, self.eps, qo, ldq, state["k"], state["v"], step.st)
+        if ring is not None and T > step.nseg:
+            ops.ring_store(step.b, q, ld, self.channels, c.conv, ring, step.st)
+        ws = step.scratch("attn_ws", T * c.heads * step.nsplit * (c.vdim + 2))
+        ops.attention(step.b, qo, ldq, c.heads, c.kv_heads, c.dim, c.vdim, c.scale, state["k"], state["v"], step.nsplit, ws, step.st, opts=self.opts)
+        rows16 = self.out.operand_rows(step)
+        ops.attention_finish(step.b, ws, step.nsplit, c.heads, c.vdim, None, 0, None, 0, None if rows16 is not None else out, self.width, step.st, out16=rows16)
+        return rows16 is not None
+
+
 class MixerGroup:
     """One or more mechanisms reading the same input: their input projections run as one fused product, each mechanism's result goes
-    through its own output projection, and the results are added with the given weights."""
+    through its own output projection, and the results are added with the given weights — or, when ``forward`` is handed one output per
+    member, kept apart: the members then run side by side (``Step.side_by_side``) and the caller adds their results. A feed-forward that
+    brings products of its own beyond input and output (``run``) can be a member of such a group."""
 
     def __init__(self, members, ops, device):
         self.members = members                       # [(name, mechanism, weight)]
@@ -651,17 +818,68 @@ class MixerGroup:
             spec["borrow"] += [(f"{name}.{n}", run, f"{name}.{src}") for n, run, src in s.get("borrow", [])]
         return spec
 
-    def forward(self, step, h, state, y, h16_ready=False):
-        """h [T][d] -> y [T][d]; ``h16_ready``: the kernel that wrote h also left it in ``self.proj.operand_rows(step)``."""
+    def reads_f32(self, step) -> bool:
+        """Whether a step whose input exists as bf16 rows (``self.proj.takes_rows16``) needs the fp32 rows too."""
+        return any(m.reads_f32(step) for _, m, _ in self.members if hasattr(m, "run"))
+
+    def _side_by_side(self, step, h, cols, state, outs, h16):
+        N = self.proj.N
+
+        def task(name, m, span, y):
+            ptrs = [cols.data_ptr() + o * F32B for o in span]
+            sub = {k[len(name) + 1:]: t for k, t in state.items() if k.startswith(name + ".")}
+
+            def run():
+                if hasattr(m, "run"):
+                    m.run(step, ptrs, N, h, h16, y)
+                    return
+                part = step.scratch("mix_part", step.T * m.width)
+                ready = m.forward(step, ptrs, N, sub, part)
+                m.out(step, part.data_ptr(), m.width, y.data_ptr(), m.out.N, a16_ready=ready is True)
+            return run
+
+        for _, m, _ in self.members:           # what several members may share is made before they part
+            if hasattr(m, "prepare"):
+                m.prepare(step)
+        step.side_by_side([task(name, m, span, y) for (name, m, _), span, y in zip(self.members, self.spans, outs)])
+
+    def forward(self, step, h, state, y, h16_ready=False, h16=None):
+        """h [T][d] -> y [T][d], or y = a list with an output per member; ``h16_ready``: the kernel that wrote h also left it in
+        ``self.proj.operand_rows(step)``; ``h16``: bf16 rows of h that the caller keeps (then h may be None where ``reads_f32`` says no)."""
         T, N = step.T, self.proj.N
         cols = step.scratch("mix_cols", T * N)
-        self.proj(step, h.data_ptr(), self.proj.K, cols.data_ptr(), N, a16_ready=h16_ready)
+        self.proj(step, None if h16 is not None else h.data_ptr(), self.proj.K, cols.data_ptr(), N, a16_ready=h16_ready, a16=h16)
+        if isinstance(y, (list, tuple)):
+            self._side_by_side(step, h, cols, state, y, h16)
+            return
         for i, ((name, m, weight), span) in enumerate(zip(self.members, self.spans)):
             part = step.scratch("mix_part", T * m.width)
             sub = {k[len(name) + 1:]: t for k, t in state.items() if k.startswith(name + ".")}
             # a member whose forward says True has left its result as bf16 operand rows of its output projection
             ready = m.forward(step, [cols.data_ptr() + o * F32B for o in span], N, sub, part)
             m.out(step, part.data_ptr(), m.width, y.data_ptr(), m.out.N, alpha=weight, accumulate=i > 0, a16_ready=ready is True)
+
+
+class SiluGluFeedForward:
+    """Gated feed-forward W_down (silu(W_gate h) * (W_up h)) with the interface of a mixer, so that a ``MixerGroup`` runs it beside a mixer on
+    the same normed input: one fused input product."""
+
+    def __init__(self, cfg, w, pre, ops, device):
+        self.ops = ops
+        self.inputs = [(w[pre + "gate"], None), (w[pre + "up"], None)]
+        self.out = FusedLinear([(w[pre + "down"], None)], ops, device)
+        self.width = cfg.ff
+        if self.out.K != cfg.ff:
+            raise ValueError(f"{pre}down has {self.out.K} columns, the configuration says {cfg.ff}")
+
+    def state_spec(self):
+        return {"pages": [], "slots": []}
+
+    def forward(self, step, cols, ld, state, out):
+        gate, up = cols
+        rows16 = self.out.operand_rows(step)
+        self.ops.gated_act(gate, ld, up, ld, None if rows16 is not None else out, self.width, step.T, self.width, step.st, out16=rows16)
+        return rows16 is not None
 
 
 class ClampedGluFeedForward:
@@ -764,63 +982,89 @@ class ExpertsFeedForward:
 
     Steps of ``gather_min_tokens`` tokens and more (portions of prompts) take the gathered form instead, which multiplies a token only
     with the experts it uses: the router alone, then a routing kernel that copies every token's input into a buffer per chosen expert,
-    per expert an up product, the activation, a down product over the rows in use (their count never leaves the device), and a kernel
-    that adds each token's rows times their scores. Steps of one or two tokens (decoding) whose experts are large take the indexed
-    form: the router, a routing kernel, and ONE up and ONE down launch in which every (token, choice) pair streams only its own expert's
-    matrix, chosen on the device. All forms give the same numbers up to where the score is multiplied in.
+    ONE up product and ONE down product over all experts' buffers (as many row tiles per expert as it has tokens: the counts never leave the
+    device) with the activation between them, and a kernel that adds each token's rows times their scores. Steps of one or two tokens
+    (decoding) whose experts are large take the indexed form: the router, a routing kernel, and ONE up and ONE down launch in which every
+    (token, choice) pair streams only its own expert's matrix, chosen on the device. All forms give the same numbers up to where the score
+    is multiplied in.
 
     ``shared`` > 0 (tensors ``shared.gate`` / ``shared.up`` / ``shared.down``; gated experts): one more expert of that width which every token
     uses with weight one. Its first product rides with the experts' (wide form) or the router's (the others), its second with the wide down
-    product or as a product of its own that adds to the result."""
+    product or as a product of its own that adds to the result.
+
+    ``in_group``: the layer is a member of a ``MixerGroup`` (``inputs`` / ``run``): router and the shared expert's first product are part of the
+    group's fused input product."""
 
     activation = 0          # the exact (erf) gelu
-    GATED, SCALE_INPUT, SIGMOID = 4, 8, 16      # SLLM_MOE_* bits beside the activation
-    # The gathered form trades arithmetic for launches (two products per expert): it is taken when the products it saves, at the rate the
-    # tensor-core product sustains, outweigh what its launches cost (both measured on B200: small experts are faster computed densely).
-    gather_min_tokens = 256
-    gather_launch_cost = 35e-6     # seconds per expert product
+    CLAMPED = 3             # activation number of gated experts with clamped branches, g * sigmoid(1.702 g) * (u + 1)
+    clamped_alpha = 1.702
+    GATED, SCALE_INPUT, SIGMOID, NORMALISE = 4, 8, 16, 32      # SLLM_MOE_* bits beside the activation
+    # The gathered form is taken when the products it saves, at the rate the tensor-core product sustains, outweigh its extra launches and the
+    # rows it copies.
+    gather_min_tokens = 64
+    gather_launch_cost = 30e-6     # seconds per layer
     gather_product_rate = 7e14     # multiply-adds * 2 per second
     # The indexed form reads (pairs / experts) of the expert bytes at the price of three more launches per layer
     index_launch_cost = 12e-6      # seconds for the three extra launches of a step replayed as a graph
     index_stream_rate = 5e12       # bytes per second the weight-streaming body sustains
 
-    def __init__(self, cfg, w, pre, ops, device, activation=None, gated=False, sigmoid_scores=False, scale_input=False):
+    def __init__(self, cfg, w, pre, ops, device, activation=None, gated=False, sigmoid_scores=False, scale_input=False, normalise=False, in_group=False):
         """``gated``: experts W_down (act(W_gate h) * (W_up h)) with tensors ``e<i>.gate`` beside ``up`` / ``down``; ``sigmoid_scores``: the score
-        of a router output is its own sigmoid (no softmax over all); ``scale_input``: the score multiplies what the expert reads."""
+        of a router output is its own sigmoid (no softmax over all); ``scale_input``: the score multiplies what the expert reads;
+        ``normalise``: the weights are the chosen scores divided by their sum. ``cfg.scale`` multiplies the weights, ``cfg.groups`` /
+        ``cfg.keep`` restrict the choice to the best groups of experts, ``cfg.limit`` / ``cfg.shared_limit`` are the clamped activation's."""
         self.cfg, self.ops = cfg, ops
         E = cfg.experts
-        self.gated, self.scale_input = bool(gated), bool(scale_input)
+        self.gated, self.scale_input, self.in_group = bool(gated), bool(scale_input), bool(in_group)
         act = self.activation if activation is None else activation
-        self.mode = act | (self.GATED if gated else 0) | (self.SCALE_INPUT if scale_input else 0) | (self.SIGMOID if sigmoid_scores else 0)
+        self.clamped = act == self.CLAMPED
+        self.mode = (act | (self.GATED if gated else 0) | (self.SCALE_INPUT if scale_input else 0) | (self.SIGMOID if sigmoid_scores else 0)
+                     | (self.NORMALISE if normalise else 0))
+        self.opts = ops.moe_options(cfg.groups, cfg.keep, cfg.scale, cfg.limit, cfg.shared_limit)
         self.ff_up = (2 if gated else 1) * cfg.ff          # columns of one expert's first product: [gate | up] or up
         self.n_route = E + cfg.identity
         if int(w[pre + "router"].shape[0]) != self.n_route:
             raise ValueError(f"{pre}router has {int(w[pre + 'router'].shape[0])} outputs, the configuration names {self.n_route} experts")
         self.correction = w[pre + "correction"].float().contiguous() if pre + "correction" in w else None
-        # experts first, router last: the experts' columns then start at a 16-byte boundary for every ff
         first = [torch.cat([w[f"{pre}e{e}.gate"], w[f"{pre}e{e}.up"]], dim=0) if gated else w[f"{pre}e{e}.up"] for e in range(E)]
         self.shared_ff = cfg.shared
         if self.shared_ff and not gated:
             raise ValueError("an expert that every token uses is a gated one here")
+        # what every token needs: [shared gate | shared up |] router
         common = [(w[f"{pre}shared.{n}"], None) for n in ("gate", "up")] if self.shared_ff else []
-        self.up = FusedLinear([(m, None) for m in first] + common + [(w[pre + "router"], None)], ops, device, pad_rows=8)
+        common.append((w[pre + "router"], None))
+        if int(common[0][0].shape[0]) != (self.shared_ff or self.n_route):
+            raise ValueError(f"{pre}shared.gate has {int(common[0][0].shape[0])} rows, the configuration says {self.shared_ff}")
+        self.inputs = common
+        # experts first, the common columns last: the experts' columns then start at a 16-byte boundary for every ff
+        self.up = FusedLinear([(m, None) for m in first] + ([] if in_group else common), ops, device, pad_rows=8)
         downs = [w[f"{pre}e{e}.down"] for e in range(E)] + ([w[pre + "shared.down"]] if self.shared_ff else [])
         self.down = FusedLinear([(torch.cat(downs, dim=1).contiguous(), None)], ops, device)
         self.wide = E * cfg.ff + self.shared_ff    # columns of the activation = rows of the concatenated down matrices
-        self.wide_up = E * self.ff_up              # columns of all experts' first products; the shared expert's, then the router's follow
-        if self.up.sizes[E] != (self.shared_ff or self.n_route):
-            raise ValueError(f"{pre}shared.gate has {self.up.sizes[E]} rows, the configuration says {self.shared_ff}")
+        self.wide_up = E * self.ff_up              # columns of all experts' first products; the common ones follow
         # the gathered form: the router as a product of its own, the down matrices one behind the other [E][d][ff]
         self.gathers = cfg.top < self.n_route and E > 0
         if self.gathers:
             # padded to be wide enough for the tensor-core tiles
-            self.router = FusedLinear(common + [(w[pre + "router"], None)], ops, device, pad_rows=64)
+            self.router = None if in_group else FusedLinear(common, ops, device, pad_rows=64)
             self.shared_down = FusedLinear([(w[pre + "shared.down"], None)], ops, device) if self.shared_ff else None
             self.down_each = torch.stack([w[f"{pre}e{e}.down"] for e in range(E)]).contiguous()
 
     @property
     def proj(self):
         return self.up
+
+    def state_spec(self):
+        return {"pages": [], "slots": []}
+
+    def _common(self, step, h, h16_ready):
+        """(address, row stride) of the common columns as a product of their own."""
+        logits = step.scratch("moe_logits", step.T * self.router.N)
+        self.router(step, h.data_ptr(), self.up.K, logits.data_ptr(), self.router.N, a16_ready=h16_ready)     # the bf16 rows left for the up product serve this one
+        return logits.data_ptr(), self.router.N
+
+    def _identity_rows(self, h):
+        return h if self.cfg.identity else None
 
     def _add_shared(self, step, first_ptr, ld, y):
         """y += the shared expert's result; its [gate | up] columns lie at ``first_ptr``."""
@@ -829,47 +1073,47 @@ class ExpertsFeedForward:
         n = self.shared_ff
         rows16 = self.shared_down.operand_rows(step)
         act = step.scratch("moe_shared", step.T * n)
-        self.ops.gated_act(first_ptr, ld, first_ptr + n * F32B, ld, None if rows16 is not None else act, n, step.T, n, step.st, out16=rows16)
+        out = None if rows16 is not None else act
+        if self.clamped:
+            self.ops.clamped_glu(first_ptr, ld, first_ptr + n * F32B, ld, self.cfg.shared_limit, self.clamped_alpha, out, n, step.T, n, step.st, out16=rows16)
+        else:
+            self.ops.gated_act(first_ptr, ld, first_ptr + n * F32B, ld, out, n, step.T, n, step.st, out16=rows16)
         self.shared_down(step, act.data_ptr(), n, y.data_ptr(), self.shared_down.N, accumulate=True, a16_ready=rows16 is not None)
 
-    def _forward_gathered(self, step, h, y, h16_ready=False):
+    def _gathers_rows16(self, step) -> bool:
+        """Whether the gathered form's products run on the tensor cores (else, in fp32 mode and for odd shapes, on FMA tiles)."""
+        d, ff, fu = self.up.K, self.cfg.ff, self.ff_up
+        return bool(step.engine.tensor_cores and self.ops.on_tensor_cores(step.T, fu, d) and self.ops.on_tensor_cores(step.T, d, ff) and (fu * d) % 8 == 0
+                    and (d * ff) % 8 == 0 and self.up.w.data_ptr() % 16 == 0 and self.down_each.data_ptr() % 16 == 0)
+
+    def _forward_gathered(self, step, h, y, common, ld, h16=None):
         c, ops, T, d, st = self.cfg, self.ops, step.T, self.up.K, step.st
         E, top, ff, cap, fu = c.experts, c.top, c.ff, step.T, self.ff_up
-        ldl = self.router.N
-        logits = step.scratch("moe_logits", T * ldl)
-        self.router(step, h.data_ptr(), d, logits.data_ptr(), ldl, a16_ready=h16_ready)     # the bf16 rows left for the up product serve this one
         # counts [E] | expert, row [T][top] each (int32) | score [T][top] | identity sum [T]
         book = step.scratch("moe_book", E + 3 * T * top + T).data_ptr()
         counts, sel_e, sel_pos, sel_w, ident = book, book + 4 * E, book + 4 * (E + T * top), book + 4 * (E + 2 * T * top), book + 4 * (E + 3 * T * top)
-        # operands of the tensor-core products are gathered as bf16 rows; shapes its tiles do not take (and the fp32 mode) gather fp32 rows
-        tc = (step.gemm_scratch(d, fu) is not None and ops.on_tensor_cores(cap, fu, d) and ops.on_tensor_cores(cap, d, ff)
-              and self.up.w.data_ptr() % 16 == 0 and self.down_each.data_ptr() % 16 == 0)
+        tc = self._gathers_rows16(step)
         per = 2 if tc else 1                       # operand elements per float of scratch
         rows = step.scratch("moe_rows", -(-E * cap * d // per)).data_ptr()
         up_out = step.scratch("moe_up", E * cap * fu).data_ptr()
         act = step.scratch("moe_act", -(-E * cap * ff // per)).data_ptr()
         down_out = step.scratch("moe_down", E * cap * d).data_ptr()
         ops.zero(counts, 4 * E, st)
-        scores = logits.data_ptr() + 2 * self.shared_ff * F32B         # the shared expert's columns come first
-        ops.moe_route(scores, ldl, self.n_route, E, top, self.correction, h, d, d, counts, cap, sel_e, sel_pos, sel_w, ident,
-                      rows if tc else None, None if tc else rows, T, st, mode=self.mode)
-        wb = self.up.w.element_size()
-        for e in range(E):
-            a = rows + e * cap * d * (2 if tc else 4)
-            ops.linear(a, d, self.up.w, d, None, up_out + 4 * e * cap * fu, fu, cap, fu, d, st, scratch=a if tc else None, a16_ready=tc, rows_dev=counts + 4 * e,
-                       w_ptr=self.up.w.data_ptr() + e * fu * d * wb)
-        ops.moe_expert_act(up_out, counts, E, cap, ff, self.mode, act if tc else None, None if tc else act, st)
-        for e in range(E):
-            a = act + e * cap * ff * (2 if tc else 4)
-            ops.linear(a, ff, self.down_each, ff, None, down_out + 4 * e * cap * d, d, cap, d, ff, st, scratch=a if tc else None, a16_ready=tc,
-                       rows_dev=counts + 4 * e, w_ptr=self.down_each.data_ptr() + e * d * ff * wb)
-        ops.moe_combine(down_out, sel_e, sel_pos, sel_w, top, ident, h, d, cap, d, y, d, T, st)
-        self._add_shared(step, logits.data_ptr(), ldl, y)
+        scores = common + 2 * self.shared_ff * F32B         # the shared expert's columns come first
+        copies = tc and h16 is not None and d % 8 == 0 and not self.scale_input
+        ops.moe_route(scores, ld, self.n_route, E, top, self.correction, None if copies else h, d, d, counts, cap, sel_e, sel_pos, sel_w, ident,
+                      rows if tc else None, None if tc else rows, T, st, mode=self.mode, h16=h16 if copies else None, opts=self.opts)
+        hint = max(1, T * top // self.n_route)
+        ops.linear_grouped(rows, tc, self.up.w, up_out, counts, E, cap, hint, fu, d, st)
+        ops.moe_expert_act(up_out, counts, E, cap, ff, self.mode, act if tc else None, None if tc else act, st, limit=c.limit)
+        ops.linear_grouped(act, tc, self.down_each, down_out, counts, E, cap, hint, d, ff, st)
+        ops.moe_combine(down_out, sel_e, sel_pos, sel_w, top, ident, self._identity_rows(h), d, cap, d, y, d, T, st)
+        self._add_shared(step, common, ld, y)
 
     def _gathered_pays(self, T: int) -> bool:
         c = self.cfg
         saved = 2.0 * T * (c.ff + self.ff_up) * self.up.K * (c.experts - min(c.top, c.experts)) / self.gather_product_rate
-        return self.gathers and T >= self.gather_min_tokens and saved > 2 * c.experts * self.gather_launch_cost
+        return self.gathers and T >= self.gather_min_tokens and saved > self.gather_launch_cost
 
     def _indexed_pays(self, T: int) -> bool:
         c = self.cfg
@@ -877,46 +1121,62 @@ class ExpertsFeedForward:
         saved = (c.experts - pairs) * float(c.ff + self.ff_up) * self.up.K * self.up.w.element_size() / self.index_stream_rate
         return self.gathers and T <= 8 and pairs < c.experts and saved > self.index_launch_cost
 
-    def _forward_indexed(self, step, h, y):
+    def _forward_indexed(self, step, h, y, common, ld):
         c, ops, T, d, st = self.cfg, self.ops, step.T, self.up.K, step.st
         E, top, ff, fu = c.experts, c.top, c.ff, self.ff_up
-        pairs, ldl = T * top, self.router.N
-        logits = step.scratch("moe_logits", T * ldl)
-        self.router(step, h.data_ptr(), d, logits.data_ptr(), ldl)
+        pairs = T * top
         book = step.scratch("moe_book", E + 3 * pairs + T).data_ptr()       # as in the gathered form; the counters stay unused
         sel_e, sel_pos, sel_w, ident = book + 4 * E, book + 4 * (E + pairs), book + 4 * (E + 2 * pairs), book + 4 * (E + 3 * pairs)
         # the products read the token's row as it is; a score on the expert's input is applied to their results (they are linear), so the
         # routing kernel is asked for the plain scores
-        scores = logits.data_ptr() + 2 * self.shared_ff * F32B         # the shared expert's columns come first
-        ops.moe_route(scores, ldl, self.n_route, E, top, self.correction, h, d, d, None, T, sel_e, sel_pos, sel_w, ident, None, None, T, st,
-                      mode=self.mode & ~self.SCALE_INPUT)
+        scores = common + 2 * self.shared_ff * F32B         # the shared expert's columns come first
+        ops.moe_route(scores, ld, self.n_route, E, top, self.correction, h, d, d, None, T, sel_e, sel_pos, sel_w, ident, None, None, T, st,
+                      mode=self.mode & ~self.SCALE_INPUT, opts=self.opts)
         up_out = step.scratch("moe_up", pairs * fu).data_ptr()
         down_out = step.scratch("moe_down", pairs * d).data_ptr()
         ops.linear_indexed(h.data_ptr(), d, d, top, self.up.w, d, fu * d, sel_e, up_out, fu, fu, pairs, fu, d, st)
         if self.gated or self.scale_input:
             act = step.scratch("moe_act", pairs * ff).data_ptr()
             weights = step.scratch("moe_pair_w", pairs).data_ptr()
-            ops.moe_pair_act(up_out, sel_w, pairs, ff, self.mode, act, weights, st)
+            ops.moe_pair_act(up_out, sel_w, pairs, ff, self.mode, act, weights, st, limit=c.limit)
         else:
             ops.act(up_out, pairs * ff, self.mode & 3, st)
             act, weights = up_out, sel_w
         ops.linear_indexed(act, ff, ff, 1, self.down_each, ff, d * ff, sel_e, down_out, d, d, pairs, d, ff, st)
         # row (t, k) of down_out is pair t * top + k: the combine kernel's (expert, row) address with buffers of 0 rows
-        ops.moe_combine(down_out, sel_e, sel_pos, weights, top, ident, h, d, 0, d, y, d, T, st)
-        self._add_shared(step, logits.data_ptr(), ldl, y)
+        ops.moe_combine(down_out, sel_e, sel_pos, weights, top, ident, self._identity_rows(h), d, 0, d, y, d, T, st)
+        self._add_shared(step, common, ld, y)
+
+    def _forward_wide(self, step, h, y, common, ld, h16_ready=False, h16=None):
+        """Every expert computed; ``common`` None: its columns are the last ones of the up product."""
+        c, T, d, N = self.cfg, step.T, self.up.K, self.up.N
+        z = step.scratch("ff_z", T * N)
+        self.up(step, h.data_ptr(), d, z.data_ptr(), N, a16_ready=h16_ready, a16=h16 if h16 is not None and self.up.takes_rows16(step) else None)
+        if common is None:
+            common, ld = z.data_ptr() + self.wide_up * F32B, N
+        rows16 = self.down.operand_rows(step)
+        act = step.scratch("ff_act", T * self.wide)   # fp32 rows; not written when the product reads the bf16 rows
+        self.ops.moe_act(common + 2 * self.shared_ff * F32B, ld, self.n_route, c.experts, c.top, self.correction, z.data_ptr(), N, c.ff, self.mode,
+                         h, d, d, None if rows16 is not None else act, rows16, y, d, T, step.st, shared_ptr=common if self.shared_ff else None, ld_shared=ld,
+                         shared_ff=self.shared_ff, opts=self.opts)
+        self.down(step, act.data_ptr(), self.wide, y.data_ptr(), d, accumulate=True, a16_ready=rows16 is not None)
 
     def forward(self, step, h, y, h16_ready=False):
         if self._gathered_pays(step.T):
-            return self._forward_gathered(step, h, y, h16_ready)
-        if self._indexed_pays(step.T):
-            return self._forward_indexed(step, h, y)
-        c, T, d, N = self.cfg, step.T, self.up.K, self.up.N
-        z = step.scratch("ff_z", T * N)
-        self.up(step, h.data_ptr(), d, z.data_ptr(), N, a16_ready=h16_ready)
-        rows16 = self.down.operand_rows(step)
-        act = step.scratch("ff_act", T * self.wide)   # fp32 rows; not written when the product reads the bf16 rows
-        common = z.data_ptr() + self.wide_up * F32B
-        self.ops.moe_act(common + 2 * self.shared_ff * F32B, N, self.n_route, c.experts, c.top, self.correction, z.data_ptr(), N, c.ff, self.mode,
-                         h, d, d, None if rows16 is not None else act, rows16, y, d, T, step.st, shared_ptr=common if self.shared_ff else None,
-                         shared_ff=self.shared_ff)
-        self.down(step, act.data_ptr(), self.wide, y.data_ptr(), d, accumulate=True, a16_ready=rows16 is not None)
+            self._forward_gathered(step, h, y, *self._common(step, h, h16_ready))
+        elif self._indexed_pays(step.T):
+            self._forward_indexed(step, h, y, *self._common(step, h, False))
+        else:
+            self._forward_wide(step, h, y, None, 0, h16_ready)
+
+    # ---- as a member of a MixerGroup ----
+    def reads_f32(self, step) -> bool:
+        return not (self._gathered_pays(step.T) and self._gathers_rows16(step) and self.up.K % 8 == 0 and not self.scale_input and not self.cfg.identity)
+
+    def run(self, step, cols, ld, h, h16, y):
+        if self._gathered_pays(step.T):
+            self._forward_gathered(step, h, y, cols[0], ld, h16)
+        elif self._indexed_pays(step.T):
+            self._forward_indexed(step, h, y, cols[0], ld)
+        else:
+            self._forward_wide(step, h, y, cols[0], ld, h16=h16)

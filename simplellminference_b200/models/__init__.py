@@ -6,11 +6,12 @@ from ..config import BF16, F32, read_model_config
 from .kodezen import KodezenModel
 from .lovulix import LovulixModel
 from .munazen import MunazenModel
+from .nelutar import NelutarModel
 from .sopetar import SopetarModel
 from .vasosun import VasosunModel
 
 MODEL_CLASSES = {"Munazen": MunazenModel, "Sopetar": SopetarModel, "Vasosun": VasosunModel, "Kodezen": KodezenModel,
-                 "Lovulix": LovulixModel}
+                 "Lovulix": LovulixModel, "Nelutar": NelutarModel}
 
 
 def build_model(model_dir: str, dtype: str = "bfloat16", device="cuda", build: bool = False):

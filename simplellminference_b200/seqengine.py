@@ -41,10 +41,40 @@ class Step:
         self.max_len = engine.max_len     # the most positions a request can hold
         self.sms = torch.cuda.get_device_properties(engine.device).multi_processor_count if engine.device.type == "cuda" else 1
         self.turned = set()       # frequency sets whose angles this step has already
+        self.branch = 0           # which of several mechanisms that run side by side is being enqueued (each has scratch of its own)
         self.prev_ids = None      # device array [T]: the token before each token in its sequence, -1 at a sequence's start
 
     def scratch(self, name: str, n_floats: int) -> torch.Tensor:
-        return self.engine._scratch(name, n_floats)
+        return self.engine._scratch(name if self.branch == 0 else (self.branch, name), n_floats)
+
+    def side_by_side(self, tasks) -> None:
+        """Enqueue independent pieces of work (callables that launch on ``self.st``): each on a stream of its own that starts after everything
+        enqueued so far and is waited for before anything enqueued later — in a captured step they become parallel branches of the graph.
+        A task may use any scratch it asks for here, but nothing another task writes."""
+        eng = self.engine
+        if len(tasks) == 1 or not eng.branch_streams:
+            for task in tasks:
+                task()
+            return
+        main, main_st = torch.cuda.current_stream(eng.device), self.st
+        start = torch.cuda.Event()
+        start.record(main)
+        joins = []
+        try:
+            for i, task in enumerate(tasks[1:], 1):
+                side = eng._side_stream(i)
+                side.wait_event(start)
+                self.branch, self.st = i, side.cuda_stream
+                task()
+                done = torch.cuda.Event()
+                done.record(side)
+                joins.append(done)
+            self.branch, self.st = 0, main_st
+            tasks[0]()
+        finally:
+            self.branch, self.st = 0, main_st
+            for done in joins:
+                main.wait_event(done)
 
     def angles(self, key: tuple, freq: torch.Tensor) -> torch.Tensor:
         """(cos, sin) of every token's position times every frequency of ``freq``, [T][n][2]: made by the step's first layer with these
@@ -52,6 +82,8 @@ class Step:
         n = len(key)
         table = self.engine._scratch(("angles", key), 2 * self.T * n)
         if key not in self.turned:
+            if self.branch:
+                raise RuntimeError("angles are made before mechanisms run side by side (prepare)")
             self.engine.ops.angles(self.b, freq, n, table, self.st)
             self.turned.add(key)
         return table
@@ -61,11 +93,12 @@ class Step:
         if not self.engine.tensor_cores or self.T < 64:
             return None
         n_bytes = ((self.T * K * 2 + 255) // 256) * 256 + self.T * N * 4
-        return self.engine._scratch("gemm", (n_bytes + 3) // 4)
+        return self.scratch("gemm", (n_bytes + 3) // 4)
 
 
 class SequenceEngine:
-    def __init__(self, model, max_tokens: int, max_seqs: int = 4, page_len: int = 64, tensor_cores: bool | None = None, graphs: bool = True):
+    def __init__(self, model, max_tokens: int, max_seqs: int = 4, page_len: int = 64, tensor_cores: bool | None = None, graphs: bool = True,
+                 branch_streams: bool = True):
         if page_len % KEY_TILE:
             raise ValueError(f"page_len must be a multiple of {KEY_TILE}")
         self.model, self.ops, self.device = model, model.ops, model.device
@@ -105,6 +138,9 @@ class SequenceEngine:
         # rows of logits are asked for (tokens, positions, slots and the block table are device memory), so it is captured once per such
         # pair as a CUDA graph and replayed. The first step of a kind runs directly (it sizes the scratch buffers), the second is captured.
         self.graphs = graphs and self.device.type == "cuda"
+        self.branch_streams = branch_streams and self.device.type == "cuda"     # mechanisms of a layer that run side by side: a stream each
+        self._sides = {}
+        self._retired = []      # scratch a larger one took the place of: other streams of the step may still use it
         self._graphs = {}
         self.graph_replays = 0
 
@@ -137,10 +173,17 @@ class SequenceEngine:
     def _scratch(self, name, n_floats: int) -> torch.Tensor:
         t = self._bufs.get(name)
         if t is None or t.numel() < n_floats:
+            if t is not None:
+                self._retired.append(t)
             t = torch.empty(max(n_floats, 1), dtype=torch.float32, device=self.device)
             self._bufs[name] = t
             self._graphs = {}          # captured steps hold the old address
         return t
+
+    def _side_stream(self, i: int):
+        if i not in self._sides:
+            self._sides[i] = torch.cuda.Stream(self.device)
+        return self._sides[i]
 
     def _upload(self, arrays):
         """The step's index arrays as ONE host-to-device copy; returns their device addresses."""
@@ -214,6 +257,7 @@ class SequenceEngine:
         step = self.step_obj
         step.T, step.nseg = T, nseg
         step.turned.clear()
+        self._retired.clear()       # the previous step's streams have met again
         b = step.b
         b.T, b.nseg = T, nseg
         b.tok_slot, b.tok_pos, b.seg_start, b.seg_len, b.seg_slot, b.seg_pos0 = p[1], p[2], p[3], p[4], p[5], p[6]

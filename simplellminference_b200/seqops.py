@@ -69,16 +69,29 @@ class Ops:
                                           self.round_a, batch, a_bs, w_bs, bias_bs, c_bs,
                                           (scratch if isinstance(scratch, int) else _p(scratch)) if self.tensor_cores else None, int(a16_ready), rows_dev, st))
 
+    def linear_grouped(self, a_ptr, a_bf16, w, c_ptr, counts_ptr, groups, cap, rows_hint, N, K, st):
+        """``groups`` products one behind the other in one launch, each over the rows its count (device memory) says are in use."""
+        self._ck(self.lib.sllm_seq_linear_grouped(a_ptr, int(bool(a_bf16)), _p(w), self.w_dtype, c_ptr, counts_ptr, groups, cap, rows_hint, N, K, st))
+
+    def branch_seam(self, x_in, x_out, branches, eps, norm_w, h, T, d, st, h16=None):
+        """x_out = x_in + sum of gain * y over ``branches`` [(y, gain, normed)], then (``norm_w``) the RMS norm of the sum -> h and / or h16."""
+        n = len(branches)
+        ys, gains, normed = (C.c_void_p * max(n, 1))(), (C.c_void_p * max(n, 1))(), (C.c_int32 * max(n, 1))()
+        for i, (y, gain, is_normed) in enumerate(branches):
+            ys[i], gains[i], normed[i] = _p(y), _p(gain), int(bool(is_normed))
+        self._ck(self.lib.sllm_seq_branch_seam(_p(x_in), _p(x_out), n, ys, gains, normed, eps, _p(norm_w), _p(h), _p(h16), T, d, st))
+
     def polynorm(self, z, ldz, coef, eps, out, ldo, T, n, st):
         self._ck(self.lib.sllm_seq_polynorm(_p(z), ldz, _p(coef), eps, _p(out), ldo, T, n, st))
 
     def gather_rows(self, x, ldx, rows, n, d, out, st):
         self._ck(self.lib.sllm_seq_gather_rows(_p(x), ldx, _p(rows), n, d, _p(out), st))
 
-    def headnorm_gate(self, o_ptr, ldo, g_ptr, ldg, w, heads, dv, eps, out, ldout, T, st, out16=None, gate_first=False, wide_weight=False):
-        """``gate_first``: the gate multiplies before the norm; ``wide_weight``: w holds heads * dv entries instead of dv."""
+    def headnorm_gate(self, o_ptr, ldo, g_ptr, ldg, w, heads, dv, eps, out, ldout, T, st, out16=None, gate_first=False, wide_weight=False, sigmoid_gate=False):
+        """``gate_first``: the gate multiplies before the norm; ``wide_weight``: w holds heads * dv entries instead of dv (None: no weight);
+        ``sigmoid_gate``: the gate is sigmoid(g) instead of silu(g)."""
         self._ck(self.lib.sllm_seq_headnorm_gate(o_ptr, ldo, g_ptr, ldg, _p(w), heads, dv, eps, _p(out), ldout, _p(out16), T,
-                                                 int(bool(gate_first)) | 2 * int(bool(wide_weight)), st))
+                                                 int(bool(gate_first)) | 2 * int(bool(wide_weight)) | 4 * int(bool(sigmoid_gate)), st))
 
     # ---- attention over the paged cache ----
     def rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, freq, n_freq, magnitude, vfreq, layout, k_pool, v_pool, st):
@@ -123,6 +136,12 @@ class Ops:
                                                          _p(angles), n_freq, layout, _p(v_shared), share, lam, _p(talk), _p(q_mixed), int(bool(k_joint)), _p(k_pool),
                                                          _p(v_pool), self.kv_dtype, st))
 
+    def conv_rotary_kv(self, b, q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, conv_w, taps, ring, angles, n_freq, layout, unit, eps, q_out, ldqo, k_pool,
+                       v_pool, st):
+        """``conv_w`` [taps][channels] or None; ``q_out``: address (the queries' own when there is no convolution)."""
+        self._ck(self.lib.sllm_seq_conv_rotary_kv(C.byref(b), q_ptr, ldq, heads, dk, k_ptr, ldk, kv_heads, v_ptr, ldv, dv, _p(conv_w), taps, _p(ring), _p(angles), n_freq,
+                                                  layout, int(bool(unit)), eps, q_out, ldqo, _p(k_pool), _p(v_pool), self.kv_dtype, st))
+
     def head_mix(self, x, ldx, mix, heads, kv_heads, dv, out, ldo, T, st, out16=None):
         self._ck(self.lib.sllm_seq_head_mix(_p(x), ldx, _p(mix), heads, kv_heads, dv, _p(out), ldo, _p(out16), T, st))
 
@@ -157,19 +176,23 @@ class Ops:
     def softcap(self, x, n, cap, st):
         self._ck(self.lib.sllm_seq_softcap(_p(x), n, cap, st))
 
+    @staticmethod
+    def moe_options(groups=0, keep=0, scale=1.0, limit=0.0, shared_limit=0.0):
+        return _lib.SeqMoeOpts(int(groups or 0), int(keep or 0), float(scale), float(limit or 0.0), float(shared_limit or 0.0))
+
     def moe_act(self, logits_ptr, ldl, n_route, experts, top, correction, up_ptr, ldu, ff, act, h, ldh, d, out, out16, y, ldy, T, st, route_w=None, shared_ptr=None,
-                shared_ff=0):
+                ld_shared=0, shared_ff=0, opts=None):
         self._ck(self.lib.sllm_seq_moe_act(logits_ptr, ldl, n_route, experts, top, _p(correction), up_ptr, ldu, ff, act, _p(h), ldh, d, _p(out), _p(out16),
-                                           _p(y), ldy, _p(route_w), shared_ptr, shared_ff, T, st))
+                                           _p(y), ldy, _p(route_w), shared_ptr, ld_shared, shared_ff, T, C.byref(opts) if opts is not None else None, st))
 
     # ---- mixture of experts with the tokens gathered per expert ----
     def zero(self, ptr, n_bytes, st):
         self._ck(self.lib.sllm_seq_zero(ptr, n_bytes, st))
 
     def moe_route(self, logits_ptr, ldl, n_route, experts, top, correction, h, ldh, d, counts_ptr, cap, sel_e, sel_pos, sel_w, ident, rows16, rows32, T, st,
-                  mode=0):
+                  mode=0, h16=None, opts=None):
         self._ck(self.lib.sllm_seq_moe_route(logits_ptr, ldl, n_route, experts, top, _p(correction), _p(h), ldh, d, counts_ptr, cap, sel_e, sel_pos, sel_w, ident,
-                                             rows16, rows32, T, mode, st))
+                                             rows16, rows32, T, mode, _p(h16), C.byref(opts) if opts is not None else None, st))
 
     def act(self, x_ptr, n, kind, st):
         self._ck(self.lib.sllm_seq_act(x_ptr, n, kind, st))
@@ -178,11 +201,11 @@ class Ops:
         """``batch`` products of one row each, product b with the matrix ``w_index[b]`` (device array) of ``w``."""
         self._ck(self.lib.sllm_seq_linear_indexed(a_ptr, lda, a_bs, a_div, _p(w), self.w_dtype, ldw, w_bs, w_index, c_ptr, ldc, c_bs, batch, N, K, self.round_a, st))
 
-    def moe_expert_act(self, up_ptr, counts_ptr, experts, cap, ff, act, out16, out32, st):
-        self._ck(self.lib.sllm_seq_moe_expert_act(up_ptr, counts_ptr, experts, cap, ff, act, out16, out32, st))
+    def moe_expert_act(self, up_ptr, counts_ptr, experts, cap, ff, act, out16, out32, st, limit=0.0):
+        self._ck(self.lib.sllm_seq_moe_expert_act(up_ptr, counts_ptr, experts, cap, ff, act, out16, out32, limit, st))
 
-    def moe_pair_act(self, up_ptr, sel_w_ptr, pairs, ff, act, out_ptr, w_out_ptr, st):
-        self._ck(self.lib.sllm_seq_moe_pair_act(up_ptr, sel_w_ptr, pairs, ff, act, out_ptr, w_out_ptr, st))
+    def moe_pair_act(self, up_ptr, sel_w_ptr, pairs, ff, act, out_ptr, w_out_ptr, st, limit=0.0):
+        self._ck(self.lib.sllm_seq_moe_pair_act(up_ptr, sel_w_ptr, pairs, ff, act, out_ptr, w_out_ptr, limit, st))
 
     def moe_combine(self, down_ptr, sel_e, sel_pos, sel_w, top, ident, h, ldh, cap, d, y, ldy, T, st):
         self._ck(self.lib.sllm_seq_moe_combine(down_ptr, sel_e, sel_pos, sel_w, top, ident, _p(h), ldh, cap, d, _p(y), ldy, T, st))
@@ -208,6 +231,16 @@ class Ops:
                    state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st):
         self._ck(self.lib.sllm_seq_delta_rule(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, _p(a_log), _p(dt_bias), heads,
                                               kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), st))
+
+    def channel_delta_rule(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, a_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale,
+                           state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st):
+        """As ``delta_rule`` with a step logit and a bias per head and key channel."""
+        self._ck(self.lib.sllm_seq_channel_delta_rule(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, _p(a_log), _p(dt_bias), heads,
+                                                      kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), st))
+
+    def decay_scan(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, decay, rate, angles, n_freq, layout, silu, kscale, heads, dk, dv, state, o, ldo, st, scratch=None):
+        self._ck(self.lib.sllm_seq_decay_scan(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, _p(decay), _p(rate), _p(angles), n_freq, layout, int(bool(silu)), kscale, heads,
+                                              dk, dv, _p(state), _p(o), ldo, _p(scratch), st))
 
     def conv(self, b, x_ptr, ldx, channels, taps, w, cb, tail, u, ldu, st):
         self._ck(self.lib.sllm_seq_conv(C.byref(b), x_ptr, ldx, channels, taps, _p(w), _p(cb), _p(tail), _p(u), ldu, st))
