@@ -82,6 +82,11 @@ def parse():
                          "over the heads before the softmax; gated experts beside a shared one) beside the closest model (Kodezen) at equal width and depth, and "
                          "the two designs' attention alone, at the sizes of simplellminference_b200/bench_lovulix.py (w1024,w2048,w4096) or 'all'. One GPU; prints "
                          "one JSON line {\"lovulix\": [...]}")
+    ap.add_argument("--nelutar", default=None, metavar="SIZES",
+                    help="instead of the headline workload: prefill and decode throughput of the Nelutar design (parallel layers; window attention beside the gated "
+                         "delta rule or lightning attention, retention; clamped experts with a grouped router) beside the closest model (Vasosun) at equal width and "
+                         "depth, and the designs' mechanisms alone, at the sizes of simplellminference_b200/bench_nelutar.py (w1024,w2048,w4096) or 'all'. One GPU; "
+                         "prints one JSON line {\"nelutar\": [...]}")
     ap.add_argument("--no-batch", action="store_true", help="(kept for old command lines: the secondary measurements are opt-in now, see --extras)")
     return ap.parse_args()
 
@@ -657,9 +662,12 @@ def main():
     real_stdout = os.dup(1)
     os.dup2(2, 1)
     sys.stdout = os.fdopen(real_stdout, "w", buffering=1)
-    if args.hybrid or args.sopetar or args.vasosun or args.kodezen or args.lovulix:
+    if args.hybrid or args.sopetar or args.vasosun or args.kodezen or args.lovulix or args.nelutar:
         import torch
-        if args.lovulix:
+        if args.nelutar:
+            from simplellminference_b200 import bench_nelutar as bench_hybrid
+            key, wanted = "nelutar", args.nelutar
+        elif args.lovulix:
             from simplellminference_b200 import bench_lovulix as bench_hybrid
             key, wanted = "lovulix", args.lovulix
         elif args.kodezen:

@@ -564,24 +564,30 @@ int sllm_seq_ring_store(const sllm_seq_batch* b, const float* x, int32_t ldx, in
 /* Gated delta rule per head h over each sequence, state [slots][heads][dk][dv] fp32: S <- g S; u = beta (v - S^T k); S <- S + k u^T;
  * o = S^T q, with q, k (of key head h / (heads / kv_heads)) divided by sqrt(sum(x^2) + unit_eps), q times qscale,
  * beta = sigmoid(beta_logit), g = exp(-exp(A_log[h]) * softplus(step_logit + dt_bias[h])). ring (or NULL): the last taps-1 rows of
- * conv_x [T][channels] of every portion are stored there for the convolution of the next step. */
+ * conv_x [T][channels] of every portion are stored there for the convolution of the next step. chunk_ws (NULL = token by token):
+ * sllm_seq_chunk_ws_bytes of scratch, 16-byte aligned; with it the portions are walked in blocks of 16 tokens on the tensor cores (dk <= 128;
+ * state and sums fp32, operands as two bf16 terms each). */
 int sllm_seq_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                         const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias,
                         int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o,
-                        int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, sllm_stream_t stream);
+                        int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, void* chunk_ws,
+                        sllm_stream_t stream);
+/* scratch of the block form of the recurrences (0: these sizes have none); n_qtiles as in the batch description */
+int64_t sllm_seq_chunk_ws_bytes(int32_t n_qtiles, int32_t heads, int32_t dk);
 /* The same rule with a decay per head and key channel: step_logit [T][heads * dk], dt_bias [heads * dk], S[c][:] <- g[c] S[c][:] with
  * g[c] = exp(-exp(A_log[h]) * softplus(step_logit[h * dk + c] + dt_bias[h * dk + c])); everything else as above. */
 int sllm_seq_channel_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                                 const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log,
                                 const float* dt_bias, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale,
                                 float* state, float* o, int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps,
-                                float* ring, sllm_stream_t stream);
+                                float* ring, void* chunk_ws, sllm_stream_t stream);
 /* Linear attention with a constant decay per head over each sequence, state [slots][heads][dk][dv] fp32: S <- decay[h] S + k v^T, o = S^T q.
  * rate[h] = -ln(decay[h]). silu 1: q, k and v pass silu first; angles (or NULL): (cos, sin) [T][n_freq] of sllm_seq_angles that turn q and k,
- * pairs by layout as in sllm_seq_rotary_kv; k is then multiplied by kscale. scratch as in sllm_seq_ssd_scan. */
+ * pairs by layout as in sllm_seq_rotary_kv; k is then multiplied by kscale. scratch as in sllm_seq_ssd_scan, chunk_ws as in sllm_seq_delta_rule. */
 int sllm_seq_decay_scan(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                         const float* decay, const float* rate, const float* angles, int32_t n_freq, int32_t layout, int32_t silu, float kscale,
-                        int32_t heads, int32_t dk, int32_t dv, float* state, float* o, int32_t ldo, float* scratch, sllm_stream_t stream);
+                        int32_t heads, int32_t dk, int32_t dv, float* state, float* o, int32_t ldo, float* scratch, void* chunk_ws,
+                        sllm_stream_t stream);
 /* State-space duality (Mamba-2) per head h over each sequence, state [slots][heads][n_state][dv] fp32: dt = softplus(step_logit + dt_bias[h]),
  * S <- exp(-exp(A_log[h]) dt) S + dt B x^T, y = S^T C + skip[h] x (skip NULL = no such term); x [T][heads * dv], B and C
  * [T][groups * n_state], head h reads group h / (heads / groups). The kernel of sllm_seq_delta_rule without its correction term; ring as there.

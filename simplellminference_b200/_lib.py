@@ -171,12 +171,13 @@ SIGNATURES.update({
     "sllm_seq_selective_scan": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _P, _P, _I, _P, _P, _I, _I, _P, _P, _P]),
     "sllm_seq_normed_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _I, _P]),
     "sllm_seq_head_mix": (C.c_int, [_P, _I, _P, _I, _I, _I, _P, _I, _P, _I, _P]),
-    "sllm_seq_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P]),
+    "sllm_seq_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P, _P]),
+    "sllm_seq_chunk_ws_bytes": (_L, [_I, _I, _I]),
     "sllm_seq_moe_act": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, C.POINTER(SeqMoeOpts), _P]),
     "sllm_seq_linear_grouped": (C.c_int, [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
     "sllm_seq_branch_seam": (C.c_int, [_P, _P, _I, C.POINTER(_P), C.POINTER(_P), C.POINTER(_I), _F, _P, _P, _P, _I, _I, _P]),
-    "sllm_seq_channel_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P]),
-    "sllm_seq_decay_scan": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P, _P, _I, _P, _P]),
+    "sllm_seq_channel_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P, _P]),
+    "sllm_seq_decay_scan": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _I, _I, _F, _I, _I, _I, _P, _P, _I, _P, _P, _P]),
     "sllm_seq_conv_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _I, _F, _P, _I, _P, _P, _I, _P]),
     "sllm_seq_layernorm": (C.c_int, [_P, _I, _P, _P, _F, _P, _I, _P, _I, _I, _P]),
     "sllm_seq_depth_average": (C.c_int, [_P, _P, _P, _I, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
@@ -188,7 +189,7 @@ SIGNATURES.update({
 })
 
 # The ragged-token-batch part of the library can be built and loaded on its own (`make -C csrc seq` -> libsllm_b200_seq.so: the
-# sllm_seq_* kernels, the tensor-core GEMM, the page bookkeeping, the sampler): a model made of those blocks then needs fourteen
+# sllm_seq_* kernels, the tensor-core GEMM, the page bookkeeping, the sampler): a model made of those blocks then needs fifteen
 # translation units compiled, not all of them. The full library contains the same objects and is preferred when it exists.
 SEQ_LIB_PATH = os.path.join(HERE, "lib", "libsllm_b200_seq.so")
 SEQ_SYMBOL_PREFIXES = ("sllm_seq_", "sllm_kvpages_", "sllm_sample_", "sllm_last_error", "sllm_abi_version", "sllm_tune", "sllm_device_info",

@@ -16,11 +16,13 @@
 // whose queries and keys may be rotated by their position and scaled (retention) and whose q, k and v may pass silu (lightning attention)
 // as they arrive in shared memory.
 //
+// Portions of prompts in bf16 mode take the block form of seq_chunk.cu instead (a caller that hands over its scratch asks for it).
+//
 // The convolution keeps its last taps-1 inputs per sequence in a ring (position p at row p % (taps-1)); the recurrence kernel, which
 // runs after the convolution has read the ring, stores the portion's last inputs there.
 #include <cstdlib>
 
-#include "seq_common.cuh"
+#include "seq_chunk.cuh"
 
 namespace sllm {
 
@@ -372,6 +374,7 @@ struct DeltaExtra {
     bool channel = false;                                // the decay's step logits are [heads * dk] per token, dt_bias [heads * dk]
     const float *decay = nullptr, *rate = nullptr;       // constant decay per head
     const float* angles = nullptr; int n_freq = 0, layout = 0, silu = 0;
+    void* chunk_ws = nullptr;                            // walk the portions in blocks of tokens (seq_chunk.cu)
 };
 
 // all recurrences: `ssd` = no correction by the old state (skip [heads] or NULL)
@@ -384,6 +387,12 @@ static int delta_run(bool ssd, const float* skip, const DeltaExtra& ex, const sl
                  "seq_delta_rule / seq_ssd_scan / seq_decay_scan: bad argument");
     SLLM_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0, SLLM_EINVAL, "seq_delta_rule: %d heads over %d key heads", heads, kv_heads);
     SLLM_REQUIRE(!ring || (conv_x && channels > 0 && taps >= 1), SLLM_EINVAL, "seq_delta_rule: the ring needs the convolution's inputs");
+    if (ex.chunk_ws) {
+        ChunkArgs c{*b, q, k, v, ldq, ldk, ldv, !ssd, beta_logit, step_logit, ldb, lda, A_log, dt_bias, ex.channel, ex.rate, (const float2*)ex.angles, ex.n_freq, ex.layout,
+                    ex.silu, heads, kv_heads, dk, dv, unit_eps, qscale, state, o, ldo, (uint8_t*)ex.chunk_ws};
+        if (int rc = launch_chunk_scan(c, as_stream(stream))) return rc;
+        return ring && taps > 1 ? sllm_seq_ring_store(b, conv_x, ldx, channels, taps, ring, stream) : SLLM_OK;
+    }
     static const int tune_kp = getenv("SLLM_DELTA_KP") ? atoi(getenv("SLLM_DELTA_KP")) : 0;      // measurement aids: 8 / 16 / 32 channels per thread,
     static const int tune_cb = getenv("SLLM_DELTA_CB") ? atoi(getenv("SLLM_DELTA_CB")) : 0;      // columns per CTA
     int KP = dk <= 512 ? 16 : 32;
@@ -462,8 +471,10 @@ extern "C" {
 int sllm_seq_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv, const float* beta_logit,
                         int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias, int32_t heads, int32_t kv_heads,
                         int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o, int32_t ldo, const float* conv_x, int32_t ldx,
-                        int32_t channels, int32_t taps, float* ring, sllm_stream_t stream) {
-    return delta_run(false, nullptr, DeltaExtra{}, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
+                        int32_t channels, int32_t taps, float* ring, void* chunk_ws, sllm_stream_t stream) {
+    DeltaExtra ex;
+    ex.chunk_ws = chunk_ws;
+    return delta_run(false, nullptr, ex, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
                      o, ldo, conv_x, ldx, channels, taps, ring, nullptr, stream);
 }
 
@@ -478,19 +489,20 @@ int sllm_seq_ssd_scan(const sllm_seq_batch* b, const float* x, int32_t ldx, cons
 int sllm_seq_channel_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,
                                 const float* beta_logit, int32_t ldb, const float* step_logit, int32_t lda, const float* A_log, const float* dt_bias,
                                 int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float unit_eps, float qscale, float* state, float* o, int32_t ldo,
-                                const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, sllm_stream_t stream) {
+                                const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, void* chunk_ws, sllm_stream_t stream) {
     DeltaExtra ex;
     ex.channel = true;
+    ex.chunk_ws = chunk_ws;
     return delta_run(false, nullptr, ex, b, q, ldq, k, ldk, v, ldv, beta_logit, ldb, step_logit, lda, A_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale, state,
                      o, ldo, conv_x, ldx, channels, taps, ring, nullptr, stream);
 }
 
 int sllm_seq_decay_scan(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv, const float* decay,
                         const float* rate, const float* angles, int32_t n_freq, int32_t layout, int32_t silu, float kscale, int32_t heads, int32_t dk, int32_t dv,
-                        float* state, float* o, int32_t ldo, float* scratch, sllm_stream_t stream) {
+                        float* state, float* o, int32_t ldo, float* scratch, void* chunk_ws, sllm_stream_t stream) {
     SLLM_REQUIRE(decay && rate && n_freq >= 0 && 2 * n_freq <= dk && (n_freq == 0 || angles) && (layout == 0 || layout == 1), SLLM_EINVAL, "seq_decay_scan: bad argument");
     DeltaExtra ex;
-    ex.decay = decay; ex.rate = rate; ex.angles = angles; ex.n_freq = n_freq; ex.layout = layout; ex.silu = silu;
+    ex.decay = decay; ex.rate = rate; ex.angles = angles; ex.n_freq = n_freq; ex.layout = layout; ex.silu = silu; ex.chunk_ws = chunk_ws;
     return delta_run(true, nullptr, ex, b, q, ldq, k, ldk, v, ldv, nullptr, 0, nullptr, 0, nullptr, nullptr, heads, heads, dk, dv, 0.0f, kscale, state, o, ldo, nullptr, 0, 0,
                      0, nullptr, scratch, stream);
 }

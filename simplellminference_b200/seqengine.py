@@ -30,6 +30,8 @@ KEY_TILE = 32
 class Step:
     """What the mechanisms see of one step: sizes, the batch description, the stream, scratch memory."""
 
+    chunk_min_tokens = 16      # portions shorter than this are walked token by token
+
     def __init__(self, engine):
         # no strong reference back: an engine must die with its last user (by reference count), not whenever the cycle collector runs —
         # its captured graphs free device memory when they go, and that is not allowed while another engine is capturing a step
@@ -87,6 +89,14 @@ class Step:
             self.engine.ops.angles(self.b, freq, n, table, self.st)
             self.turned.add(key)
         return table
+
+    def chunk_scratch(self, heads: int, dk: int):
+        """Scratch with which the recurrences walk this step's portions in blocks of tokens on the tensor cores, or None: the all-fp32 mode, steps
+        without a portion worth a block, key heads the form does not take."""
+        if not self.engine.tensor_cores or self.T - self.nseg + 1 < self.chunk_min_tokens:
+            return None
+        n = self.engine.ops.chunk_ws_floats(self.b.n_qtiles, heads, dk)
+        return self.scratch("chunk_blocks", n) if n else None
 
     def gemm_scratch(self, K: int, N: int):
         """bf16 copy of the activations + the plain product, for products that go to the tensor cores (None: too few rows to pay)."""

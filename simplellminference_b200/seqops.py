@@ -228,19 +228,25 @@ class Ops:
                                                   _p(state), _p(out), ldo, _p(out16), conv_x_ptr, ld_conv, taps, _p(ring), _p(scratch), st))
 
     def delta_rule(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, a_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale,
-                   state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st):
+                   state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st, chunk_ws=None):
+        """``chunk_ws``: scratch of ``chunk_ws_floats``: portions are walked in blocks of tokens on the tensor cores."""
         self._ck(self.lib.sllm_seq_delta_rule(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, _p(a_log), _p(dt_bias), heads,
-                                              kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), st))
+                                              kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), _p(chunk_ws), st))
+
+    def chunk_ws_floats(self, n_qtiles, heads, dk):
+        """Floats of scratch of the block form of the recurrences, 0 when these sizes have none."""
+        return (self.lib.sllm_seq_chunk_ws_bytes(n_qtiles, heads, dk) + 3) // 4
 
     def channel_delta_rule(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, a_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale,
-                           state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st):
+                           state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st, chunk_ws=None):
         """As ``delta_rule`` with a step logit and a bias per head and key channel."""
         self._ck(self.lib.sllm_seq_channel_delta_rule(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, _p(a_log), _p(dt_bias), heads,
-                                                      kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), st))
+                                                      kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), _p(chunk_ws), st))
 
-    def decay_scan(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, decay, rate, angles, n_freq, layout, silu, kscale, heads, dk, dv, state, o, ldo, st, scratch=None):
+    def decay_scan(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, decay, rate, angles, n_freq, layout, silu, kscale, heads, dk, dv, state, o, ldo, st, scratch=None,
+                   chunk_ws=None):
         self._ck(self.lib.sllm_seq_decay_scan(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, _p(decay), _p(rate), _p(angles), n_freq, layout, int(bool(silu)), kscale, heads,
-                                              dk, dv, _p(state), _p(o), ldo, _p(scratch), st))
+                                              dk, dv, _p(state), _p(o), ldo, _p(scratch), _p(chunk_ws), st))
 
     def conv(self, b, x_ptr, ldx, channels, taps, w, cb, tail, u, ldu, st):
         self._ck(self.lib.sllm_seq_conv(C.byref(b), x_ptr, ldx, channels, taps, _p(w), _p(cb), _p(tail), _p(u), ldu, st))

@@ -189,6 +189,92 @@ def test_recurrences_over_long_portions_beside_short_ones(dtype):
             assert _rel(np.concatenate(got), want) < tol, (kind, kw, _rel(np.concatenate(got), want))
 
 
+def _scan_stub(kind, H, G, dk, dv, consts, blocks):
+    """Columns [q | k | v | beta logits | step logits] straight into the recurrence kernels, in blocks of tokens or token by token."""
+    import torch
+
+    from simplellminference_b200.config import BF16, RotaryConfig
+    from simplellminference_b200.layers import rotary_frequencies
+    from simplellminference_b200.seqops import Ops
+    dev, ops = torch.device("cuda"), Ops(BF16)
+    t = lambda a: torch.tensor(np.asarray(a), dtype=torch.float32, device=dev)   # noqa: E731
+    steps = {"channel": H * dk, "head": H}.get(kind, 0)
+    sizes = [G * dk, G * dk, H * dv, H if steps else 0, steps]
+    offs, width = [4 * sum(sizes[:i]) for i in range(5)], sum(sizes)
+    c = {k: t(v) for k, v in consts.items()}
+    key, freq = rotary_frequencies(RotaryConfig(dk // 4 * 2, 50.0), dev) if kind == "retention" and dk >= 4 else ((), None)
+
+    def fn(step, h, states):
+        base, S = h.data_ptr(), states[0]["S"]
+        q, k, v, bl, al = (base + o for o in offs)
+        out = torch.empty(step.T, H * dv, device=dev)
+        ws = step.chunk_scratch(H, dk) if blocks else None
+        assert (ws is not None) == (blocks and step.T - step.nseg + 1 >= step.chunk_min_tokens)
+        if steps:
+            rule = ops.channel_delta_rule if kind == "channel" else ops.delta_rule
+            rule(step.b, q, width, k, width, v, width, bl, width, al, width, c["A_log"], c["dt_bias"], H, G, dk, dv, 1e-6, dk ** -0.5, S, out, H * dv, None, 0, 0, 0, None,
+                 step.st, chunk_ws=ws)
+        else:
+            ops.decay_scan(step.b, q, width, k, width, v, width, c["decay"], c["rate"], step.angles(key, freq) if key else None, len(key), 1, kind == "lightning",
+                           dk ** -0.5 if kind == "retention" else 1.0, H, dk, dv, S, out, H * dv, step.st, chunk_ws=ws)
+        return [out]
+    rot = {"dims": len(key) * 2, "base": 50.0}
+    return L.Stub([{"pages": [], "slots": [("S", (H, dk, dv))]}], fn, ops, dev), sizes, rot
+
+
+def _scan_oracle(kind, x, sizes, H, G, dk, dv, consts, rot):
+    n = x.shape[0]
+    q, k, v, bl, al = np.split(x.astype(np.float64), np.cumsum(sizes)[:-1], axis=1)
+    q, k, v = q.reshape(n, G, dk), k.reshape(n, G, dk), v.reshape(n, H, dv)
+    out = np.zeros((n, H, dv))
+    if kind in ("channel", "head"):
+        q, k, beta = O.unit_vectors(q) * dk ** -0.5, O.unit_vectors(k), O.sigmoid(bl)
+        step = O.softplus(al + consts["dt_bias"]).reshape(n, H, -1)
+        g = np.broadcast_to(np.exp(-np.exp(np.asarray(consts["A_log"], np.float64))[None, :, None] * step), (n, H, dk))
+        for h in range(H):
+            out[:, h] = O.channel_delta_rule(q[:, h * G // H], k[:, h * G // H], v[:, h], beta[:, h], g[:, h])
+        return out.reshape(n, H * dv)
+    if kind == "lightning":
+        q, k, v = O.silu(q), O.silu(k), O.silu(v)
+    else:
+        q, k = O.rotate(q, rot, False), O.rotate(k, rot, False) * dk ** -0.5
+    for h in range(H):
+        out[:, h] = O.decayed_attention(q[:, h], k[:, h], v[:, h], consts["decay64"][h])
+    return out.reshape(n, H * dv)
+
+
+def test_recurrences_in_blocks_of_tokens_keep_fp32_accuracy():
+    """The block form of the recurrences (tensor cores, operands as two bf16 terms) and the form that walks token by token, both against the
+    restatement on the same fp32 inputs: weak and strong decays (a channel that forgets everything within a token), step sizes near one,
+    keys that repeat, one head and shared key heads, widths that are multiples of nothing, portions that end inside a block, a state that is
+    carried from portion to portion and into single tokens."""
+    rng = np.random.default_rng(51)
+    cases = [("channel", 2, 1, 128, 128), ("channel", 3, 3, 64, 40), ("channel", 1, 1, 1, 1), ("channel", 4, 2, 33, 130), ("channel", 2, 2, 100, 5), ("head", 4, 2, 128, 64),
+             ("head", 3, 1, 20, 70), ("retention", 2, 2, 128, 128), ("retention", 3, 3, 6, 33), ("retention", 1, 1, 70, 200), ("lightning", 2, 2, 64, 64), ("lightning", 3, 3, 97, 3)]
+    for kind, H, G, dk, dv in cases:
+        for flavour in ("weak", "mixed", "strong"):
+            n = 150
+            decay = {"weak": 1.0 - 10.0 ** -np.linspace(3, 5, H), "mixed": np.linspace(0.3, 0.999, H), "strong": np.linspace(1e-4, 0.2, H)}[flavour]
+            consts = {"A_log": rng.uniform(*{"weak": (-9, -6), "mixed": (-3, 1), "strong": (1, 4)}[flavour], size=H).astype(np.float32), "decay": decay.astype(np.float32),
+                      "rate": -np.log(decay), "decay64": decay.astype(np.float32).astype(np.float64),
+                      "dt_bias": rng.uniform(-3, 3, size=H * dk if kind == "channel" else H).astype(np.float32)}
+            consts["rate"] = (-np.log(consts["decay64"])).astype(np.float32)
+            results = []
+            for blocks in (True, False):
+                stub, sizes, rot = _scan_stub(kind, H, G, dk, dv, consts, blocks)
+                if not results:
+                    x = rng.standard_normal((n, sum(sizes))).astype(np.float32)
+                    if sizes[3]:
+                        x[:, sum(sizes[:3]):sum(sizes[:4])] += 3.0          # step sizes near one
+                        x[20:60, sizes[0]:2 * sizes[0]] = x[19, sizes[0]:2 * sizes[0]] + 0.05 * x[20:60, sizes[0]:2 * sizes[0]]   # keys that nearly repeat
+                    want = _scan_oracle(kind, x, sizes, H, G, dk, dv, consts, rot)
+                for portions in ([n], [37, 16, 1, 40, 2, 54], [100] + [1] * 50):
+                    got = L.feed(stub, x, portions)[0]
+                    assert _rel(got, want) < 5e-5, (kind, H, dk, dv, flavour, blocks, portions[:3], _rel(got, want))
+                    results.append(_rel(got, want))
+            print(kind, H, G, dk, dv, flavour, ["%.1e" % r for r in results])
+
+
 def test_state_and_rings_of_a_slot_used_again():
     """A slot that carried one sequence's state and convolution inputs serves another: its first tokens see zeros, not the old state."""
     from simplellminference_b200.seqengine import SequenceEngine
