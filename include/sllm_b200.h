@@ -485,6 +485,11 @@ typedef struct {
 int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv,
                        float scale, const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws,
                        const sllm_seq_attn_opts* opts, sllm_stream_t stream);
+/* sllm_seq_attention and the merge of its shares in one call (no gate, no sink, no turned values): the result as fp32 [T][ldo] (out) and / or dense
+ * bf16 [T][heads * dv] (out16). With one share the tensor-core body writes it itself. */
+int sllm_seq_attention_out(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv,
+                           float scale, const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws,
+                           const sllm_seq_attn_opts* opts, float* out, int32_t ldo, void* out16, sllm_stream_t stream);
 /* Merges the shares, normalises (sink [heads] or NULL: the denominator of head h also holds exp(sink[h]), a term without key or value),
  * turns every head's output back by -pos * vfreq[m] (vfreq NULL = not), multiplies head h by sigmoid(gate[t][h]), or with gate_channels
  * column c of head h by sigmoid(gate[t][h*dv + c]) (gate NULL = not), and stores out[t][h*dv ..] and / or out16, dense bf16 rows. */

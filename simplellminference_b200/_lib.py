@@ -153,6 +153,7 @@ SIGNATURES.update({
     "sllm_seq_gather_rows": (C.c_int, [_P, _I, _P, _I, _I, _P, _P]),
     "sllm_seq_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _I, _F, _P, _I, _P, _P, _I, _P]),
     "sllm_seq_attention": (C.c_int, [_B, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I, _P, C.POINTER(SeqAttnOpts), _P]),
+    "sllm_seq_attention_out": (C.c_int, [_B, _P, _I, _I, _I, _I, _I, _F, _P, _P, _I, _I, _P, C.POINTER(SeqAttnOpts), _P, _I, _P, _P]),
     "sllm_seq_attention_finish": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _P, _I, _I, _P, _P, _I, _P, _P]),
     "sllm_seq_attention_talk": (C.c_int, [_B, _P, _I, _P, _I, _I, _I, _I, _F, _P, _P, _P, _I, _I, _P, C.POINTER(SeqAttnOpts), _P, _I, _P, _P, _I, _P, _P]),
     "sllm_seq_attention_talk_takes_mixed": (C.c_int, [_I, _I, _I, _I, _I]),

@@ -35,6 +35,7 @@ struct AttnArgs {
     // head u / q_heads, query head u % q_heads); the query head reads the KEYS of its own key/value head as always. Otherwise q_heads = heads.
     int q_heads, cross;
     int chunk;                // > 0: a query sees its own chunk of `chunk` positions only (then window / keep_first are not used)
+    float* out; int ldo; uint16_t* out16;   // tensor-core body, one share: the normalised result goes here (fp32 [T][ldo] and / or dense bf16) instead of ws
 };
 
 __device__ __forceinline__ float seq_score(float dot, float scale, float softcap, float slope, float r1, float r2, int qpos, int key) {
@@ -370,6 +371,22 @@ __global__ void __launch_bounds__(128) seq_attention_mma_kernel(AttnArgs p) {
     for (int half = 0; half < 2; ++half) {
         const int r = half ? r1 : r0;
         if (r >= nq) continue;
+        if (p.out || p.out16) {                        // the only share: nothing to merge
+            const float inv = 1.0f / (half ? l1 : l0);
+#pragma unroll
+            for (int nt = 0; nt < kMmaDvTiles; ++nt) {
+                if (nt < dvt) {
+                    const float a = o[nt][2 * half] * inv, bb = o[nt][2 * half + 1] * inv;
+                    const size_t col = (size_t)h * dv + nt * 8 + 2 * c;
+                    if (p.out16) *reinterpret_cast<uint32_t*>(p.out16 + (size_t)(t0 + r) * p.heads * dv + col) = pack_bf16(a, bb);
+                    if (p.out) {
+                        p.out[(size_t)(t0 + r) * p.ldo + col] = a;
+                        p.out[(size_t)(t0 + r) * p.ldo + col + 1] = bb;
+                    }
+                }
+            }
+            continue;
+        }
         float* rec = p.ws + (((size_t)(t0 + r) * p.heads + h) * p.nsplit + split) * (dv + 2);
         if (c == 0) {
             rec[0] = half ? m1 : m0;
@@ -558,9 +575,13 @@ int sllm_seq_rotary_kv(const sllm_seq_batch* b, float* q, int32_t ldq, int32_t h
     return SLLM_OK;
 }
 
-int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float scale,
-                       const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws, const sllm_seq_attn_opts* opts,
-                       sllm_stream_t stream) {
+}  // extern "C"
+
+// out / out16 given: the merged result goes there; *merged says whether this launch has written it (else the shares wait in ws)
+static int attention_run(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float scale, const void* k_pool,
+                         const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws, const sllm_seq_attn_opts* opts, float* out, int32_t ldo, uint16_t* out16,
+                         bool* merged, sllm_stream_t stream) {
+    *merged = false;
     if (int rc = check_batch(b, "seq_attention")) return rc;
     const int v_in_k = opts && opts->values_in_keys;
     SLLM_REQUIRE(q && k_pool && (v_pool || v_in_k) && ws && b->block_table && b->qt_seg && b->qt_off && b->n_qtiles > 0, SLLM_EINVAL, "seq_attention: bad argument");
@@ -575,7 +596,7 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
     const int dkp = ((dk + 3) & ~3) + 4;
     const size_t smem = ((size_t)(kBQ + kBK) * dkp + (v_in_k ? 0 : (size_t)kBK * dv)) * sizeof(float);
     SLLM_REQUIRE(smem <= (size_t)smem_optin_bytes(), SLLM_ENOTSUP, "seq_attention: heads of %d + %d floats need %zu bytes of shared memory", dk, dv, smem);
-    AttnArgs p{*b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, nsplit, ws, 0, INT_MAX, 0, 0.0f, nullptr, 0, nullptr, heads, 0, 0};
+    AttnArgs p{*b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, nsplit, ws, 0, INT_MAX, 0, 0.0f, nullptr, 0, nullptr, heads, 0, 0, nullptr, 0, nullptr};
     if (opts && opts->cross_values) {
         SLLM_REQUIRE(!v_in_k, SLLM_EINVAL, "seq_attention: values of every head need a value pool");
         p.cross = 1;
@@ -598,6 +619,10 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
         grid.y = p.heads / hpc;
         const dim3 block(64 * hpc);
         cudaStream_t st = as_stream(stream);
+        if (nsplit == 1 && !p.cross && (out || out16)) {
+            p.out = out; p.ldo = ldo; p.out16 = out16;
+            *merged = true;
+        }
         if (dk == 128 && dv == 128) seq_attention_mma_kernel<8, 16, true><<<grid, block, smem_mma, st>>>(p);
         else if (dk == 192 && dv == 128) seq_attention_mma_kernel<12, 16, true><<<grid, block, smem_mma, st>>>(p);
         else if (dk == 64 && dv == 64) seq_attention_mma_kernel<4, 8, true><<<grid, block, smem_mma, st>>>(p);
@@ -626,6 +651,25 @@ int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     return SLLM_OK;
+}
+
+extern "C" {
+
+int sllm_seq_attention(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float scale,
+                       const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws, const sllm_seq_attn_opts* opts,
+                       sllm_stream_t stream) {
+    bool merged;
+    return attention_run(b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, kv_dtype, nsplit, ws, opts, nullptr, 0, nullptr, &merged, stream);
+}
+
+int sllm_seq_attention_out(const sllm_seq_batch* b, const float* q, int32_t ldq, int32_t heads, int32_t kv_heads, int32_t dk, int32_t dv, float scale,
+                           const void* k_pool, const void* v_pool, int32_t kv_dtype, int32_t nsplit, float* ws, const sllm_seq_attn_opts* opts, float* out,
+                           int32_t ldo, void* out16, sllm_stream_t stream) {
+    SLLM_REQUIRE((out || out16) && !(opts && opts->cross_values), SLLM_EINVAL, "seq_attention_out: no output, or values of every head (they are merged by their own call)");
+    bool merged;
+    if (int rc = attention_run(b, q, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, kv_dtype, nsplit, ws, opts, out, ldo, (uint16_t*)out16, &merged, stream)) return rc;
+    return merged ? SLLM_OK
+                  : launch_attention_finish(b, ws, nsplit, heads, dv, nullptr, 0, nullptr, 0, 0, nullptr, out, ldo, (uint16_t*)out16, as_stream(stream));
 }
 
 int sllm_seq_attention_finish(const sllm_seq_batch* b, const float* ws, int32_t nsplit, int32_t heads, int32_t dv, const double* vfreq, int32_t layout,

@@ -206,11 +206,11 @@ __global__ void __launch_bounds__(kPrepThreads) seq_chunk_prepare_kernel(ChunkAr
     }
 }
 
-// three products of two-term operands: d += (ah + al) (bh + bl) without al * bl; the small terms go to an accumulator of their own
-__device__ __forceinline__ void mma_split(float (&d)[4], float (&dl)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t h0, uint32_t h1, uint32_t l0, uint32_t l1) {
+// three products of two-term operands: (ah + al) (bh + bl) without al * bl, each into an accumulator of its own (no product waits for another)
+__device__ __forceinline__ void mma_split(float (&d)[4], float (&dl)[4], float (&dm)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t h0, uint32_t h1, uint32_t l0, uint32_t l1) {
     mma_bf16_16816(d, ah, h0, h1);
     mma_bf16_16816(dl, al, h0, h1);
-    mma_bf16_16816(dl, ah, l0, l1);
+    mma_bf16_16816(dm, ah, l0, l1);
 }
 
 // KS: k-steps of 16 key channels
@@ -280,7 +280,7 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
         const float* sv = reinterpret_cast<const float*>(rec + rec_bytes);
         const int n = min(kChunk, len - blk * kChunk);
         if (col0 + warp * 16 < p.dv) {                   // the same answer in every lane of the warp
-        float x[2][4] = {}, xl[2][4] = {}, o[2][4] = {}, ol[2][4] = {};     // rows r0 / r1, columns (tokens) nt * 8 + 2c, + 1
+        float x[2][4] = {}, xl[2][4] = {}, xm[2][4] = {}, o[2][4] = {}, ol[2][4] = {}, om[2][4] = {};     // rows r0 / r1, columns (tokens) nt * 8 + 2c, + 1
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
             uint32_t ah[4], al[4];
@@ -290,12 +290,12 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
             split_bf16(S[2 * ks + 1][2], S[2 * ks + 1][3], &ah[3], &al[3]);
             if (kDelta) {
                 const uint4 kh = Kh[ks * 32], kl = Kl[ks * 32];
-                mma_split(x[0], xl[0], ah, al, kh.x, kh.y, kl.x, kl.y);
-                mma_split(x[1], xl[1], ah, al, kh.z, kh.w, kl.z, kl.w);
+                mma_split(x[0], xl[0], xm[0], ah, al, kh.x, kh.y, kl.x, kl.y);
+                mma_split(x[1], xl[1], xm[1], ah, al, kh.z, kh.w, kl.z, kl.w);
             }
             const uint4 qh = Qh[ks * 32], ql = Ql[ks * 32];
-            mma_split(o[0], ol[0], ah, al, qh.x, qh.y, ql.x, ql.y);
-            mma_split(o[1], ol[1], ah, al, qh.z, qh.w, ql.z, ql.w);
+            mma_split(o[0], ol[0], om[0], ah, al, qh.x, qh.y, ql.x, ql.y);
+            mma_split(o[1], ol[1], om[1], ah, al, qh.z, qh.w, ql.z, ql.w);
         }
 #pragma unroll
         for (int nt = 0; nt < 2 * KS; ++nt) {            // the old state decays to the block's end
@@ -311,7 +311,7 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
             for (int e = 0; e < 4; ++e) {
                 float v = sv[(nt * 8 + 2 * c + (e & 1)) * kWalkCols + cl + (e < 2 ? 0 : 8)];
                 if (!kDelta && p.silu) v = v * seq_sigmoid(v);
-                x[nt][e] = v - (x[nt][e] + xl[nt][e]);
+                x[nt][e] = v - (x[nt][e] + (xl[nt][e] + xm[nt][e]));
             }
         uint32_t uh[4], ul[4];
         auto operand = [&](const float (&y)[2][4]) {     // rows x 16 tokens as an A fragment
@@ -322,19 +322,19 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
         };
         operand(x);
         if (kDelta) {
-            float u[2][4] = {}, lo[2][4] = {};
+            float u[2][4] = {}, lo[2][4] = {}, mid[2][4] = {};
             const uint4 mh = Mh[0], ml = Mh[32];
-            mma_split(u[0], lo[0], uh, ul, mh.x, mh.y, ml.x, ml.y);
-            mma_split(u[1], lo[1], uh, ul, mh.z, mh.w, ml.z, ml.w);
+            mma_split(u[0], lo[0], mid[0], uh, ul, mh.x, mh.y, ml.x, ml.y);
+            mma_split(u[1], lo[1], mid[1], uh, ul, mh.z, mh.w, ml.z, ml.w);
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) u[nt][e] += lo[nt][e];
+                for (int e = 0; e < 4; ++e) u[nt][e] += lo[nt][e] + mid[nt][e];
             operand(u);
         }
         const uint4 bh = Mh[64], bl = Mh[96];
-        mma_split(o[0], ol[0], uh, ul, bh.x, bh.y, bl.x, bl.y);
-        mma_split(o[1], ol[1], uh, ul, bh.z, bh.w, bl.z, bl.w);
+        mma_split(o[0], ol[0], om[0], uh, ul, bh.x, bh.y, bl.x, bl.y);
+        mma_split(o[1], ol[1], om[1], uh, ul, bh.z, bh.w, bl.z, bl.w);
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
             const uint4 eh = Eh[ks * 32], el = El[ks * 32];
@@ -350,7 +350,7 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int tok = nt * 8 + 2 * c + (e & 1);
-                if (tok < n && (e < 2 ? ok0 : ok1)) p.o[(size_t)(start + blk * kChunk + tok) * p.ldo + (size_t)h * p.dv + (e < 2 ? r0 : r1)] = o[nt][e] + ol[nt][e];
+                if (tok < n && (e < 2 ? ok0 : ok1)) p.o[(size_t)(start + blk * kChunk + tok) * p.ldo + (size_t)h * p.dv + (e < 2 ? r0 : r1)] = o[nt][e] + (ol[nt][e] + om[nt][e]);
             }
         }
     }

@@ -43,6 +43,54 @@ __global__ void seq_conv_ring_kernel(sllm_seq_batch b, const float* __restrict__
     out[(size_t)t * ldo + c] = acc;
 }
 
+// The same four channels at a time for portions: thread = (four channels, tile of kConvTile tokens); the weights and the last TAPS-1 inputs
+// stay in registers while the thread walks its tokens.
+constexpr int kConvTile = 8;
+template <int TAPS>
+__global__ void seq_conv_ring_vec_kernel(sllm_seq_batch b, const float* __restrict__ x, int ldx, int channels, const float* __restrict__ w, const float* __restrict__ cb,
+                                         const float* __restrict__ ring, int act, float* __restrict__ out, int ldo) {
+    const int ch = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+    if (ch >= channels) return;
+    float4 wt[TAPS];                                     // wt[back]: the weights of the input `back` positions before the token
+    {
+        float raw[4 * TAPS];
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) *reinterpret_cast<float4*>(raw + 4 * i) = *reinterpret_cast<const float4*>(w + (size_t)ch * TAPS + 4 * i);
+#pragma unroll
+        for (int back = 0; back < TAPS; ++back)
+            wt[back] = make_float4(raw[TAPS - 1 - back], raw[2 * TAPS - 1 - back], raw[3 * TAPS - 1 - back], raw[4 * TAPS - 1 - back]);
+    }
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f), bias = cb ? *reinterpret_cast<const float4*>(cb + ch) : zero;
+    float4 past[TAPS];                                   // past[back], back >= 1
+    int at = -1, prev_slot = -1;
+    const int t1 = min(b.T, (int)(blockIdx.y + 1) * kConvTile);
+    for (int t = blockIdx.y * kConvTile; t < t1; ++t) {
+        const int slot = b.tok_slot[t];
+        if (slot != prev_slot) {                         // the tile's first token, or another sequence's
+            at = b.tok_pos[t];
+            prev_slot = slot;
+#pragma unroll
+            for (int back = 1; back < TAPS; ++back) {
+                past[back] = zero;
+                if (at - back >= 0)
+                    past[back] = (t - back >= 0 && b.tok_slot[t - back] == slot)
+                                     ? *reinterpret_cast<const float4*>(x + (size_t)(t - back) * ldx + ch)
+                                     : *reinterpret_cast<const float4*>(ring + ((size_t)slot * (TAPS - 1) + (at - back) % (TAPS - 1)) * channels + ch);
+            }
+        }
+        const float4 own = *reinterpret_cast<const float4*>(x + (size_t)t * ldx + ch);
+        float4 a = make_float4(fmaf(wt[0].x, own.x, bias.x), fmaf(wt[0].y, own.y, bias.y), fmaf(wt[0].z, own.z, bias.z), fmaf(wt[0].w, own.w, bias.w));
+#pragma unroll
+        for (int back = 1; back < TAPS; ++back)
+            a = make_float4(fmaf(wt[back].x, past[back].x, a.x), fmaf(wt[back].y, past[back].y, a.y), fmaf(wt[back].z, past[back].z, a.z), fmaf(wt[back].w, past[back].w, a.w));
+#pragma unroll
+        for (int back = TAPS - 1; back >= 2; --back) past[back] = past[back - 1];
+        past[1] = own;
+        if (act == 1) a = make_float4(a.x * seq_sigmoid(a.x), a.y * seq_sigmoid(a.y), a.z * seq_sigmoid(a.z), a.w * seq_sigmoid(a.w));
+        *reinterpret_cast<float4*>(out + (size_t)t * ldo + ch) = a;
+    }
+}
+
 struct DeltaArgs {
     sllm_seq_batch b;
     const float *q, *k, *v; int ldq, ldk, ldv;          // after convolution and activation; q / k [kv_heads][dk], v [heads][dv] per token
@@ -361,6 +409,16 @@ int sllm_seq_conv_ring(const sllm_seq_batch* b, const float* x, int32_t ldx, int
     SLLM_REQUIRE(b && b->T > 0 && b->tok_slot && b->tok_pos, SLLM_EINVAL, "seq_conv_ring: incomplete batch description");
     SLLM_REQUIRE(x && w && out && channels > 0 && taps >= 1 && (taps == 1 || ring) && (act == 0 || act == 1), SLLM_EINVAL, "seq_conv_ring: bad argument");
     SLLM_REQUIRE(b->T <= 65535, SLLM_ENOTSUP, "seq_conv_ring: at most 65535 tokens per step");
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    if (b->T > b->nseg && taps >= 2 && taps <= 4 && channels % 4 == 0 && ldx % 4 == 0 && ldo % 4 == 0 && aligned(x) && aligned(w) && aligned(cb) && aligned(ring) && aligned(out)) {
+        const dim3 grid((channels / 4 + 127) / 128, (b->T + kConvTile - 1) / kConvTile);
+        if (taps == 2) seq_conv_ring_vec_kernel<2><<<grid, 128, 0, as_stream(stream)>>>(*b, x, ldx, channels, w, cb, ring, act, out, ldo);
+        else if (taps == 3) seq_conv_ring_vec_kernel<3><<<grid, 128, 0, as_stream(stream)>>>(*b, x, ldx, channels, w, cb, ring, act, out, ldo);
+        else seq_conv_ring_vec_kernel<4><<<grid, 128, 0, as_stream(stream)>>>(*b, x, ldx, channels, w, cb, ring, act, out, ldo);
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     seq_conv_ring_kernel<<<dim3((channels + 127) / 128, b->T), 128, 0, as_stream(stream)>>>(*b, x, ldx, channels, taps, w, cb, ring, act, out, ldo);
     ++g_launches;
     SLLM_LAUNCH_CHECK();

@@ -203,6 +203,48 @@ __global__ void __launch_bounds__(1024) seq_headnorm_gate_wide_kernel(const floa
     }
 }
 
+// the same four columns at a time: a team of `team` threads (a warp, or the whole CTA) per (token, part), R groups of four columns per thread,
+// everything in registers between the sum of squares and the scaling
+template <int R>
+__global__ void __launch_bounds__(1024) seq_headnorm_gate_vec_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ g, int ldg, const float* __restrict__ w,
+                                                                     int heads, int dv, float eps, float* __restrict__ out, int ldout, uint16_t* __restrict__ out16, int items,
+                                                                     int team, int mode) {
+    __shared__ float red[33];
+    const int per_cta = blockDim.x / team, item = blockIdx.x * per_cta + threadIdx.x / team, me = threadIdx.x % team;
+    const bool live = item < items;                      // (a CTA that is one team has one item: no thread leaves before the barriers)
+    const int t = live ? item / heads : 0, h = live ? item % heads : 0;
+    const float* orow = o + (size_t)t * ldo + (size_t)h * dv;
+    const float* grow = g + (size_t)t * ldg + (size_t)h * dv;
+    const float* wrow = (w && (mode & 2)) ? w + (size_t)h * dv : w;
+    const bool gate_first = mode & 1;
+    float4 v[R], s[R];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = 4 * (me + i * team);
+        v[i] = s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (live && j < dv) {
+            v[i] = *reinterpret_cast<const float4*>(orow + j);
+            const float4 gv = *reinterpret_cast<const float4*>(grow + j);
+            s[i] = make_float4(headnorm_gate_of(gv.x, mode), headnorm_gate_of(gv.y, mode), headnorm_gate_of(gv.z, mode), headnorm_gate_of(gv.w, mode));
+            if (gate_first) v[i] = make_float4(v[i].x * s[i].x, v[i].y * s[i].y, v[i].z * s[i].z, v[i].w * s[i].w);
+            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+        }
+    }
+    ss = team == 32 ? warp_sum(ss) : block_sum(ss, red);
+    const float inv = 1.0f / sqrtf(ss / (float)dv + eps);
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int j = 4 * (me + i * team);
+        if (!live || j >= dv) continue;
+        const float4 wj = wrow ? *reinterpret_cast<const float4*>(wrow + j) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+        float4 r = make_float4((v[i].x * inv) * wj.x, (v[i].y * inv) * wj.y, (v[i].z * inv) * wj.z, (v[i].w * inv) * wj.w);
+        if (!gate_first) r = make_float4(r.x * s[i].x, r.y * s[i].y, r.z * s[i].z, r.w * s[i].w);
+        if (out) *reinterpret_cast<float4*>(out + (size_t)t * ldout + (size_t)h * dv + j) = r;
+        if (out16) *reinterpret_cast<uint2*>(out16 + ((size_t)t * heads + h) * dv + j) = make_uint2(pack_bf16(r.x, r.y), pack_bf16(r.z, r.w));
+    }
+}
+
 // (row - mean) / sqrt(variance + eps) * w + b of one row that the CTA's threads hold strided; the variance is the mean of the squared
 // deviations (two passes: the mean first), as the definition says
 __device__ __forceinline__ void seq_layernorm_row(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float eps,
@@ -302,6 +344,23 @@ __global__ void seq_clamped_glu_kernel(const float* __restrict__ gate, int ldg, 
         const float v = (g * seq_sigmoid(alpha * g)) * (u + 1.0f);
         if (out) out[t * ldo + j] = v;
         if (out16) out16[i] = f32_to_bf16_bits(v);
+    }
+}
+
+// the same four columns at a time: grid (T, parts of a row)
+__global__ void seq_clamped_glu_vec_kernel(const float* __restrict__ gate, int ldg, const float* __restrict__ up, int ldu, float limit, float alpha, float* __restrict__ out,
+                                           int ldo, uint16_t* __restrict__ out16, int n) {
+    const size_t t = blockIdx.x;
+    auto one = [&](float g, float u) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return (g * seq_sigmoid(alpha * g)) * (u + 1.0f);
+    };
+    for (int j = (blockIdx.y * blockDim.x + threadIdx.x) * 4; j < n; j += gridDim.y * blockDim.x * 4) {
+        const float4 g = *reinterpret_cast<const float4*>(gate + t * ldg + j), u = *reinterpret_cast<const float4*>(up + t * ldu + j);
+        const float4 v = make_float4(one(g.x, u.x), one(g.y, u.y), one(g.z, u.z), one(g.w, u.w));
+        if (out) *reinterpret_cast<float4*>(out + t * ldo + j) = v;
+        if (out16) *reinterpret_cast<uint2*>(out16 + t * n + j) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
     }
 }
 
@@ -451,6 +510,15 @@ int sllm_seq_headnorm_gate(const float* o, int32_t ldo, const float* g, int32_t 
                            int32_t ldout, void* out16, int32_t T, int32_t mode, sllm_stream_t stream) {
     SLLM_REQUIRE(o && g && (out || out16) && heads > 0 && dv > 0 && T > 0 && mode >= 0 && mode <= 7, SLLM_EINVAL, "seq_headnorm_gate: bad argument");
     const int items = T * heads;
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    if (dv % 4 == 0 && ldo % 4 == 0 && ldg % 4 == 0 && (!out || ldout % 4 == 0) && dv <= 8192 && aligned(o) && aligned(g) && aligned(w) && aligned(out) && aligned(out16)) {
+        cudaStream_t st = as_stream(stream);
+        const int team = dv <= 256 ? 32 : std::min(1024, ((dv + 7) / 8 + 31) / 32 * 32), cta = team == 32 ? 128 : team, grid = team == 32 ? (items + 3) / 4 : items;
+        seq_headnorm_gate_vec_kernel<2><<<grid, cta, 0, st>>>(o, ldo, g, ldg, w, heads, dv, eps, out, ldout, (uint16_t*)out16, items, team, mode);
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     if (dv >= 512 && dv <= 1024 * kNormPer)       // a warp per part would walk such a part in 16 and more rounds, twice
         seq_headnorm_gate_wide_kernel<<<items, std::max(256, ((dv + kNormPer - 1) / kNormPer + 31) / 32 * 32), 0, as_stream(stream)>>>(o, ldo, g, ldg, w, heads, dv, eps, out, ldout,
                                                                                                                     (uint16_t*)out16, mode);
@@ -493,6 +561,14 @@ int sllm_seq_depth_average(float* x, const float* y, float* hist, int32_t n_prev
 int sllm_seq_clamped_glu(const float* gate, int32_t ldg, const float* up, int32_t ldu, float limit, float alpha, float* out, int32_t ldo, void* out16,
                          int32_t T, int32_t n, sllm_stream_t stream) {
     SLLM_REQUIRE(gate && up && (out || out16) && T > 0 && n > 0 && ldg >= n && ldu >= n && (!out || ldo >= n), SLLM_EINVAL, "seq_clamped_glu: bad argument");
+    auto aligned = [](const void* q) { return q == nullptr || ((uintptr_t)q % 16) == 0; };
+    if (n % 4 == 0 && ldg % 4 == 0 && ldu % 4 == 0 && (!out || ldo % 4 == 0) && aligned(gate) && aligned(up) && aligned(out) && aligned(out16)) {
+        seq_clamped_glu_vec_kernel<<<dim3(T, std::min(64, (n / 4 + 255) / 256)), n >= 1024 ? 256 : 64, 0, as_stream(stream)>>>(gate, ldg, up, ldu, limit, alpha, out, ldo,
+                                                                                                                           (uint16_t*)out16, n);
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     const size_t total = (size_t)T * n;
     seq_clamped_glu_kernel<<<(int)std::min<size_t>((total + 255) / 256, (size_t)sm_count() * 8), 256, 0, as_stream(stream)>>>(gate, ldg, up, ldu, limit, alpha, out,
                                                                                                                        ldo, (uint16_t*)out16, T, n);

@@ -788,9 +788,9 @@ class ConvRotaryAttention:
         if ring is not None and T > step.nseg:
             ops.ring_store(step.b, q, ld, self.channels, c.conv, ring, step.st)
         ws = step.scratch("attn_ws", T * c.heads * step.nsplit * (c.vdim + 2))
-        ops.attention(step.b, qo, ldq, c.heads, c.kv_heads, c.dim, c.vdim, c.scale, state["k"], state["v"], step.nsplit, ws, step.st, opts=self.opts)
         rows16 = self.out.operand_rows(step)
-        ops.attention_finish(step.b, ws, step.nsplit, c.heads, c.vdim, None, 0, None, 0, None if rows16 is not None else out, self.width, step.st, out16=rows16)
+        ops.attention_out(step.b, qo, ldq, c.heads, c.kv_heads, c.dim, c.vdim, c.scale, state["k"], state["v"], step.nsplit, ws, None if rows16 is not None else out,
+                          self.width, step.st, opts=self.opts, out16=rows16)
         return rows16 is not None
 
 

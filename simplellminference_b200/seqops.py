@@ -102,6 +102,11 @@ class Ops:
         self._ck(self.lib.sllm_seq_attention(C.byref(b), q_ptr, ldq, heads, kv_heads, dk, dv, scale, _p(k_pool), _p(v_pool), self.kv_dtype, nsplit,
                                              _p(ws), C.byref(opts) if opts is not None else None, st))
 
+    def attention_out(self, b, q_ptr, ldq, heads, kv_heads, dk, dv, scale, k_pool, v_pool, nsplit, ws, out, ldo, st, opts=None, out16=None):
+        """``attention`` and the plain merge of its shares."""
+        self._ck(self.lib.sllm_seq_attention_out(C.byref(b), q_ptr, ldq, heads, kv_heads, dk, dv, scale, _p(k_pool), _p(v_pool), self.kv_dtype, nsplit, _p(ws),
+                                                 C.byref(opts) if opts is not None else None, _p(out), ldo, _p(out16), st))
+
     def attention_finish(self, b, ws, nsplit, heads, dv, vfreq, layout, gate_ptr, ldg, out, ldo, st, sink=None, gate_channels=False, out16=None):
         """``gate_channels``: the gate has a column per output column instead of one per head."""
         self._ck(self.lib.sllm_seq_attention_finish(C.byref(b), _p(ws), nsplit, heads, dv, _p(vfreq), layout, gate_ptr, ldg, int(bool(gate_channels)), _p(sink),
