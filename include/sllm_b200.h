@@ -578,7 +578,7 @@ int sllm_seq_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, co
                         int32_t ldo, const float* conv_x, int32_t ldx, int32_t channels, int32_t taps, float* ring, void* chunk_ws,
                         sllm_stream_t stream);
 /* scratch of the block form of the recurrences (0: these sizes have none); n_qtiles as in the batch description */
-int64_t sllm_seq_chunk_ws_bytes(int32_t n_qtiles, int32_t heads, int32_t dk);
+int64_t sllm_seq_chunk_ws_bytes(int32_t n_qtiles, int32_t heads, int32_t dk, int32_t dv);
 /* The same rule with a decay per head and key channel: step_logit [T][heads * dk], dt_bias [heads * dk], S[c][:] <- g[c] S[c][:] with
  * g[c] = exp(-exp(A_log[h]) * softplus(step_logit[h * dk + c] + dt_bias[h * dk + c])); everything else as above. */
 int sllm_seq_channel_delta_rule(const sllm_seq_batch* b, const float* q, int32_t ldq, const float* k, int32_t ldk, const float* v, int32_t ldv,

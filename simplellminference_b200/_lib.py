@@ -173,7 +173,7 @@ SIGNATURES.update({
     "sllm_seq_normed_rotary_kv": (C.c_int, [_B, _P, _I, _I, _I, _P, _I, _I, _P, _I, _I, _P, _P, _F, _P, _I, _I, _P, _P, _I, _P]),
     "sllm_seq_head_mix": (C.c_int, [_P, _I, _P, _I, _I, _I, _P, _I, _P, _I, _P]),
     "sllm_seq_delta_rule": (C.c_int, [_B, _P, _I, _P, _I, _P, _I, _P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P, _I, _I, _I, _P, _P, _P]),
-    "sllm_seq_chunk_ws_bytes": (_L, [_I, _I, _I]),
+    "sllm_seq_chunk_ws_bytes": (_L, [_I, _I, _I, _I]),
     "sllm_seq_moe_act": (C.c_int, [_P, _I, _I, _I, _I, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, C.POINTER(SeqMoeOpts), _P]),
     "sllm_seq_linear_grouped": (C.c_int, [_P, _I, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
     "sllm_seq_branch_seam": (C.c_int, [_P, _P, _I, C.POINTER(_P), C.POINTER(_P), C.POINTER(_I), _F, _P, _P, _P, _I, _I, _P]),

@@ -10,9 +10,9 @@
 // (1) seq_chunk_prepare_kernel, CTA = (block, head), all blocks of the step in parallel: silu / rotation / unit vectors, G, A and B (fp32,
 // a pair of threads per entry), M by forward substitution; leaves e^G k, e^G q, e^(G_n - G) k, M and B as the tensor-core fragments the walk
 // will load, each as two bf16 terms (x = hi + lo, |x - hi - lo| <= 2^-17 |x|), and e^G_n in fp32.
-// (2) seq_chunk_walk_kernel, CTA = (portion, head, 64 value columns), warp = 16 value columns: S^T [16][dk] stays in the accumulators
-// (fp32) from the portion's first token to its last. An accumulator fragment is register for register an A fragment of the next product, so
-// state, u and o never leave the warp; all products take both operands as two bf16 terms (three products, fp32 accumulation), which keeps
+// (2) seq_chunk_walk_kernel, CTA = (portion, head, 16 or 32 value columns), two or four warps = 16 value columns, a share of the key channels each: their part of
+// S^T [16][dk] stays in the accumulators (fp32) from the portion's first token to its last. An accumulator fragment is register for register
+// an A fragment of the next product, so state and u never leave the registers; all products take both operands as two bf16 terms (three products, fp32 accumulation), which keeps
 // the recurrence at fp32 working accuracy. The blocks' records arrive by cp.async, three stages.
 #include "seq_attn.cuh"
 #include "seq_chunk.cuh"
@@ -20,7 +20,7 @@
 namespace sllm {
 
 constexpr int kPrepThreads = 288;    // two threads per entry of a triangle of 16 x 16
-constexpr int kWalkStages = 3, kWalkCols = 64;
+constexpr int kWalkStages = 3;
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct ChunkPlace { int seg, start, n, id; };      // segment, first token in the batch, tokens, number of the block in segment order
@@ -78,6 +78,12 @@ __global__ void __launch_bounds__(kPrepThreads) seq_chunk_prepare_kernel(ChunkAr
             s_G[tok * ld + ch] = g;
         }
     }
+    if (!kDelta && p.silu)                               // the values too, for the walk
+        for (int i = threadIdx.x; i < c.n * p.dv; i += kPrepThreads) {
+            const int tok = i / p.dv, j = i % p.dv;
+            const float v = p.v[(size_t)(c.start + tok) * p.ldv + (size_t)h * p.dv + j];
+            p.v_ws[((size_t)c.id * kChunk + tok) * p.heads * p.dv + (size_t)h * p.dv + j] = v * seq_sigmoid(v);
+        }
     if (kDelta && threadIdx.x < kChunk) s_beta[threadIdx.x] = (int)threadIdx.x < c.n ? seq_sigmoid(p.bl[(size_t)(c.start + threadIdx.x) * p.ldb + h]) : 0.0f;
     __syncthreads();
     for (int tok = warp; tok < c.n; tok += kPrepThreads / 32) {
@@ -213,40 +219,49 @@ __device__ __forceinline__ void mma_split(float (&d)[4], float (&dl)[4], float (
     mma_bf16_16816(dm, ah, l0, l1);
 }
 
-// KS: k-steps of 16 key channels
-template <int KS, bool kDelta>
-__global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int vec) {
+// KS: k-steps of 16 key channels. PARTS warps share 16 value columns, each owning KS / PARTS of the k-steps; they add their parts of the
+// products with the old state through shared memory and finish 16 / PARTS outputs per column each. GROUPS: how many times 16 columns a CTA takes.
+template <int KS, int PARTS, int GROUPS, bool kDelta>
+__global__ void __launch_bounds__(PARTS * GROUPS * 32) seq_chunk_walk_kernel(ChunkArgs p, int vec) {
     extern __shared__ __align__(16) uint8_t cw_sm[];
-    constexpr int dkp = KS * 16;
+    constexpr int dkp = KS * 16, HS = KS / PARTS, kThreads = PARTS * GROUPS * 32, kCols = GROUPS * 16;
     constexpr uint32_t kPlane = kChunk * dkp * 2;
-    const size_t rec_bytes = chunk_record_bytes(dkp);
-    const size_t stage_bytes = rec_bytes + kChunk * kWalkCols * 4;
+    constexpr uint32_t rec_bytes = (uint32_t)chunk_record_bytes(dkp), stage_bytes = rec_bytes + kChunk * kCols * 4;
     const sllm_seq_batch& b = p.b;
-    const int seg = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kWalkCols;
+    const int seg = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * kCols;
     const int start = b.seg_start[seg], len = b.seg_len[seg], slot = b.seg_slot[seg];
     const int blocks = (len + kChunk - 1) / kChunk;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, c = lane & 3;
-    const int cl = warp * 16 + g, r0 = col0 + cl, r1 = r0 + 8;      // this thread's two value columns
+    const int group = warp % GROUPS, part = warp / GROUPS, k0 = part * HS;   // this warp's value columns and first k-step
+    const int cl = group * 16 + g, r0 = col0 + cl, r1 = r0 + 8;              // this thread's two value columns
     const bool ok0 = r0 < p.dv, ok1 = r1 < p.dv;
-    const uint8_t* recs = p.ws + ((size_t)(2 * b.seg_tile0[seg]) * p.heads + h) * rec_bytes;
+    // what the warps of a group hand each other: [group][part][x, x, o, o][lane]
+    float4* exchange = reinterpret_cast<float4*>(cw_sm + kWalkStages * stage_bytes) + group * (PARTS * 4 * 32) + lane;
+    const size_t first = 2 * (size_t)b.seg_tile0[seg];   // number of the portion's first block
+    const uint8_t* recs = p.ws + (first * p.heads + h) * rec_bytes;
+    // values: the batch's rows, or those the preparation left (passed through silu), 16 rows per block
+    const bool own_v = !kDelta && p.silu;
+    const float* vsrc = own_v ? p.v_ws + first * kChunk * p.heads * p.dv + (size_t)h * p.dv + col0 : p.v + (size_t)start * p.ldv + (size_t)h * p.dv + col0;
+    const size_t ldv = own_v ? (size_t)p.heads * p.dv : (size_t)p.ldv;
     auto issue = [&](int blk) {
-        uint8_t* dst = cw_sm + (size_t)(blk % kWalkStages) * stage_bytes;
+        uint8_t* dst = cw_sm + (blk % kWalkStages) * stage_bytes;
         const uint8_t* src = recs + (size_t)blk * p.heads * rec_bytes;
-        for (uint32_t i = threadIdx.x + (kDelta ? 0 : 2 * kPlane / 16); i < rec_bytes / 16; i += 128) cp_async16(dst + 16 * i, src + 16 * i, 16);
+#pragma unroll 4
+        for (uint32_t i = threadIdx.x + (kDelta ? 0 : 2 * kPlane / 16); i < rec_bytes / 16; i += kThreads) cp_async16(dst + 16 * i, src + 16 * i, 16);
         float* dv = reinterpret_cast<float*>(dst + rec_bytes);
         const int n = min(kChunk, len - blk * kChunk);
+        const float* vb = vsrc + (size_t)blk * kChunk * ldv;
         if (vec) {
-            for (int i = threadIdx.x; i < kChunk * kWalkCols / 4; i += 128) {
-                const int tok = i / (kWalkCols / 4), j = (i % (kWalkCols / 4)) * 4;
+            for (int i = threadIdx.x; i < kChunk * kCols / 4; i += kThreads) {
+                const int tok = i / (kCols / 4), j = (i % (kCols / 4)) * 4;
                 const bool has = tok < n && col0 + j < p.dv;
-                cp_async16(dv + tok * kWalkCols + j, has ? p.v + (size_t)(start + blk * kChunk + tok) * p.ldv + (size_t)h * p.dv + col0 + j : p.v, has ? 16 : 0);
+                cp_async16(dv + tok * kCols + j, has ? vb + tok * ldv + j : vsrc, has ? 16 : 0);
             }
         } else {
-            for (int i = threadIdx.x; i < kChunk * kWalkCols; i += 128) {
-                const int tok = i / kWalkCols, j = i % kWalkCols;
+            for (int i = threadIdx.x; i < kChunk * kCols; i += kThreads) {
+                const int tok = i / kCols, j = i % kCols;
                 const bool has = tok < n && col0 + j < p.dv;
-                const float* s = has ? p.v + (size_t)(start + blk * kChunk + tok) * p.ldv + (size_t)h * p.dv + col0 + j : p.v;
-                asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dv + i)), "l"(s), "r"(has ? 4 : 0) : "memory");
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dv + i)), "l"(has ? vb + tok * ldv + j : p.v), "r"(has ? 4 : 0) : "memory");
             }
         }
         cp_async_commit();
@@ -255,34 +270,37 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
     if (blocks > 1) issue(1);
     else cp_async_commit();
     float* st = p.state + ((size_t)slot * p.heads + h) * p.dk * p.dv;
-    float S[2 * KS][4];                                  // S^T: rows r0 / r1, columns (key channels) nt * 8 + 2c, + 1
+    float S[2 * HS][4];                                  // S^T: rows r0 / r1, columns (key channels) k0 * 16 + nt * 8 + 2c, + 1
 #pragma unroll
-    for (int nt = 0; nt < 2 * KS; ++nt)
+    for (int nt = 0; nt < 2 * HS; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int ch = nt * 8 + 2 * c + (e & 1);
+            const int ch = k0 * 16 + nt * 8 + 2 * c + (e & 1);
             S[nt][e] = (e < 2 ? ok0 : ok1) && ch < p.dk ? st[(size_t)ch * p.dv + (e < 2 ? r0 : r1)] : 0.0f;
         }
-    for (int blk = 0; blk < blocks; ++blk) {
+    const bool work = col0 + group * 16 < p.dv;          // the same answer in all warps of a group
+    // the outputs this warp finishes: tokens mt * 8 + 2c and + 1 of columns r0 and r1 (two parts) or of one of them (four)
+    const int mt = PARTS == 4 ? part >> 1 : part, mrow = PARTS == 4 ? part & 1 : 0;
+    float* orow = p.o + (size_t)(start + mt * 8 + 2 * c) * p.ldo + (size_t)h * p.dv + (mrow ? r1 : r0);
+    for (int blk = 0; blk < blocks; ++blk, orow += (size_t)kChunk * p.ldo) {
         cp_async_wait<1>();
         __syncthreads();                                 // this block has landed for everyone, and everyone has left the block before
         if (blk + 2 < blocks) issue(blk + 2);
         else cp_async_commit();
-        const uint8_t* rec = cw_sm + (size_t)(blk % kWalkStages) * stage_bytes;
-        const uint4* Kh = reinterpret_cast<const uint4*>(rec) + lane;
+        if (!work) continue;
+        const uint8_t* rec = cw_sm + (blk % kWalkStages) * stage_bytes;
+        const uint4* Kh = reinterpret_cast<const uint4*>(rec) + k0 * 32 + lane;
         const uint4* Kl = Kh + kPlane / 16;
         const uint4* Qh = Kl + kPlane / 16;
         const uint4* Ql = Qh + kPlane / 16;
         const uint4* Eh = Ql + kPlane / 16;              // keys decayed to the block's end
         const uint4* El = Eh + kPlane / 16;
-        const uint4* Mh = El + kPlane / 16;              // M hi, M lo, B hi, B lo: 32 pieces each
-        const float* D = reinterpret_cast<const float*>(rec + 6 * kPlane + 4 * kChunk * kChunk * 2);
-        const float* sv = reinterpret_cast<const float*>(rec + rec_bytes);
-        const int n = min(kChunk, len - blk * kChunk);
-        if (col0 + warp * 16 < p.dv) {                   // the same answer in every lane of the warp
+        const uint4* Mh = reinterpret_cast<const uint4*>(rec + 6 * kPlane) + lane;              // M hi, M lo, B hi, B lo: 32 pieces each
+        const float* D = reinterpret_cast<const float*>(rec + 6 * kPlane + 4 * kChunk * kChunk * 2) + k0 * 16 + 2 * c;
+        const float* sv = reinterpret_cast<const float*>(rec + rec_bytes) + 2 * c * kCols + cl;
         float x[2][4] = {}, xl[2][4] = {}, xm[2][4] = {}, o[2][4] = {}, ol[2][4] = {}, om[2][4] = {};     // rows r0 / r1, columns (tokens) nt * 8 + 2c, + 1
 #pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
+        for (int ks = 0; ks < HS; ++ks) {
             uint32_t ah[4], al[4];
             split_bf16(S[2 * ks][0], S[2 * ks][1], &ah[0], &al[0]);
             split_bf16(S[2 * ks][2], S[2 * ks][3], &ah[1], &al[1]);
@@ -297,22 +315,45 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
             mma_split(o[0], ol[0], om[0], ah, al, qh.x, qh.y, ql.x, ql.y);
             mma_split(o[1], ol[1], om[1], ah, al, qh.z, qh.w, ql.z, ql.w);
         }
+        auto sum3 = [](const float (&p0)[4], const float (&p1)[4], const float (&p2)[4]) {
+            return make_float4(p0[0] + (p1[0] + p2[0]), p0[1] + (p1[1] + p2[1]), p0[2] + (p1[2] + p2[2]), p0[3] + (p1[3] + p2[3]));
+        };
+        float4* mine = exchange + part * 4 * 32;
+        if (kDelta) {
+            mine[0] = sum3(x[0], xl[0], xm[0]);
+            mine[32] = sum3(x[1], xl[1], xm[1]);
+        }
+        mine[64] = sum3(o[0], ol[0], om[0]);
+        mine[96] = sum3(o[1], ol[1], om[1]);
 #pragma unroll
-        for (int nt = 0; nt < 2 * KS; ++nt) {            // the old state decays to the block's end
-            const float2 d = *reinterpret_cast<const float2*>(D + nt * 8 + 2 * c);
+        for (int nt = 0; nt < 2 * HS; ++nt) {            // the old state decays to the block's end
+            const float2 d = *reinterpret_cast<const float2*>(D + nt * 8);
             S[nt][0] *= d.x;
             S[nt][1] *= d.y;
             S[nt][2] *= d.x;
             S[nt][3] *= d.y;
         }
+        float v[2][4];
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                float v = sv[(nt * 8 + 2 * c + (e & 1)) * kWalkCols + cl + (e < 2 ? 0 : 8)];
-                if (!kDelta && p.silu) v = v * seq_sigmoid(v);
-                x[nt][e] = v - (x[nt][e] + (xl[nt][e] + xm[nt][e]));
+            for (int e = 0; e < 4; ++e) v[nt][e] = sv[(nt * 8 + (e & 1)) * kCols + (e < 2 ? 0 : 8)];
+        asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(PARTS * 32) : "memory");   // the warps of the group
+        if (kDelta) {
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt) {
+                float4 y = exchange[nt * 32];
+#pragma unroll
+                for (int q = 1; q < PARTS; ++q) {
+                    const float4 z = exchange[(q * 4 + nt) * 32];
+                    y = make_float4(y.x + z.x, y.y + z.y, y.z + z.z, y.w + z.w);
+                }
+                v[nt][0] -= y.x;
+                v[nt][1] -= y.y;
+                v[nt][2] -= y.z;
+                v[nt][3] -= y.w;
             }
+        }
         uint32_t uh[4], ul[4];
         auto operand = [&](const float (&y)[2][4]) {     // rows x 16 tokens as an A fragment
             split_bf16(y[0][0], y[0][1], &uh[0], &ul[0]);
@@ -320,7 +361,7 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
             split_bf16(y[1][0], y[1][1], &uh[2], &ul[2]);
             split_bf16(y[1][2], y[1][3], &uh[3], &ul[3]);
         };
-        operand(x);
+        operand(v);
         if (kDelta) {
             float u[2][4] = {}, lo[2][4] = {}, mid[2][4] = {};
             const uint4 mh = Mh[0], ml = Mh[32];
@@ -332,11 +373,8 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
                 for (int e = 0; e < 4; ++e) u[nt][e] += lo[nt][e] + mid[nt][e];
             operand(u);
         }
-        const uint4 bh = Mh[64], bl = Mh[96];
-        mma_split(o[0], ol[0], om[0], uh, ul, bh.x, bh.y, bl.x, bl.y);
-        mma_split(o[1], ol[1], om[1], uh, ul, bh.z, bh.w, bl.z, bl.w);
 #pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
+        for (int ks = 0; ks < HS; ++ks) {
             const uint4 eh = Eh[ks * 32], el = El[ks * 32];
             mma_bf16_16816(S[2 * ks], uh, eh.x, eh.y);
             mma_bf16_16816(S[2 * ks + 1], uh, eh.z, eh.w);
@@ -345,59 +383,77 @@ __global__ void __launch_bounds__(128) seq_chunk_walk_kernel(ChunkArgs p, int ve
             mma_bf16_16816(S[2 * ks], uh, el.x, el.y);
             mma_bf16_16816(S[2 * ks + 1], uh, el.z, el.w);
         }
+        const uint4 bh = Mh[64], bl = Mh[96];
+        float y[4] = {}, yl[4] = {}, ym[4] = {};
+        if (mt == 0) mma_split(y, yl, ym, uh, ul, bh.x, bh.y, bl.x, bl.y);
+        else mma_split(y, yl, ym, uh, ul, bh.z, bh.w, bl.z, bl.w);
+        const int n = min(kChunk, len - blk * kChunk), tok = mt * 8 + 2 * c;
+        if (PARTS == 4) {                                // two tokens of one column
+            const float* at = reinterpret_cast<const float*>(exchange + (2 + mt) * 32) + 2 * mrow;
+            float2 z = *reinterpret_cast<const float2*>(at);
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int tok = nt * 8 + 2 * c + (e & 1);
-                if (tok < n && (e < 2 ? ok0 : ok1)) p.o[(size_t)(start + blk * kChunk + tok) * p.ldo + (size_t)h * p.dv + (e < 2 ? r0 : r1)] = o[nt][e] + (ol[nt][e] + om[nt][e]);
+            for (int q = 1; q < PARTS; ++q) {
+                const float2 w = *reinterpret_cast<const float2*>(at + q * 4 * 32 * 4);
+                z = make_float2(z.x + w.x, z.y + w.y);
             }
+            const float o0 = (mrow ? y[2] + (yl[2] + ym[2]) : y[0] + (yl[0] + ym[0])) + z.x, o1 = (mrow ? y[3] + (yl[3] + ym[3]) : y[1] + (yl[1] + ym[1])) + z.y;
+            if (mrow ? ok1 : ok0) {
+                if (tok < n) orow[0] = o0;
+                if (tok + 1 < n) orow[p.ldo] = o1;
+            }
+        } else {                                         // two tokens of both columns
+            const float4 z0 = exchange[(2 + mt) * 32], z1 = exchange[(4 + 2 + mt) * 32];
+            if (ok0 && tok < n) orow[0] = y[0] + (yl[0] + ym[0]) + (z0.x + z1.x);
+            if (ok0 && tok + 1 < n) orow[p.ldo] = y[1] + (yl[1] + ym[1]) + (z0.y + z1.y);
+            if (ok1 && tok < n) orow[8] = y[2] + (yl[2] + ym[2]) + (z0.z + z1.z);
+            if (ok1 && tok + 1 < n) orow[p.ldo + 8] = y[3] + (yl[3] + ym[3]) + (z0.w + z1.w);
         }
     }
 #pragma unroll
-    for (int nt = 0; nt < 2 * KS; ++nt)
+    for (int nt = 0; nt < 2 * HS; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const int ch = nt * 8 + 2 * c + (e & 1);
+            const int ch = k0 * 16 + nt * 8 + 2 * c + (e & 1);
             if ((e < 2 ? ok0 : ok1) && ch < p.dk) st[(size_t)ch * p.dv + (e < 2 ? r0 : r1)] = S[nt][e];
         }
 }
 
-int launch_chunk_scan(const ChunkArgs& p, cudaStream_t st) {
-    const int dkp = chunk_key(p.dk);
-    SLLM_REQUIRE(p.dk <= kChunkMaxKey && p.ws && ((uintptr_t)p.ws % 16) == 0 && p.b.seg_tile0 && p.b.qt_seg && p.b.qt_off && p.b.n_qtiles > 0, SLLM_EINVAL,
-                 "chunk scan: heads of %d key channels, or an incomplete batch description", p.dk);
-    const size_t smem_prep = (size_t)3 * kChunk * (dkp + 4) * sizeof(float);
-    const size_t smem_walk = kWalkStages * (chunk_record_bytes(dkp) + kChunk * kWalkCols * 4);
-    const dim3 gp(2 * p.b.n_qtiles, p.heads), gw(p.b.nseg, p.heads, (p.dv + kWalkCols - 1) / kWalkCols);
-    if (p.delta) seq_chunk_prepare_kernel<true><<<gp, kPrepThreads, smem_prep, st>>>(p);
-    else seq_chunk_prepare_kernel<false><<<gp, kPrepThreads, smem_prep, st>>>(p);
-    ++g_launches;
-    SLLM_LAUNCH_CHECK();
-    const int vec = p.ldv % 4 == 0 && p.dv % 4 == 0 && ((uintptr_t)p.v % 16) == 0;
-#define SLLM_CHUNK_LAUNCH(KS, DELTA)                                                                                                                      \
-    do {                                                                                                                                                  \
-        SLLM_CUDA(cudaFuncSetAttribute(seq_chunk_walk_kernel<KS, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_walk));                   \
-        seq_chunk_walk_kernel<KS, DELTA><<<gw, 128, smem_walk, st>>>(p, vec);                                                                             \
-    } while (0)
-#define SLLM_CHUNK_LAUNCH_KS(DELTA)                          \
-    do {                                                     \
-        if (dkp == 32) SLLM_CHUNK_LAUNCH(2, DELTA);          \
-        else if (dkp == 64) SLLM_CHUNK_LAUNCH(4, DELTA);     \
-        else if (dkp == 96) SLLM_CHUNK_LAUNCH(6, DELTA);     \
-        else SLLM_CHUNK_LAUNCH(8, DELTA);                    \
-    } while (0)
-    if (p.delta) SLLM_CHUNK_LAUNCH_KS(true);
-    else SLLM_CHUNK_LAUNCH_KS(false);
-#undef SLLM_CHUNK_LAUNCH_KS
-#undef SLLM_CHUNK_LAUNCH
+template <int KS, int PARTS, int GROUPS, bool kDelta>
+static int launch_walk(const ChunkArgs& p, int vec, cudaStream_t st) {
+    constexpr size_t smem = kWalkStages * (chunk_record_bytes(KS * 16) + kChunk * GROUPS * 16 * 4) + GROUPS * PARTS * 4 * 32 * sizeof(float4);
+    SLLM_CUDA(cudaFuncSetAttribute(seq_chunk_walk_kernel<KS, PARTS, GROUPS, kDelta>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    seq_chunk_walk_kernel<KS, PARTS, GROUPS, kDelta><<<dim3(p.b.nseg, p.heads, (p.dv + GROUPS * 16 - 1) / (GROUPS * 16)), PARTS * GROUPS * 32, smem, st>>>(p, vec);
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     return SLLM_OK;
 }
 
+template <bool kDelta>
+static int launch_chunk_as(ChunkArgs p, cudaStream_t st) {
+    const int dkp = chunk_key(p.dk);
+    p.v_ws = reinterpret_cast<float*>(p.ws + 2 * (size_t)p.b.n_qtiles * p.heads * chunk_record_bytes(dkp));
+    seq_chunk_prepare_kernel<kDelta><<<dim3(2 * p.b.n_qtiles, p.heads), kPrepThreads, (size_t)3 * kChunk * (dkp + 4) * sizeof(float), st>>>(p);
+    ++g_launches;
+    SLLM_LAUNCH_CHECK();
+    const bool own_v = !kDelta && p.silu;
+    const int vec = p.dv % 4 == 0 && (own_v || (p.ldv % 4 == 0 && ((uintptr_t)p.v % 16) == 0));
+    // a walk is a chain of dependent blocks: few heads are spread over the machine 16 value columns a CTA, many take 32 (every CTA of a head
+    // loads all of the head's records)
+    const bool narrow = (long long)p.b.nseg * p.heads * ((p.dv + 31) / 32) < sm_count() / 2;
+    if (dkp == 32) return narrow ? launch_walk<2, 2, 1, kDelta>(p, vec, st) : launch_walk<2, 2, 2, kDelta>(p, vec, st);
+    if (dkp == 64) return narrow ? launch_walk<4, 4, 1, kDelta>(p, vec, st) : launch_walk<4, 4, 2, kDelta>(p, vec, st);
+    if (dkp == 96) return narrow ? launch_walk<6, 2, 1, kDelta>(p, vec, st) : launch_walk<6, 2, 2, kDelta>(p, vec, st);
+    return narrow ? launch_walk<8, 4, 1, kDelta>(p, vec, st) : launch_walk<8, 4, 2, kDelta>(p, vec, st);
+}
+
+int launch_chunk_scan(const ChunkArgs& p, cudaStream_t st) {
+    SLLM_REQUIRE(p.dk <= kChunkMaxKey && p.ws && ((uintptr_t)p.ws % 16) == 0 && p.b.seg_tile0 && p.b.qt_seg && p.b.qt_off && p.b.n_qtiles > 0, SLLM_EINVAL,
+                 "chunk scan: heads of %d key channels, or an incomplete batch description", p.dk);
+    return p.delta ? launch_chunk_as<true>(p, st) : launch_chunk_as<false>(p, st);
+}
+
 }  // namespace sllm
 
-extern "C" int64_t sllm_seq_chunk_ws_bytes(int32_t n_qtiles, int32_t heads, int32_t dk) {
-    return dk > 0 && dk <= sllm::kChunkMaxKey && n_qtiles > 0 && heads > 0 ? (int64_t)sllm::chunk_ws_bytes(n_qtiles, heads, dk) : 0;
+extern "C" int64_t sllm_seq_chunk_ws_bytes(int32_t n_qtiles, int32_t heads, int32_t dk, int32_t dv) {
+    return dk > 0 && dk <= sllm::kChunkMaxKey && dv > 0 && n_qtiles > 0 && heads > 0 ? (int64_t)sllm::chunk_ws_bytes(n_qtiles, heads, dk, dv) : 0;
 }

@@ -18,15 +18,18 @@ struct ChunkArgs {
     int heads, kv_heads, dk, dv;
     float unit_eps, scale;                               // delta rule: q times scale; constant decay: k times scale
     float* state; float* o; int ldo;
-    uint8_t* ws;                                         // chunk_ws_bytes
+    uint8_t* ws;                                         // chunk_ws_bytes: the blocks' records, then
+    float* v_ws;                                         // values passed through silu [blocks][16][heads * dv] (set by the launch)
 };
 
 // key channels rounded up to what the kernel is instantiated for
 __host__ __device__ __forceinline__ int chunk_key(int dk) { return dk <= 32 ? 32 : dk <= 64 ? 64 : dk <= 96 ? 96 : 128; }
 // per block and head: decayed keys, decayed queries and keys decayed to the block's end as (hi, lo) bf16 fragments, the two 16 x 16 matrices
 // likewise, the block's decay per key channel
-__host__ __device__ __forceinline__ size_t chunk_record_bytes(int dkp) { return (size_t)dkp * (6 * kChunk * 2 + 4) + 4 * kChunk * kChunk * 2; }
-inline size_t chunk_ws_bytes(int n_qtiles, int heads, int dk) { return 2 * (size_t)n_qtiles * heads * chunk_record_bytes(chunk_key(dk)); }
+__host__ __device__ constexpr size_t chunk_record_bytes(int dkp) { return (size_t)dkp * (6 * kChunk * 2 + 4) + 4 * kChunk * kChunk * 2; }
+inline size_t chunk_ws_bytes(int n_qtiles, int heads, int dk, int dv) {
+    return 2 * (size_t)n_qtiles * heads * (chunk_record_bytes(chunk_key(dk)) + (size_t)kChunk * dv * sizeof(float));
+}
 int launch_chunk_scan(const ChunkArgs& p, cudaStream_t st);
 
 }  // namespace sllm

@@ -447,7 +447,7 @@ static int delta_run(bool ssd, const float* skip, const DeltaExtra& ex, const sl
     SLLM_REQUIRE(!ring || (conv_x && channels > 0 && taps >= 1), SLLM_EINVAL, "seq_delta_rule: the ring needs the convolution's inputs");
     if (ex.chunk_ws) {
         ChunkArgs c{*b, q, k, v, ldq, ldk, ldv, !ssd, beta_logit, step_logit, ldb, lda, A_log, dt_bias, ex.channel, ex.rate, (const float2*)ex.angles, ex.n_freq, ex.layout,
-                    ex.silu, heads, kv_heads, dk, dv, unit_eps, qscale, state, o, ldo, (uint8_t*)ex.chunk_ws};
+                    ex.silu, heads, kv_heads, dk, dv, unit_eps, qscale, state, o, ldo, (uint8_t*)ex.chunk_ws, nullptr};
         if (int rc = launch_chunk_scan(c, as_stream(stream))) return rc;
         return ring && taps > 1 ? sllm_seq_ring_store(b, conv_x, ldx, channels, taps, ring, stream) : SLLM_OK;
     }

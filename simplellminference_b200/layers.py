@@ -389,7 +389,7 @@ class GatedDeltaRule:
         o = step.scratch("delta_o", T * self.width)
         ops.delta_rule(step.b, u.data_ptr(), C, u.data_ptr() + nk * F32B, C, u.data_ptr() + 2 * nk * F32B, C, bl, ld, al, ld, self.a_log, self.dt_bias,
                        c.heads, c.kv_heads, c.dim, c.vdim, self.unit_eps, c.dim ** -0.5, state["S"], o, self.width, q, ld, C, c.conv, ring, step.st,
-                       chunk_ws=step.chunk_scratch(c.heads, c.dim))
+                       chunk_ws=step.chunk_scratch(c.heads, c.dim, c.vdim))
         ops.headnorm_gate(o.data_ptr(), self.width, g, ld, self.norm_w, c.heads, c.vdim, self.eps, out, self.width, T, step.st)
 
 
@@ -440,7 +440,7 @@ class ChannelDeltaRule:
         o = step.scratch("delta_o", T * self.width)
         ops.channel_delta_rule(step.b, u.data_ptr(), C, u.data_ptr() + nk * F32B, C, u.data_ptr() + 2 * nk * F32B, C, bl, ld, al.data_ptr(), self.a2.N, self.a_log,
                                self.dt_bias, c.heads, c.kv_heads, c.dim, c.vdim, self.unit_eps, c.dim ** -0.5, state["S"], o, self.width, q, ld, C, c.conv, ring,
-                               step.st, chunk_ws=step.chunk_scratch(c.heads, c.dim))
+                               step.st, chunk_ws=step.chunk_scratch(c.heads, c.dim, c.vdim))
         rows16 = self.out.operand_rows(step)
         ops.headnorm_gate(o.data_ptr(), self.width, gate.data_ptr(), self.width, self.norm_w, c.heads, c.vdim, self.eps, None if rows16 is not None else out, self.width, T,
                           step.st, out16=rows16, sigmoid_gate=True)
@@ -478,7 +478,7 @@ class DecayedAttention:
         q, k, v, g = cols
         o = step.scratch("decay_o", T * self.width)
         # a portion longer than a range of the scan: per range and head its end state from zero and its token count (three passes)
-        blocks = step.chunk_scratch(c.heads, c.dim)
+        blocks = step.chunk_scratch(c.heads, c.dim, c.vdim)
         ws = None
         if blocks is None and T - step.nseg + 1 > self.scan_range:
             ws = step.scratch("decay_ranges", (step.b.n_qtiles // 4 + step.nseg + 1) * c.heads * (c.dim * c.vdim + 1))

@@ -90,12 +90,12 @@ class Step:
             self.turned.add(key)
         return table
 
-    def chunk_scratch(self, heads: int, dk: int):
+    def chunk_scratch(self, heads: int, dk: int, dv: int):
         """Scratch with which the recurrences walk this step's portions in blocks of tokens on the tensor cores, or None: the all-fp32 mode, steps
         without a portion worth a block, key heads the form does not take."""
         if not self.engine.tensor_cores or self.T - self.nseg + 1 < self.chunk_min_tokens:
             return None
-        n = self.engine.ops.chunk_ws_floats(self.b.n_qtiles, heads, dk)
+        n = self.engine.ops.chunk_ws_floats(self.b.n_qtiles, heads, dk, dv)
         return self.scratch("chunk_blocks", n) if n else None
 
     def gemm_scratch(self, K: int, N: int):
@@ -160,8 +160,8 @@ class SequenceEngine:
         if not self.free_slots:
             raise RuntimeError(f"all {self.max_seqs} state slots are in use")
         slot = self.free_slots.pop()
-        for t in self._slot_tensors:
-            t[slot].zero_()
+        if self._slot_tensors:
+            torch._foreach_zero_([t[slot] for t in self._slot_tensors])      # a few launches for all of them, not one each
         self.pos[slot] = 0
         self.last_token[slot] = -1
         self.live.add(slot)

@@ -238,9 +238,9 @@ class Ops:
         self._ck(self.lib.sllm_seq_delta_rule(C.byref(b), q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, _p(a_log), _p(dt_bias), heads,
                                               kv_heads, dk, dv, unit_eps, qscale, _p(state), _p(o), ldo, conv_x_ptr, ldx, channels, taps, _p(ring), _p(chunk_ws), st))
 
-    def chunk_ws_floats(self, n_qtiles, heads, dk):
+    def chunk_ws_floats(self, n_qtiles, heads, dk, dv):
         """Floats of scratch of the block form of the recurrences, 0 when these sizes have none."""
-        return (self.lib.sllm_seq_chunk_ws_bytes(n_qtiles, heads, dk) + 3) // 4
+        return (self.lib.sllm_seq_chunk_ws_bytes(n_qtiles, heads, dk, dv) + 3) // 4
 
     def channel_delta_rule(self, b, q_ptr, ldq, k_ptr, ldk, v_ptr, ldv, beta_ptr, ldb, step_ptr, lda, a_log, dt_bias, heads, kv_heads, dk, dv, unit_eps, qscale,
                            state, o, ldo, conv_x_ptr, ldx, channels, taps, ring, st, chunk_ws=None):

@@ -208,7 +208,7 @@ def _scan_stub(kind, H, G, dk, dv, consts, blocks):
         base, S = h.data_ptr(), states[0]["S"]
         q, k, v, bl, al = (base + o for o in offs)
         out = torch.empty(step.T, H * dv, device=dev)
-        ws = step.chunk_scratch(H, dk) if blocks else None
+        ws = step.chunk_scratch(H, dk, dv) if blocks else None
         assert (ws is not None) == (blocks and step.T - step.nseg + 1 >= step.chunk_min_tokens)
         if steps:
             rule = ops.channel_delta_rule if kind == "channel" else ops.delta_rule
