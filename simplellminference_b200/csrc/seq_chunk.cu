@@ -44,45 +44,64 @@ __device__ __forceinline__ void chunk_put(uint8_t* hi, uint8_t* lo, int at, cons
     reinterpret_cast<uint4*>(lo)[at] = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
-template <bool kDelta>
-__global__ void __launch_bounds__(kPrepThreads) seq_chunk_prepare_kernel(ChunkArgs p) {
+// vec: rows of q, k, v (and of the channels' steps) may be read 16 bytes at a time
+template <bool kDelta, int dkp>
+__global__ void __launch_bounds__(kPrepThreads) seq_chunk_prepare_kernel(ChunkArgs p, int vec) {
     extern __shared__ __align__(16) float cp_sm[];
     __shared__ float s_A[kChunk][kChunk + 1], s_B[kChunk][kChunk + 1], s_M[kChunk][kChunk + 1], s_beta[kChunk];
     const sllm_seq_batch& b = p.b;
     const ChunkPlace c = chunk_place(b, blockIdx.x);
     if (c.n <= 0) return;
-    const int h = blockIdx.y, kvh = h / (p.heads / p.kv_heads), dk = p.dk, dkp = chunk_key(dk), ld = dkp + 4;
+    const int h = blockIdx.y, kvh = h / (p.heads / p.kv_heads), dk = p.dk;
+    constexpr int ld = dkp + 4;
     float* s_k = cp_sm;                 // [16][ld]
     float* s_q = s_k + kChunk * ld;     // [16][ld]
     float* s_G = s_q + kChunk * ld;     // [16][ld], delta rule only
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const float rate = kDelta ? expf(p.A_log[h]) : p.rate[h];
     const float lg = -rate * kLog2e;    // constant decay: its base-2 logarithm
-    for (int i = threadIdx.x; i < kChunk * dkp; i += kPrepThreads) {
-        const int tok = i / dkp, ch = i % dkp;
-        const bool has = tok < c.n && ch < dk;
-        const size_t t = (size_t)(c.start + tok);
-        float kv = has ? p.k[t * p.ldk + (size_t)kvh * dk + ch] : 0.0f, qv = has ? p.q[t * p.ldq + (size_t)kvh * dk + ch] : 0.0f;
+    auto load4 = [&](const float* row, int ch, bool has) {             // channels ch .. ch + 3 of a row, zeros beyond the head
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (!has) return v;
+        if (vec && ch < dk) return *reinterpret_cast<const float4*>(row + ch);
+        if (ch < dk) v.x = row[ch];
+        if (ch + 1 < dk) v.y = row[ch + 1];
+        if (ch + 2 < dk) v.z = row[ch + 2];
+        if (ch + 3 < dk) v.w = row[ch + 3];
+        return v;
+    };
+    auto silu4 = [](float4 v) { return make_float4(v.x * seq_sigmoid(v.x), v.y * seq_sigmoid(v.y), v.z * seq_sigmoid(v.z), v.w * seq_sigmoid(v.w)); };
+    for (int i = threadIdx.x; i < kChunk * dkp / 4; i += kPrepThreads) {
+        const int tok = i / (dkp / 4), ch = (i % (dkp / 4)) * 4;
+        const bool has = tok < c.n;
+        const size_t t = (size_t)(c.start + (has ? tok : 0));
+        float4 kv = load4(p.k + t * p.ldk + (size_t)kvh * dk, ch, has), qv = load4(p.q + t * p.ldq + (size_t)kvh * dk, ch, has);
         if (!kDelta && p.silu) {
-            kv = kv * seq_sigmoid(kv);
-            qv = qv * seq_sigmoid(qv);
+            kv = silu4(kv);
+            qv = silu4(qv);
         }
-        s_k[tok * ld + ch] = kv;
-        s_q[tok * ld + ch] = qv;
+        *reinterpret_cast<float4*>(s_k + tok * ld + ch) = kv;
+        *reinterpret_cast<float4*>(s_q + tok * ld + ch) = qv;
         if (kDelta) {
-            float g = 0.0f;
-            if (has) {
-                const int at = p.channel ? h * dk + ch : h;
-                g = lg * seq_softplus(p.al[t * p.lda + at] + p.dt_bias[at]);
+            float4 g = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (has && p.channel) {
+                const float4 a = load4(p.al + t * p.lda + (size_t)h * dk, ch, true), bias = load4(p.dt_bias + (size_t)h * dk, ch, true);
+                g = make_float4(ch < dk ? lg * seq_softplus(a.x + bias.x) : 0.0f, ch + 1 < dk ? lg * seq_softplus(a.y + bias.y) : 0.0f,
+                                ch + 2 < dk ? lg * seq_softplus(a.z + bias.z) : 0.0f, ch + 3 < dk ? lg * seq_softplus(a.w + bias.w) : 0.0f);
+            } else if (has) {
+                g.x = g.y = g.z = g.w = lg * seq_softplus(p.al[t * p.lda + h] + p.dt_bias[h]);
             }
-            s_G[tok * ld + ch] = g;
+            *reinterpret_cast<float4*>(s_G + tok * ld + ch) = g;
         }
     }
     if (!kDelta && p.silu)                               // the values too, for the walk
-        for (int i = threadIdx.x; i < c.n * p.dv; i += kPrepThreads) {
-            const int tok = i / p.dv, j = i % p.dv;
-            const float v = p.v[(size_t)(c.start + tok) * p.ldv + (size_t)h * p.dv + j];
-            p.v_ws[((size_t)c.id * kChunk + tok) * p.heads * p.dv + (size_t)h * p.dv + j] = v * seq_sigmoid(v);
+        for (int tok = warp; tok < c.n; tok += kPrepThreads / 32) {
+            const float* src = p.v + (size_t)(c.start + tok) * p.ldv + (size_t)h * p.dv;
+            float* dst = p.v_ws + ((size_t)c.id * kChunk + tok) * p.heads * p.dv + (size_t)h * p.dv;
+            if (vec)
+                for (int j = 4 * lane; j < p.dv; j += 128) *reinterpret_cast<float4*>(dst + j) = silu4(*reinterpret_cast<const float4*>(src + j));
+            else
+                for (int j = lane; j < p.dv; j += 32) dst[j] = src[j] * seq_sigmoid(src[j]);
         }
     if (kDelta && threadIdx.x < kChunk) s_beta[threadIdx.x] = (int)threadIdx.x < c.n ? seq_sigmoid(p.bl[(size_t)(c.start + threadIdx.x) * p.ldb + h]) : 0.0f;
     __syncthreads();
@@ -174,7 +193,7 @@ __global__ void __launch_bounds__(kPrepThreads) seq_chunk_prepare_kernel(ChunkAr
     const int last = c.n - 1;
     // logarithm of the decay from the block's start to after token i, and from after token i to the block's end
     auto G = [&](int i, int ch) { return kDelta ? s_G[i * ld + ch] : lg * (float)(min(i, last) + 1); };
-    const int granules = dkp * 2;                        // 16-byte pieces of a plane: [k-step][lane]
+    constexpr int granules = dkp * 2;                    // 16-byte pieces of a plane: [k-step][lane]
     for (int x = threadIdx.x; x < 3 * granules; x += kPrepThreads) {
         const int which = x / granules, at = x % granules, ks = at >> 5, gr = (at & 31) >> 2, cc = at & 3;
         float v[8];
@@ -432,7 +451,15 @@ template <bool kDelta>
 static int launch_chunk_as(ChunkArgs p, cudaStream_t st) {
     const int dkp = chunk_key(p.dk);
     p.v_ws = reinterpret_cast<float*>(p.ws + 2 * (size_t)p.b.n_qtiles * p.heads * chunk_record_bytes(dkp));
-    seq_chunk_prepare_kernel<kDelta><<<dim3(2 * p.b.n_qtiles, p.heads), kPrepThreads, (size_t)3 * kChunk * (dkp + 4) * sizeof(float), st>>>(p);
+    auto aligned = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
+    const int vec_prep = p.dk % 4 == 0 && p.dv % 4 == 0 && p.ldq % 4 == 0 && p.ldk % 4 == 0 && p.ldv % 4 == 0 && aligned(p.q) && aligned(p.k) && aligned(p.v) &&
+                         (!p.channel || (p.lda % 4 == 0 && aligned(p.al) && aligned(p.dt_bias)));
+    const dim3 grid(2 * p.b.n_qtiles, p.heads);
+    const size_t smem = (size_t)3 * kChunk * (dkp + 4) * sizeof(float);
+    if (dkp == 32) seq_chunk_prepare_kernel<kDelta, 32><<<grid, kPrepThreads, smem, st>>>(p, vec_prep);
+    else if (dkp == 64) seq_chunk_prepare_kernel<kDelta, 64><<<grid, kPrepThreads, smem, st>>>(p, vec_prep);
+    else if (dkp == 96) seq_chunk_prepare_kernel<kDelta, 96><<<grid, kPrepThreads, smem, st>>>(p, vec_prep);
+    else seq_chunk_prepare_kernel<kDelta, 128><<<grid, kPrepThreads, smem, st>>>(p, vec_prep);
     ++g_launches;
     SLLM_LAUNCH_CHECK();
     const bool own_v = !kDelta && p.silu;

@@ -441,6 +441,85 @@ __global__ void __launch_bounds__(128) seq_conv_rotary_kv_kernel(ConvRotaryArgs 
     }
 }
 
+// The same for heads of up to 128 channels in interleaved pairs, 16-byte rows and up to four taps: a lane keeps four channels of its head in
+// registers over the tile of tokens — the weights, the last TAPS-1 inputs, the pairs that turn — and nothing passes through shared memory.
+template <typename KV, int TAPS>   // TAPS 0: no convolution
+__global__ void __launch_bounds__(128) seq_conv_rotary_kv_row_kernel(ConvRotaryArgs p) {
+    const sllm_seq_batch& b = p.b;
+    const int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (item >= p.heads + 2 * p.kv_heads) return;
+    const bool is_q = item < p.heads, is_v = item >= p.heads + p.kv_heads;
+    const int g = is_q ? item : (is_v ? item - p.heads - p.kv_heads : item - p.heads), width = is_v ? p.dv : p.dk;
+    const int ld = is_q ? p.ldq : (is_v ? p.ldv : p.ldk), j = 4 * lane;
+    const float* src = (is_q ? p.q : (is_v ? p.v : p.k)) + (size_t)g * width + j;
+    const int channels = (p.heads + p.kv_heads) * p.dk + p.kv_heads * p.dv;
+    const int ch = (is_q ? g * p.dk : (is_v ? (p.heads + p.kv_heads) * p.dk + g * p.dv : (p.heads + g) * p.dk)) + j;   // of the convolution
+    const bool live = j < width;
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    float4 w[TAPS > 0 ? TAPS : 1], past[TAPS > 0 ? TAPS : 1];      // [back]
+#pragma unroll
+    for (int back = 0; back < TAPS; ++back) w[back] = live ? *reinterpret_cast<const float4*>(p.conv_w + (size_t)(TAPS - 1 - back) * channels + ch) : zero;
+    KV* pool = reinterpret_cast<KV*>(is_v ? p.v_pool : p.k_pool);
+    const bool turns = !is_v && lane < (p.n_freq + 1) / 2;         // this lane holds pairs 2 * lane and 2 * lane + 1
+    const int t0 = blockIdx.x * p.tile, t1 = min(b.T, t0 + p.tile);
+    int prev_slot = -1;
+    float4 next = live ? *reinterpret_cast<const float4*>(src + (size_t)t0 * ld) : zero;
+    for (int t = t0; t < t1; ++t) {
+        const float4 own = next;
+        if (t + 1 < t1 && live) next = *reinterpret_cast<const float4*>(src + (size_t)(t + 1) * ld);     // travels while this token is finished
+        const int pos = b.tok_pos[t], slot = b.tok_slot[t];
+        float4 a = own;
+        if (TAPS > 0) {
+            if (slot != prev_slot) {                               // the tile's first token, or another sequence's
+                prev_slot = slot;
+#pragma unroll
+                for (int back = 1; back < TAPS; ++back) {
+                    past[back] = zero;
+                    if (live && pos - back >= 0)
+                        past[back] = (t - back >= 0 && b.tok_slot[t - back] == slot)
+                                         ? *reinterpret_cast<const float4*>(src + (size_t)(t - back) * ld)
+                                         : *reinterpret_cast<const float4*>(p.ring + ((size_t)slot * (TAPS - 1) + (pos - back) % (TAPS - 1)) * channels + ch);
+                }
+            }
+            a = make_float4(w[0].x * own.x, w[0].y * own.y, w[0].z * own.z, w[0].w * own.w);
+#pragma unroll
+            for (int back = 1; back < TAPS; ++back)
+                a = make_float4(fmaf(w[back].x, past[back].x, a.x), fmaf(w[back].y, past[back].y, a.y), fmaf(w[back].z, past[back].z, a.z), fmaf(w[back].w, past[back].w, a.w));
+            if (TAPS > 1) {
+                // single tokens: the oldest row of the ring, read above by this thread
+                if (p.store_ring && live) *reinterpret_cast<float4*>(p.ring + ((size_t)slot * (TAPS - 1) + pos % (TAPS - 1)) * channels + ch) = own;
+#pragma unroll
+                for (int back = TAPS - 1; back >= 2; --back) past[back] = past[back - 1];
+                past[TAPS > 1 ? 1 : 0] = own;
+            }
+        }
+        if (turns) {
+            const float2 r0 = p.angles[(size_t)t * p.n_freq + 2 * lane];
+            const float u0 = a.x, v0 = a.y;
+            a.x = u0 * r0.x - v0 * r0.y;
+            a.y = v0 * r0.x + u0 * r0.y;
+            if (2 * lane + 1 < p.n_freq) {
+                const float2 r1 = p.angles[(size_t)t * p.n_freq + 2 * lane + 1];
+                const float u1 = a.z, v1 = a.w;
+                a.z = u1 * r1.x - v1 * r1.y;
+                a.w = v1 * r1.x + u1 * r1.y;
+            }
+        }
+        if (!is_v && p.unit) {
+            const float ss = warp_sum(live ? fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, a.w * a.w))) : 0.0f);
+            const float inv = 1.0f / sqrtf(ss / (float)width + p.eps);
+            a = make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+        }
+        if (!live) continue;
+        if (is_q) {
+            *reinterpret_cast<float4*>(p.q_out + (size_t)t * p.ldqo + (size_t)g * width + j) = a;
+        } else {
+            const int page = b.block_table[(size_t)slot * b.max_pages + pos / b.page_len];
+            seq_st4(pool + seq_pool_row(page, p.kv_heads, g, b.page_len, pos % b.page_len, width) + j, a);
+        }
+    }
+}
+
 // thread = (token, head, column): out[t][h][c] = sum_g mix[h][g] * in[t][(h / group) * heads + g][c], group = heads / kv_heads: `in` holds,
 // for every key/value head, the result of EVERY query head's weights on that head's values
 __global__ void seq_head_mix_kernel(const float* __restrict__ in, int ldi, const float* __restrict__ mix, int heads, int kv_heads, int dv,
@@ -586,6 +665,22 @@ int sllm_seq_conv_rotary_kv(const sllm_seq_batch* b, const float* q, int32_t ldq
                      (const float2*)angles, n_freq, layout, unit, eps, q_out, ldqo, k_pool, v_pool, tile, vec};
     const dim3 grid((b->T + tile - 1) / tile, (heads + 2 * kv_heads + 3) / 4);
     const size_t smem = 4 * (size_t)((std::max(dk, dv) + 3) & ~3) * sizeof(float);
+    if (vec && layout == 0 && dk <= 128 && dv <= 128 && (!conv_w || taps <= 4)) {
+#define SLLM_ROW_LAUNCH(TAPS)                                                                                               \
+    do {                                                                                                                    \
+        if (kv_dtype == SLLM_F32) seq_conv_rotary_kv_row_kernel<float, TAPS><<<grid, 128, 0, as_stream(stream)>>>(p);       \
+        else seq_conv_rotary_kv_row_kernel<uint16_t, TAPS><<<grid, 128, 0, as_stream(stream)>>>(p);                         \
+    } while (0)
+        if (!conv_w) SLLM_ROW_LAUNCH(0);
+        else if (taps == 1) SLLM_ROW_LAUNCH(1);
+        else if (taps == 2) SLLM_ROW_LAUNCH(2);
+        else if (taps == 3) SLLM_ROW_LAUNCH(3);
+        else SLLM_ROW_LAUNCH(4);
+#undef SLLM_ROW_LAUNCH
+        ++g_launches;
+        SLLM_LAUNCH_CHECK();
+        return SLLM_OK;
+    }
     if (kv_dtype == SLLM_F32) seq_conv_rotary_kv_kernel<float><<<grid, 128, smem, as_stream(stream)>>>(p);
     else seq_conv_rotary_kv_kernel<uint16_t><<<grid, 128, smem, as_stream(stream)>>>(p);
     ++g_launches;
