@@ -118,3 +118,22 @@ def test_clamped_expert_of_the_restatement():
     w = {"e.gate": np.array([[10.0], [-10.0]]), "e.up": np.array([[10.0], [-10.0]]), "e.down": np.eye(2)}
     out = O.clamped_expert(np.array([[1.0]]), w, "e.", 2.0)[0]
     np.testing.assert_allclose(out, [2.0 / (1 + np.exp(-1.702 * 2.0)) * 3.0, -10.0 / (1 + np.exp(17.02)) * -1.0])   # the gate is bounded above only
+
+
+def test_bench_geometries():
+    """The throughput option's sizes are valid models: heads of 128, groups of experts, and tensors under the names the model asks for."""
+    import torch
+
+    from simplellminference_b200.bench_nelutar import EXPERTS, SIZES, _state_bytes, _used_params, nelutar_config, random_nelutar_weights
+    from simplellminference_b200.config import NelutarConfig
+    for size in SIZES.values():
+        c = NelutarConfig.from_dict(nelutar_config(size["width"], size["repeats"]))
+        assert c.width == size["width"] and [l.type for l in c.layers[:4]] == ["parallel_2", "parallel", "retention", "parallel_2"] and len(c.layers) == 4 * size["repeats"]
+        assert all(l.mlp.experts == EXPERTS for l in c.layers[1:4])
+    cfg = nelutar_config(256, 1, vocab=64)
+    cfg["embedding"]["bigram"]["buckets"] = 31
+    w = random_nelutar_weights(cfg, torch.device("cpu"))
+    used, total = _used_params(cfg, w)
+    assert 0 < used < total and _state_bytes(cfg, 4096) == _state_bytes(cfg, 2048) > 0
+    names = set(L.random_weights(cfg, seed=0))
+    assert set(w) == names

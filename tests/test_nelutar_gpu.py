@@ -588,6 +588,30 @@ def test_bf16_mode_within_operand_rounding(tmp_path, cfg):
     assert np.median(e) < BF16_MODEL_TYPICAL, np.median(e)
 
 
+def test_model_whose_layers_leave_bf16_rows_only(tmp_path, monkeypatch):
+    """With the tokens gathered per expert on the tensor cores nothing of a layer reads the normed rows in fp32: the seams leave bf16 rows alone,
+    and the logits are those of the form that computes every expert."""
+    from simplellminference_b200 import layers
+    cfg = L.make_config([L.lightning_pair(heads=4, kv_heads=2, dim=32, vdim=32, rot_dims=16, rheads=2, rdim=32, rvdim=64, mlp=L.moe(experts=8, top=2, ff=64, shared=64)),
+                         L.delta_pair(heads=2, kv_heads=1, dim=64, vdim=64, rot_dims=64, rheads=4, rkv=2, rdim=32, rvdim=32, mlp=L.moe(experts=4, top=1, ff=72, groups=2, keep=1))],
+                        width=64, vocab=128)
+    w = L.random_weights(cfg, seed=23)
+    toks = np.random.default_rng(24).integers(0, cfg["vocab"], size=200).tolist()
+    want, got, read = _forward(cfg, w, toks), {}, []
+    for gathers in (False, True):
+        monkeypatch.setattr(layers.ExpertsFeedForward, "gather_min_tokens", 64 if gathers else 10 ** 9)
+        monkeypatch.setattr(layers.ExpertsFeedForward, "gather_launch_cost", 0.0)
+        eng = _engine(tmp_path, cfg, w, dtype="bfloat16")
+        plain = layers.MixerGroup.reads_f32
+        monkeypatch.setattr(layers.MixerGroup, "reads_f32", lambda self, step, plain=plain: read.append(plain(self, step)) or read[-1])
+        read.clear()
+        got[gathers] = _logits(eng, eng.admit(), toks)
+        monkeypatch.setattr(layers.MixerGroup, "reads_f32", plain)
+        assert read and all(r != gathers for r in read)
+        assert np.median(L.logit_error(got[gathers], want)) < BF16_MODEL_TYPICAL
+    assert np.median(L.logit_error(got[True], got[False])) < BF16_MODEL_TYPICAL
+
+
 @pytest.mark.parametrize("cfg", ALL, ids=IDS)
 def test_prefill_against_token_by_token_and_portions(tmp_path, cfg):
     w = L.random_weights(cfg, seed=5)
