@@ -442,7 +442,7 @@ __global__ void __launch_bounds__(128) seq_conv_rotary_kv_kernel(ConvRotaryArgs 
 }
 
 // The same for heads of up to 128 channels in interleaved pairs, 16-byte rows and up to four taps: a lane keeps four channels of its head in
-// registers over the tile of tokens — the weights, the last TAPS-1 inputs, the pairs that turn — and nothing passes through shared memory.
+// registers — the weights over the tile of tokens, the pairs that turn — and nothing passes through shared memory.
 template <typename KV, int TAPS>   // TAPS 0: no convolution
 __global__ void __launch_bounds__(128) seq_conv_rotary_kv_row_kernel(ConvRotaryArgs p) {
     const sllm_seq_batch& b = p.b;
@@ -456,42 +456,29 @@ __global__ void __launch_bounds__(128) seq_conv_rotary_kv_row_kernel(ConvRotaryA
     const int ch = (is_q ? g * p.dk : (is_v ? (p.heads + p.kv_heads) * p.dk + g * p.dv : (p.heads + g) * p.dk)) + j;   // of the convolution
     const bool live = j < width;
     const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    float4 w[TAPS > 0 ? TAPS : 1], past[TAPS > 0 ? TAPS : 1];      // [back]
+    float4 w[TAPS > 0 ? TAPS : 1];                                 // [back]
 #pragma unroll
     for (int back = 0; back < TAPS; ++back) w[back] = live ? *reinterpret_cast<const float4*>(p.conv_w + (size_t)(TAPS - 1 - back) * channels + ch) : zero;
     KV* pool = reinterpret_cast<KV*>(is_v ? p.v_pool : p.k_pool);
     const bool turns = !is_v && lane < (p.n_freq + 1) / 2;         // this lane holds pairs 2 * lane and 2 * lane + 1
     const int t0 = blockIdx.x * p.tile, t1 = min(b.T, t0 + p.tile);
-    int prev_slot = -1;
-    float4 next = live ? *reinterpret_cast<const float4*>(src + (size_t)t0 * ld) : zero;
     for (int t = t0; t < t1; ++t) {
-        const float4 own = next;
-        if (t + 1 < t1 && live) next = *reinterpret_cast<const float4*>(src + (size_t)(t + 1) * ld);     // travels while this token is finished
+        const float4 own = live ? *reinterpret_cast<const float4*>(src + (size_t)t * ld) : zero;
         const int pos = b.tok_pos[t], slot = b.tok_slot[t];
         float4 a = own;
         if (TAPS > 0) {
-            if (slot != prev_slot) {                               // the tile's first token, or another sequence's
-                prev_slot = slot;
-#pragma unroll
-                for (int back = 1; back < TAPS; ++back) {
-                    past[back] = zero;
-                    if (live && pos - back >= 0)
-                        past[back] = (t - back >= 0 && b.tok_slot[t - back] == slot)
-                                         ? *reinterpret_cast<const float4*>(src + (size_t)(t - back) * ld)
-                                         : *reinterpret_cast<const float4*>(p.ring + ((size_t)slot * (TAPS - 1) + (pos - back) % (TAPS - 1)) * channels + ch);
-                }
-            }
             a = make_float4(w[0].x * own.x, w[0].y * own.y, w[0].z * own.z, w[0].w * own.w);
 #pragma unroll
-            for (int back = 1; back < TAPS; ++back)
-                a = make_float4(fmaf(w[back].x, past[back].x, a.x), fmaf(w[back].y, past[back].y, a.y), fmaf(w[back].z, past[back].z, a.z), fmaf(w[back].w, past[back].w, a.w));
-            if (TAPS > 1) {
-                // single tokens: the oldest row of the ring, read above by this thread
-                if (p.store_ring && live) *reinterpret_cast<float4*>(p.ring + ((size_t)slot * (TAPS - 1) + pos % (TAPS - 1)) * channels + ch) = own;
-#pragma unroll
-                for (int back = TAPS - 1; back >= 2; --back) past[back] = past[back - 1];
-                past[TAPS > 1 ? 1 : 0] = own;
+            for (int back = 1; back < TAPS; ++back) {              // the rows before it: this step's (near in the cache), the ring's, or nothing
+                if (live && pos - back >= 0) {
+                    const float4 x = (t - back >= 0 && b.tok_slot[t - back] == slot)
+                                         ? *reinterpret_cast<const float4*>(src + (size_t)(t - back) * ld)
+                                         : *reinterpret_cast<const float4*>(p.ring + ((size_t)slot * (TAPS - 1) + (pos - back) % (TAPS - 1)) * channels + ch);
+                    a = make_float4(fmaf(w[back].x, x.x, a.x), fmaf(w[back].y, x.y, a.y), fmaf(w[back].z, x.z, a.z), fmaf(w[back].w, x.w, a.w));
+                }
             }
+            // single tokens: the oldest row of the ring, read above by this thread
+            if (TAPS > 1 && p.store_ring && live) *reinterpret_cast<float4*>(p.ring + ((size_t)slot * (TAPS - 1) + pos % (TAPS - 1)) * channels + ch) = own;
         }
         if (turns) {
             const float2 r0 = p.angles[(size_t)t * p.n_freq + 2 * lane];

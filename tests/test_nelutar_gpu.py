@@ -145,6 +145,19 @@ def test_each_mixer_alone(portions):
         _check_alone(kind, kw, h, portions)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_each_mixer_alone_in_a_long_portion(dtype):
+    """Portions of more than 512 tokens (kernels that let a warp walk several tokens, more work than fits the machine at once), then more portions
+    and single tokens from the state they leave."""
+    h = L.bf16_round(np.random.default_rng(6).standard_normal((1215, 64))).astype(np.float32)
+    for kind, kw in (("attention", {}), ("attention", dict(dim=36, vdim=20, rot_dims=36, size=None)), ("unit_attention", {}), ("unit_attention", dict(conv=2, dim=24, vdim=20, size=70)),
+                     ("unit_attention", dict(conv=4, dim=32, vdim=32, rot_dims=32)), ("unit_attention", dict(conv=1)), ("unit_attention", dict(conv=6, heads=6, kv_heads=3)),
+                     ("unit_attention", dict(conv=0, dim=7, vdim=5, rot_dims=2)), ("delta", {}), ("delta", dict(rheads=2, rkv=1, rdim=40, rvdim=36, conv=4)), ("lightning", {}),
+                     ("retention", {})):
+        for portions in ([1215], [519, 2, 690, 1, 1, 2]):
+            _check_alone(kind, kw, h, portions, dtype=dtype, tol=F32_TOL if dtype == "float32" else BF16_MIXER, seed=13, max_tokens=1248)
+
+
 @pytest.mark.parametrize("portions", [[80], [40, 2, 37, 1]], ids=["whole", "portions"])
 def test_each_mixer_alone_bf16(portions):
     """bf16 matrices, operands and cache; portions of a prompt take the tensor-core attention where the head widths allow it."""
@@ -565,6 +578,23 @@ def test_whole_prompt_matches_oracle_fp32_and_layers(tmp_path, cfg):
         for i, (a, b) in enumerate(zip(taps, taps_want)):
             assert _rel(a, b) < F32_MODEL, (i, _rel(a, b))
         assert L.logit_error(got, want).max() < F32_MODEL
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_long_prompt_and_what_follows_it(tmp_path, dtype):
+    """700 tokens in one portion, then a short portion and single tokens from the caches and states it leaves."""
+    cfg = CFG_TC
+    w = L.random_weights(cfg, seed=27)
+    toks = np.random.default_rng(28).integers(0, cfg["vocab"], size=720).tolist()
+    want = _forward(cfg, w, toks)
+    eng = _engine(tmp_path, cfg, w, dtype=dtype, max_tokens=768, page_len=64)
+    s = eng.admit()
+    got = np.concatenate([_logits(eng, s, toks[:700]), _logits(eng, s, toks[700:709])] + [_logits(eng, s, toks[p:p + 1]) for p in range(709, 720)])
+    e = L.logit_error(got, want)
+    if dtype == "float32":
+        assert e.max() < F32_MODEL
+    else:
+        assert np.median(e) < BF16_MODEL_TYPICAL and np.median(e[700:]) < BF16_MODEL_TYPICAL and (e > 0.3).mean() < 0.1
 
 
 @pytest.mark.parametrize("cfg", [CFG_A, CFG_TC, CFG_ODD], ids=["mixed", "tensorcore", "odd"])
