@@ -38,7 +38,7 @@ def nelutar_config(width: int, repeats: int, vocab: int = 32000) -> dict:
     dense = {"kind": "dense", "ff": ff}
     moe = {"kind": "moe", "expert": {"ff": ff // 2, "limit": 7.0}, "shared": {"ff": ff // 2, "limit": 7.0},
            "router": {"experts": EXPERTS, "top": TOP, "scale": 2.5, "groups": {"count": GROUPS, "keep": KEEP}}}
-    pair2 = {"left": dict(attention, conv=4, softcap=30.0), "right": linear, "left_scale": 0.8, "right_scale": 1.1}
+    pair2 = {"left": dict(attention, conv=4, softcap=30.0), "right": linear, "left_scale": 0.9, "right_scale": 1.05}
     layers = [{"type": "parallel_2", "mixer": pair2, "mlp": dense},
               {"type": "parallel", "mixer": {"left": attention, "right": {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "conv": 4}}, "mlp": moe},
               {"type": "retention", "mixer": dict(linear, rot={"dims": 128, "base": 10000.0}), "mlp": moe},

@@ -69,7 +69,7 @@ def again(layers, j):
     return dict(layers[j], weights_of=j)
 
 
-def make_config(layers, vocab=83, width=48, eps=1e-5, buckets=53, mul_prev=31, mul_cur=7):
+def make_config(layers, vocab=83, width=48, eps=1e-5, buckets=53, mul_prev=29, mul_cur=11):
     return {"architecture": "Nelutar", "vocab": vocab, "width": width, "norm": {"eps": eps},
             "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}, "layers": layers}
 

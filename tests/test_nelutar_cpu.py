@@ -17,7 +17,7 @@ def test_config_reader(tmp_path):
     cfg = L.make_config(layers + [L.again(layers, 1)])
     c = read_model_config(L.write_model(str(tmp_path / "m"), cfg, {"embed": np.zeros((2, 2), np.float32)}))
     assert isinstance(c, NelutarConfig) and (c.vocab, c.width, c.norm_eps) == (83, 48, 1e-5)
-    assert (c.pair_buckets, c.pair_mul_prev, c.pair_mul_cur) == (53, 31, 7)
+    assert (c.pair_buckets, c.pair_mul_prev, c.pair_mul_cur) == (53, 29, 11)
     a, b, r, e, again = c.layers
     assert (a.left.heads, a.left.kv_heads, a.left.dim, a.left.vdim, a.left.scale, a.left.mask.size, a.left.rot) == (4, 2, 16, 12, 0.3, 20, RotaryConfig(8, 1000.0))
     assert a.right == DeltaRuleConfig(6, 3, 10, 14, 3) and a.mlp == ExpertsConfig(8, 0, 3, 12, 20, 0.9, 1.3, 4, 2, 1.5)
